@@ -80,10 +80,12 @@ class PagePool:
 @dataclass(frozen=True)
 class GroupSpec:
     """Layers whose caches live and die together: ``window`` None keeps every key; ``keep_first``: with a
-    window, the pages that hold a request's first ``keep_first`` keys are never given back."""
+    window, the pages that hold a request's first ``keep_first`` keys are never given back;
+    ``chunk``: positions see their own chunk of that many positions, and a chunk's pages go back with its end."""
     window: Optional[int]
     entries: tuple  # cache entries (layer runs) of this group
     keep_first: int = 0
+    chunk: Optional[int] = None
 
 
 class RequestCache:
@@ -185,6 +187,9 @@ class CacheManager:
         for g, spec in enumerate(self.groups):
             if spec.window is not None and getattr(spec, "keep_first", 0):
                 if self._lib.bw_cm_set_keep(self._h, g, int(spec.keep_first)) < 0:
+                    _raise()
+            if getattr(spec, "chunk", None):
+                if self._lib.bw_cm_set_chunk(self._h, g, int(spec.chunk)) < 0:
                     _raise()
         self.pools = [_PoolView(self, g, int(pages_per_group[g])) for g in range(n)]
         self._info_buf = (ctypes.c_int * (3 + 2 * max(n, 1)))()
@@ -356,13 +361,14 @@ class CacheManager:
 
 def groups_from_needs(needs: Sequence[object]) -> List[GroupSpec]:
     """Group cache entries by what must be kept: entries with paged keys and the same
-    window (and the same number of first keys kept beside it) share a group (and so a block table);
-    entries without paged keys form none."""
+    window (and the same number of first keys kept beside it) or the same chunks share a group (and so a
+    block table); entries without paged keys form none."""
     from ..parts.base import PagedKVNeed, PagedLatentNeed
     by_window: Dict[tuple, List[int]] = {}
     for e, need in enumerate(needs):
         if isinstance(need, (PagedKVNeed, PagedLatentNeed)):
             keep = int(getattr(need, "keep_first", 0) or 0) if need.window is not None else 0
-            by_window.setdefault((need.window, keep), []).append(e)
-    keys = sorted(by_window, key=lambda w: (w[0] is not None, w[0] or 0, w[1]))
-    return [GroupSpec(w, tuple(by_window[(w, k)]), k) for w, k in keys]
+            chunk = int(getattr(need, "chunk", None) or 0)
+            by_window.setdefault((need.window, keep, chunk), []).append(e)
+    keys = sorted(by_window, key=lambda w: (w[0] is not None or w[2] > 0, w[0] or 0, w[1], w[2]))
+    return [GroupSpec(w, tuple(by_window[(w, k, c)]), k, c or None) for w, k, c in keys]

@@ -71,3 +71,5 @@ def _ensure_builtin() -> None:
         from ..models import sebavik  # noqa: F401
     if "Kezuvik" not in _ARCHITECTURES:
         from ..models import kezuvik  # noqa: F401
+    if "Zuzupel" not in _ARCHITECTURES:
+        from ..models import zuzupel  # noqa: F401

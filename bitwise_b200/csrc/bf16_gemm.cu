@@ -190,10 +190,10 @@ gemm_bf16_kernel(const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __res
   auto store_out = [&](int gm, int gn, float v) {
     const size_t o = static_cast<size_t>(gm) * N + gn;
     if (residual) v = residual[o] + v;
-    if (y_is_f32)
+    if (y_is_f32 == 1)
       static_cast<float*>(Y)[o] = v;
     else
-      static_cast<__nv_bfloat16*>(Y)[o] = __float2bfloat16_rn(v);
+      static_cast<__nv_bfloat16*>(Y)[o] = __float2bfloat16_rn(bw::out_act(v, y_is_f32 >> 1));
   };
 
   if (!SPLIT || num_chunks == 1) {
@@ -305,7 +305,8 @@ BW_API int bw_bf16_linear_counters(int n) { return (n + kSplitBN - 1) / kSplitBN
 
 BW_API int bw_bf16_linear_split_rows() { return 128; }
 
-// One entry for every bfloat16 product. `use_legacy` != 0 forces the mma.sync tile (tests
+// One entry for every bfloat16 product. `y_is_f32`: 1 float32 outputs, 0 bfloat16, 2 a bfloat16 after the activation
+// a (bw::out_act). `use_legacy` != 0 forces the mma.sync tile (tests
 // compare the two variants bit for bit); otherwise the tcgen05 kernel runs whenever the rows
 // start on 16 bytes, and the legacy tile takes the remaining shapes (an inner size that is no
 // multiple of 8).

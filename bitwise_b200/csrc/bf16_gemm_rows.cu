@@ -320,7 +320,7 @@ linear_rows_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
           if (residual) v = res[e] + v;
           static_cast<float*>(Y)[at] = v;
         } else {
-          static_cast<__nv_bfloat16*>(Y)[at] = __float2bfloat16_rn(v);
+          static_cast<__nv_bfloat16*>(Y)[at] = __float2bfloat16_rn(EPI == 0 ? bw::out_act(v, act) : v);
         }
       }
     }
@@ -433,8 +433,8 @@ int launch_rows_epi(const __nv_bfloat16* x, const __nv_bfloat16* w, void* y, con
     return s.rows16 ? launch_rows<EPI, true, 2>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act)
                     : launch_rows<EPI, false, 2>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act);
   if (EPI == 1) return -1;  // SwiGLU tiles always hold two groups
-  return s.rows16 ? launch_rows<EPI == 1 ? 0 : EPI, true, 1>(x, w, y, residual, m, n, k, s, stream)
-                  : launch_rows<EPI == 1 ? 0 : EPI, false, 1>(x, w, y, residual, m, n, k, s, stream);
+  return s.rows16 ? launch_rows<EPI == 1 ? 0 : EPI, true, 1>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act)
+                  : launch_rows<EPI == 1 ? 0 : EPI, false, 1>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act);
 }
 
 }  // namespace
@@ -455,22 +455,22 @@ BW_API int bw_bf16_linear_rows_usable(const void* x, const void* w, int m, int n
          (!swiglu || n % 128 == 0) && rows_shape(m, n, k, swiglu != 0, &s) && rows_encoder() != nullptr;
 }
 
-// y_kind 0: y bfloat16 [m][n].  1: SwiGLU of interleaved gate/up weights, y bfloat16 [m][n / 2];
+// y_kind 0: y bfloat16 [m][n]; 4 * act: after the activation `act` (bw::out_act).  1: SwiGLU of interleaved gate/up weights, y bfloat16 [m][n / 2];
 // 1 + 4 * act: the same step with the gate's activation `act` (bw::glu_one).
 // 2: y float32 [m][n] = (residual +) product; y may alias residual.
 BW_API int bw_bf16_linear_rows(const __nv_bfloat16* x, const __nv_bfloat16* w, void* y, int y_kind, const float* residual,
                                int m, int n, int k, cudaStream_t stream) {
   if (m <= 0 || n <= 0) return 0;
   RowsShape s;
-  const int act = (y_kind & 3) == 1 ? y_kind >> 2 : 0;
-  if ((y_kind & 3) == 1) y_kind = 1;
+  const int act = y_kind >> 2;
+  y_kind &= 3;
   if (!bw_bf16_linear_rows_usable(x, w, m, n, k, y_kind == 1) || !rows_shape(m, n, k, y_kind == 1, &s)) {
     bw::set_error("linear (few rows): shape [%d x %d] x [%d x %d] is not for this path", m, k, n, k);
     return -1;
   }
   if (y_kind == 1) return launch_rows_epi<1>(x, w, y, nullptr, m, n, k, s, stream, act);
   if (y_kind == 2) return launch_rows_epi<2>(x, w, y, residual, m, n, k, s, stream);
-  return launch_rows_epi<0>(x, w, y, nullptr, m, n, k, s, stream);
+  return launch_rows_epi<0>(x, w, y, nullptr, m, n, k, s, stream, act);
 }
 
 // Whether the fused q/k/v projection of a step can rotate and store its outputs itself

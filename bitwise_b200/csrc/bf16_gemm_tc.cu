@@ -271,10 +271,10 @@ __global__ void reduce_chunks_kernel(const float* __restrict__ partials, int num
       if (c0 + e < num_chunks) v = (c0 + e == 0) ? p[e] : v + p[e];
   }
   if (residual) v = residual[o] + v;
-  if (y_is_f32)
+  if (y_is_f32 == 1)
     static_cast<float*>(Y)[o] = v;
   else
-    static_cast<__nv_bfloat16*>(Y)[o] = __float2bfloat16_rn(v);
+    static_cast<__nv_bfloat16*>(Y)[o] = __float2bfloat16_rn(bw::out_act(v, y_is_f32 >> 1));
 }
 
 // The ordered sum of the chunk sums of one output (shared by the reduce kernels below).
@@ -313,7 +313,8 @@ __global__ void reduce_swiglu_kernel(const float* __restrict__ partials, int num
 // EPI 0: y = product in bfloat16.  EPI 2: y = (residual +) product in float32.  EPI 1 (whole
 // mode only): the product is the interleaved gate/up projection and y[m][n / 2] = SwiGLU of it
 // (bfloat16), or the same step with another activation on the gate: with EPI 1 the argument
-// `y_is_f32` names the activation (bw::glu_one). In split mode the kernel writes chunk sums and the
+// `y_is_f32` names the activation (bw::glu_one); with EPI 0 it is twice the activation of the outputs
+// (bw::out_act). In split mode the kernel writes chunk sums and the
 // second kernel finishes.
 //
 // A wide tile has no path for pieces that are cut by the matrix edge or that do not start on
@@ -663,6 +664,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           }
         }
         continue;
+      }
+      if (EPI == 0 && !GROUPED && y_is_f32) {
+#pragma unroll
+        for (int j = 0; j < 2 * PW; ++j) total[j] = bw::out_act(total[j], y_is_f32 >> 1);
       }
 #pragma unroll
       for (int piece = 0; piece < 2; ++piece) {
@@ -1061,12 +1066,12 @@ BW_API int bw_bf16_linear_tc(const __nv_bfloat16* x, const __nv_bfloat16* w, voi
     bw::set_error("linear (tcgen05): rows must start on 16 bytes (k %% 8 == 0) and the driver must offer tensor maps");
     return -1;
   }
-  if (rows_path_takes(m, n, k, 0, x, w)) return bw_bf16_linear_rows(x, w, y, y_is_f32 ? 2 : 0, residual, m, n, k, stream);
+  if (rows_path_takes(m, n, k, 0, x, w)) return bw_bf16_linear_rows(x, w, y, y_is_f32 == 1 ? 2 : 4 * (y_is_f32 >> 1), residual, m, n, k, stream);
   int* word = bw::failure_word();
   if (!word) return -1;
   const Fused none;
-  if (y_is_f32) return launch_tc_rows<2>(x, w, y, 1, residual, m, n, k, word, partials, none, stream);
-  return launch_tc_rows<0>(x, w, y, 0, nullptr, m, n, k, word, partials, none, stream);
+  if (y_is_f32 == 1) return launch_tc_rows<2>(x, w, y, 1, residual, m, n, k, word, partials, none, stream);
+  return launch_tc_rows<0>(x, w, y, y_is_f32, nullptr, m, n, k, word, partials, none, stream);
 }
 
 // Grouped products on the tcgen05 kernel: y[i] = x[i] W_g^T for the rows i of group g, x holding

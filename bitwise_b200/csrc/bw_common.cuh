@@ -219,6 +219,19 @@ __device__ __forceinline__ float glu_one(float g, float u, int act) {
   return act == kGluGeluTanh ? geglu_one(g, u) : swiglu_one(g, u);
 }
 
+// What a product's finished output may pass before it is stored: 0 nothing, 1 the square of relu, 2 tanh (through the
+// hardware's exponential: the result is rounded to bfloat16 by the caller). One definition for the epilogues of the
+// products and the stand-alone kernel of the serving precision, so all of them give the same bits.
+constexpr int kOutNone = 0, kOutRelu2 = 1, kOutTanh = 2;
+__device__ __forceinline__ float out_act(float v, int act) {
+  if (act == kOutRelu2) {
+    const float r = fmaxf(v, 0.0f);
+    return __fmul_rn(r, r);
+  }
+  if (act == kOutTanh) return __fsub_rn(1.0f, __fdividef(2.0f, __fadd_rn(__expf(__fmul_rn(2.0f, v)), 1.0f)));
+  return v;
+}
+
 // The tail of RMSNorm for one element, and the scale from the sum of squares: one definition
 // for the stand-alone kernel and the fused one.
 __device__ __forceinline__ float rms_scale(float sumsq, int width, float eps) {

@@ -3,6 +3,7 @@
 //                  number per entry or one per group of neighbouring entries (a head)
 //   glu_gelu       the gated feed-forward's inner step with the tanh form of GELU:
 //                  h = gelu_tanh(gate) * up for rows laid out [gate | up]
+//   activate_rows  the square of relu, or tanh, of float32 rows, or the rows as they are, in the activation type
 //   softcap_rows   z <- cap * tanh(z / cap) on float32 rows (the logits' cap)
 #include "bw_act.cuh"
 
@@ -94,6 +95,20 @@ __global__ void softcap_rows_kernel(float* z, float cap, size_t count) {
   if (i < count) z[i] = __fmul_rn(cap, tanhf(__fdiv_rn(z[i], cap)));
 }
 
+// (in float32 `out` may be `x`, whose rows then lie next to each other)
+__global__ void activate_rows_kernel(const float* x, int cols, int x_stride, act_t* out, int act, size_t count) {
+  bw::pdl_enter();
+  const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i >= count) return;
+  const size_t r = i / cols;
+  const float v = x[r * x_stride + (i - r * cols)];
+#if BW_ACT_BF16
+  out[i] = bw::from_f<act_t>(bw::out_act(v, act));
+#else
+  out[i] = act == bw::kOutTanh ? tanhf(v) : bw::out_act(v, act);
+#endif
+}
+
 unsigned blocks_for(size_t count) { return static_cast<unsigned>((count + 255) / 256); }
 
 }  // namespace
@@ -125,6 +140,19 @@ BW_API int BW_FN(glu_gelu)(const void* gate_up, void* out, int n, int inter, cud
   const size_t count = static_cast<size_t>(n) * inter;
   bw::launch_pdl(glu_gelu_kernel, dim3(blocks_for(count)), dim3(256), 0, stream, static_cast<const act_t*>(gate_up),
                  static_cast<act_t*>(out), inter, count);
+  return bw::launch_status();
+}
+
+// act: 0 none (the rows are rounded), 1 the square of relu, 2 tanh.
+BW_API int BW_FN(activate_rows)(const float* x, int n, int cols, int x_stride, void* out, int act, cudaStream_t stream) {
+  if (n <= 0 || cols <= 0) return 0;
+  const size_t count = static_cast<size_t>(n) * cols;
+  if (act < bw::kOutNone || act > bw::kOutTanh) {
+    bw::set_error("activate_rows: unknown activation %d", act);
+    return -1;
+  }
+  bw::launch_pdl(activate_rows_kernel, dim3(blocks_for(count)), dim3(256), 0, stream, x, cols, x_stride,
+                 static_cast<act_t*>(out), act, count);
   return bw::launch_status();
 }
 

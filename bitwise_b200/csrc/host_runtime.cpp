@@ -79,6 +79,7 @@ struct RequestCache {
 
 struct CacheManager {
   std::vector<int> windows;  // per group: -1 keeps every key
+  std::vector<int> chunks;   // per group: > 0 where a position sees its own chunk of that many positions only
   std::vector<int> keep_blocks;  // per group: the first blocks of a request that a window never gives back
   int page_size;
   std::vector<PagePool> pools;
@@ -91,6 +92,7 @@ struct CacheManager {
     for (int g = 0; g < groups; ++g) {
       windows.push_back(win[g]);
       keep_blocks.push_back(0);
+      chunks.push_back(0);
       pools.emplace_back(pages[g]);
     }
     for (int s = slots - 1; s >= 0; --s) free_slots.push_back(s);
@@ -129,7 +131,7 @@ struct CacheManager {
   }
   // Record that `length` tokens are now cached; window groups give back the pages that no later
   // query can reach: the next query sits at position >= length and reads keys from
-  // length - window + 1 on.
+  // length - window + 1 on, or from the start of its chunk.
   int advance(int64_t rid, int length) {
     RequestCache* rc = find(rid);
     if (!rc) return fail("request is not live");
@@ -142,7 +144,7 @@ struct CacheManager {
     rc->length = length;
     for (size_t g = 0; g < pools.size(); ++g) {
       if (windows[g] < 0) continue;
-      const int first_needed = length - windows[g] + 1;
+      const int first_needed = chunks[g] > 0 ? length / chunks[g] * chunks[g] : length - windows[g] + 1;
       std::vector<int>& table = rc->tables[g];
       int& fl = rc->first_live[g];
       if (fl < keep_blocks[g]) fl = keep_blocks[g];  // blocks that hold kept first keys stay with the request
@@ -392,6 +394,16 @@ BW_HOST_API int bw_cm_set_keep(void* h, int group, int tokens) {
   CacheManager* m = static_cast<CacheManager*>(h);
   if (group < 0 || group >= static_cast<int>(m->keep_blocks.size()) || tokens < 0) return fail("no group %d", group);
   m->keep_blocks[group] = (tokens + m->page_size - 1) / m->page_size;
+  return 0;
+}
+
+// The group's positions see their own chunk of `size` positions only (counted from a request's first): a window group
+// whose pages go back as soon as the next position begins another chunk.
+BW_HOST_API int bw_cm_set_chunk(void* h, int group, int size) {
+  CacheManager* m = static_cast<CacheManager*>(h);
+  if (group < 0 || group >= static_cast<int>(m->chunks.size()) || size <= 0) return fail("no group %d, or chunks of %d", group, size);
+  m->chunks[group] = size;
+  m->windows[group] = size;
   return 0;
 }
 

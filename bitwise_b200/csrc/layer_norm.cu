@@ -49,7 +49,8 @@ layernorm_kernel(const float* x, const float* __restrict__ w1, const float* __re
 // x += (d - mean(d)) / sqrt(var(d) + eps) * w, with d the sublayer's output (float32) and x the
 // float32 stream; a constant factor on what is added is folded into w by the caller. Where the
 // next sublayer's layer norm follows at once, the same block forms it from the row it has just
-// summed: xn = (x - mean(x)) / sqrt(var(x) + eps') * w', one kernel instead of two.
+// summed: xn = (x - mean(x)) / sqrt(var(x) + eps') * w', one kernel instead of two. Without w' the
+// summed row itself, rounded to the activation type, goes into xn (the next sublayer reads the stream).
 __global__ void __launch_bounds__(kThreads)
 layernorm_residual_kernel(const float* __restrict__ d, const float* __restrict__ w, float* x, int width, float eps,
                           const float* __restrict__ w_next, float eps_next, act_t* xn) {
@@ -77,8 +78,9 @@ layernorm_residual_kernel(const float* __restrict__ d, const float* __restrict__
     x[base + i] = v;
     row[i] = v;  // (each thread reads back only what it wrote)
     s2 = __fadd_rn(s2, v);
+    if (xn && !w_next) xn[base + i] = bw::from_f<act_t>(v);
   }
-  if (!xn) return;
+  if (!xn || !w_next) return;
   const float mean2 = __fdiv_rn(bw::block_sum(s2, red), fw);
   float q2 = 0.0f;
   for (int i = threadIdx.x; i < width; i += kThreads) {
@@ -117,7 +119,8 @@ BW_API int BW_FN(layernorm)(const float* x, const float* w1, const float* w2, vo
   return bw::launch_status();
 }
 
-// w_next, xn: the layer norm of the summed row into xn (activation type) as well; both null for none.
+// w_next, xn: the layer norm of the summed row into xn (activation type) as well; both null for none; xn
+// alone: the summed row, rounded.
 BW_API int BW_FN(layernorm_residual)(const float* d, const float* w, float* x, int n, int width, float eps,
                                      const float* w_next, float eps_next, void* xn, cudaStream_t stream) {
   if (n <= 0) return 0;
@@ -126,7 +129,7 @@ BW_API int BW_FN(layernorm_residual)(const float* d, const float* w, float* x, i
     return -1;
   }
   bw::launch_pdl(layernorm_residual_kernel, dim3(n), dim3(kThreads), static_cast<size_t>(width) * sizeof(float), stream,
-                 d, w, x, width, eps, w_next, eps_next, static_cast<act_t*>(w_next ? xn : nullptr));
+                 d, w, x, width, eps, w_next, eps_next, static_cast<act_t*>(xn));
   return bw::launch_status();
 }
 

@@ -4,11 +4,11 @@
 //   qkv_prepare        per row and head: a short causal convolution over time on every channel of
 //                      the projected q, k, v (inputs before the step's first row come from the
 //                      request's state slot), a root-mean-square norm per head of q and k, the
-//                      rotation of the leading entries of q and k (pair i = entries 2i, 2i + 1), q
-//                      into the step's buffer, k and v into their pages
+//                      rotation of the leading entries of q and k (pair i = entries 2i, 2i + 1, or i and
+//                      i + pairs), q into the step's buffer, k and v into their pages
 //   conv_state_update  the convolution's inputs of a request's last taps - 1 positions
 //   scored_attention   s = (q . k) * scale; s <- cap * tanh(s / cap); s <- s - slope_h * (i - j);
-//                      window; softmax with an optional extra one in the denominator; the values
+//                      window or chunks; softmax with an optional extra one in the denominator; the values
 //                      may be the keys themselves (no value pages)
 //
 // Everything after the projection is float32 in both precisions; only what is loaded and stored
@@ -45,6 +45,7 @@ struct PrepArgs {
   const float* cos_t;        // [positions, pairs] or null
   const float* sin_t;
   int pairs;
+  int half_layout;           // pair i is made of entries i and i + pairs instead of 2i and 2i + 1
   const int* pos;
   const int* row_seq;
   const int* seq_row0;
@@ -60,6 +61,7 @@ struct PrepArgs {
 
 __global__ void __launch_bounds__(kPrepWarps * 32) qkv_prepare_kernel(const PrepArgs a) {
   bw::pdl_enter();
+  __shared__ float heads_sm[kPrepWarps][kMaxE * 32];  // a head at a time, for partners that other lanes hold
   const int r = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p = a.pos[r];
@@ -123,7 +125,26 @@ __global__ void __launch_bounds__(kPrepWarps * 32) qkv_prepare_kernel(const Prep
         if (e < size) val[j] = bw::rms_apply(val[j], inv, norm_w[e]);
       }
     }
-    if (turns && a.pairs > 0) {
+    if (turns && a.pairs > 0 && a.half_layout) {
+      float* hv = heads_sm[warp];
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < kMaxE; ++j)
+        if (lane + 32 * j < size) hv[lane + 32 * j] = val[j];
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < kMaxE; ++j) {
+        const int e = lane + 32 * j;
+        if (e < 2 * a.pairs && e < size) {
+          const bool second = e >= a.pairs;
+          const int i = second ? e - a.pairs : e;
+          const float other = hv[second ? i : i + a.pairs];
+          const float c = a.cos_t[static_cast<size_t>(p) * a.pairs + i], s = a.sin_t[static_cast<size_t>(p) * a.pairs + i];
+          val[j] = second ? __fadd_rn(__fmul_rn(val[j], c), __fmul_rn(other, s))
+                          : __fsub_rn(__fmul_rn(val[j], c), __fmul_rn(other, s));
+        }
+      }
+    } else if (turns && a.pairs > 0) {
 #pragma unroll
       for (int j = 0; j < kMaxE; ++j) {
         const int e = lane + 32 * j;
@@ -170,6 +191,7 @@ __device__ __forceinline__ void store4(float* dst, float4 v) { *reinterpret_cast
 
 __global__ void __launch_bounds__(kPrepWarps * 32) qkv_prepare_vec_kernel(const PrepArgs a) {
   bw::pdl_enter();
+  __shared__ __align__(16) float heads_sm[kPrepWarps][kMaxE * 32];
   const int r = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p = a.pos[r];
@@ -244,7 +266,30 @@ __global__ void __launch_bounds__(kPrepWarps * 32) qkv_prepare_vec_kernel(const 
         }
       }
     }
-    if (turns && a.pairs > 0) {
+    if (turns && a.pairs > 0 && a.half_layout) {
+      float* hv = heads_sm[warp];
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (4 * lane + 128 * j < size) *reinterpret_cast<float4*>(hv + 4 * lane + 128 * j) = val[j];
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        float* f = &val[j].x;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int e = 4 * lane + 128 * j + k;
+          if (e < 2 * a.pairs && e < size) {
+            const bool second = e >= a.pairs;
+            const int i = second ? e - a.pairs : e;
+            const float other = hv[second ? i : i + a.pairs];
+            const float c = a.cos_t[static_cast<size_t>(p) * a.pairs + i], s = a.sin_t[static_cast<size_t>(p) * a.pairs + i];
+            f[k] = second ? __fadd_rn(__fmul_rn(f[k], c), __fmul_rn(other, s))
+                          : __fsub_rn(__fmul_rn(f[k], c), __fmul_rn(other, s));
+          }
+        }
+      }
+    } else if (turns && a.pairs > 0) {
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int e0 = 4 * lane + 128 * j;
@@ -336,7 +381,13 @@ struct ScoreArgs {
   const float* dist_b;
   const float* sinks;   // [heads] or null: with `sink`, exp(sinks[h]) joins the denominator instead of exp(0)
   int keep_first;       // with a window: the keys j < keep_first stay visible to every later position
+  int chunk;            // > 0: position i sees the keys j <= i with j / chunk == i / chunk (no window then)
 };
+// The first key that a query at position pq sees (kept first keys apart). It never falls as pq grows.
+__device__ __forceinline__ int first_seen(const ScoreArgs& sa, int pq) {
+  if (sa.chunk > 0) return pq / sa.chunk * sa.chunk;
+  return sa.window > 0 ? max(0, pq - sa.window + 1) : 0;
+}
 
 // What a query's head takes off a score by distance.
 struct HeadBias {
@@ -420,7 +471,7 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
     for (int i = 0; i < ACC; ++i) acc[j][i] = 0.0f;
   }
   const int last = p0 + rows - 1;
-  const int first = sa.window > 0 ? max(0, p0 - sa.window + 1) : 0;  // pages before it may be gone (kept first keys stay)
+  const int first = first_seen(sa, p0);  // pages before it may be gone (kept first keys stay)
   const int keep = sa.window > 0 ? sa.keep_first : 0;
   const int keep_end = (keep + kKeys - 1) / kKeys * kKeys, win_begin = first / kKeys * kKeys;
   const int* bt = block_table + static_cast<size_t>(seq) * max_blocks;
@@ -441,7 +492,7 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
       const int qi = warp + kWarps * j;
       if (qi >= nq) continue;
       const int pq = p0 + qi / nh;
-      const int lo = sa.window > 0 ? max(0, pq - sa.window + 1) : 0;
+      const int lo = first_seen(sa, pq);
       if (k0 > pq || (k0 + kKeys <= lo && k0 >= keep)) continue;  // no key of the tile is seen: the state stays
       const int kp = k0 + lane;
       const float* qv = qs + qi * dim;
@@ -554,30 +605,32 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   const int sr_a = warp * 16 + (lane >> 2), sr_b = sr_a + 8;
   const bool ok_a = sr_a < nq, ok_b = sr_b < nq;
   const int pq_a = p0 + (ok_a ? sr_a / nh : 0), pq_b = p0 + (ok_b ? sr_b / nh : 0);
-  const int lo_a = sa.window > 0 ? max(0, pq_a - sa.window + 1) : 0, lo_b = sa.window > 0 ? max(0, pq_b - sa.window + 1) : 0;
+  const int lo_a = first_seen(sa, pq_a), lo_b = first_seen(sa, pq_b);
   const HeadBias slope_a = head_bias(sa, h0 + sr_a % nh, ok_a), slope_b = head_bias(sa, h0 + sr_b % nh, ok_b);
   const int keep = sa.window > 0 ? sa.keep_first : 0;
   // the positions that this warp's queries span: tiles outside are skipped by the whole warp
   const int w_first = min(warp * 16, max(nq - 1, 0)) / nh, w_last = min(warp * 16 + 15, max(nq - 1, 0)) / nh;
-  const int w_lo = sa.window > 0 ? max(0, p0 + w_first - sa.window + 1) : 0, w_hi = p0 + w_last;
+  const int w_lo = first_seen(sa, p0 + w_first), w_hi = p0 + w_last;
   const bool warp_has_rows = warp * 16 < nq;
   const bool warp_full = warp * 16 + 15 < nq;  // all 16 stacked rows of the warp are queries
   const int w_seen_to = p0 + w_first;           // keys up to here are seen by every query of the warp ...
-  const int w_seen_from = sa.window > 0 ? max(0, p0 + w_last - sa.window + 1) : 0;  // ... from here on
+  const int w_seen_from = first_seen(sa, p0 + w_last);  // ... from here on
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
   float acc[VT][4];
 #pragma unroll
   for (int j = 0; j < VT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
   const int last = p0 + rows - 1;
-  const int first = sa.window > 0 ? max(0, p0 - sa.window + 1) : 0;  // pages before it may be gone (kept first keys stay)
+  const int first = first_seen(sa, p0);  // pages before it may be gone (kept first keys stay)
   const int keep_end = (keep + kMmaKeys - 1) / kMmaKeys * kMmaKeys, win_begin = first / kMmaKeys * kMmaKeys;
   const int* bt = block_table + static_cast<size_t>(seq) * max_blocks;
-  // With spans the block walks the key tiles span * span_tiles .. + span_tiles - 1 only (fixed
-  // absolute positions again) and leaves a record for the merge instead of the result.
+  // With spans the block walks the key tiles at * span_tiles .. + span_tiles - 1 only (fixed absolute positions
+  // again) and leaves a record for the merge instead of the result. Where the tile's queries see nothing before
+  // their first key, the spans are counted from the one that holds it.
   int k_begin = skip_gap(0, keep_end, win_begin), k_end = last;
   if (span_tiles > 0) {
-    k_begin = skip_gap(max(k_begin, span * span_tiles * kMmaKeys), keep_end, win_begin);
-    k_end = min(k_end, (span + 1) * span_tiles * kMmaKeys - 1);
+    const int at = span + (keep > 0 ? 0 : first / (span_tiles * kMmaKeys));
+    k_begin = skip_gap(max(k_begin, at * span_tiles * kMmaKeys), keep_end, win_begin);
+    k_end = min(k_end, (at + 1) * span_tiles * kMmaKeys - 1);
     if (k_begin > k_end) {
       // none of the block's queries reaches into this span: records that say so, nothing else
       for (int sr = tid; sr < nq; sr += kMmaWarps * 32) {
@@ -856,7 +909,7 @@ BW_API int BW_FN(qkv_prepare)(const float* u, int cols, const float* conv_w, con
                               const int* seq_slot, const int* block_table, int max_blocks, void* kcache, void* vcache,
                               void* q_out, int n, int heads, int kv_heads, int dim, int vdim, int page,
                               const float* bias, const float* vmix_src, const float* vmix_lambda, float* v_keep,
-                              int u_stride, cudaStream_t stream) {
+                              int u_stride, int half_layout, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (u_stride < cols) {
     bw::set_error("qkv_prepare: rows %d floats apart do not hold %d columns", u_stride, cols);
@@ -875,6 +928,7 @@ BW_API int BW_FN(qkv_prepare)(const float* u, int cols, const float* conv_w, con
   a.u = u, a.cols = cols, a.u_stride = u_stride, a.conv_w = conv_w, a.conv_wt = conv_w ? conv_wt : nullptr, a.taps = taps;
   a.conv_state = taps > 1 ? conv_state : nullptr;
   a.q_norm = q_norm, a.k_norm = k_norm, a.eps = eps, a.cos_t = cos_t, a.sin_t = sin_t, a.pairs = cos_t ? pairs : 0;
+  a.half_layout = half_layout;
   a.pos = pos, a.row_seq = row_seq, a.seq_row0 = seq_row0, a.seq_pos0 = seq_pos0, a.seq_slot = seq_slot;
   a.block_table = block_table, a.max_blocks = max_blocks;
   a.kcache = static_cast<act_t*>(kcache), a.vcache = static_cast<act_t*>(vcache), a.q_out = static_cast<act_t*>(q_out);
@@ -916,7 +970,8 @@ BW_API int BW_FN(scored_attention)(const void* q, int q_stride, const void* kcac
                                    const int* tile_rows, int tiles, const int* seq_pos0, const int* seq_row0, void* out,
                                    int o_stride, int heads, int kv_heads, int dim, int vdim, int page, float scale,
                                    float softcap, int sink, const float* slopes, int window, const float* dist_a,
-                                   const float* dist_b, const float* sinks, int keep_first, cudaStream_t stream) {
+                                   const float* dist_b, const float* sinks, int keep_first, int chunk,
+                                   cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (kv_heads <= 0 || heads % kv_heads) {
     bw::set_error("scored_attention: %d heads on %d key/value heads", heads, kv_heads);
@@ -938,6 +993,7 @@ BW_API int BW_FN(scored_attention)(const void* q, int q_stride, const void* kcac
   ScoreArgs sa;
   sa.scale = scale, sa.softcap = softcap, sa.sink = sink, sa.slopes = slopes, sa.window = window;
   sa.dist_a = dist_a, sa.dist_b = dist_a ? dist_b : nullptr, sa.sinks = sinks, sa.keep_first = window > 0 ? keep_first : 0;
+  sa.chunk = chunk;
   sa.cap_exp = 0.0f;  // (the tensor-core kernel's)
   const dim3 grid(tiles, kv_heads, (rep + hb - 1) / hb);
 #define BW_SCORED(A)                                                                                                      \
@@ -974,7 +1030,7 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
                                         int o_stride, int heads, int kv_heads, int dim, int vdim, int page, float scale,
                                         float softcap, int sink, const float* slopes, int window, int n, int spans,
                                         float* partial, const float* dist_a, const float* dist_b, const float* sinks,
-                                        int keep_first, cudaStream_t stream) {
+                                        int keep_first, int chunk, cudaStream_t stream) {
   // spans > 1 (`partial` holding n * heads * spans * (vdim + 2) floats): every query's keys are spread
   // over blocks of kSpanTiles key tiles each, at fixed absolute positions, and a second kernel joins
   // the spans' records in ascending order.
@@ -990,6 +1046,7 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
   ScoreArgs sa;
   sa.scale = scale, sa.softcap = softcap, sa.sink = sink, sa.slopes = slopes, sa.window = window;
   sa.dist_a = dist_a, sa.dist_b = dist_a ? dist_b : nullptr, sa.sinks = sinks, sa.keep_first = window > 0 ? keep_first : 0;
+  sa.chunk = chunk;
   sa.cap_exp = softcap > 0.0f ? 2.0f * scale / softcap * 1.4426950408889634f : 0.0f;
   const bool split = spans > 1 && partial != nullptr;
   if (!split) spans = 1;
@@ -1014,9 +1071,15 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
   return bw::launch_status();
 }
 
-// Spans that a step of single rows with contexts of up to max_keys keys is spread over.
-BW_API int bw_bf16_scored_attention_spans(int max_keys) {
+// Spans that the queries of a step with contexts of up to max_keys keys are spread over. `reach` > 0: a query sees at
+// most that many keys, itself the last; query tiles hold `tile_rows` rows. (A tile then spans reach + tile_rows - 1 keys, which
+// touch at most one span more than they would fill.)
+BW_API int bw_bf16_scored_attention_spans(int max_keys, int reach, int tile_rows) {
   const int per = kSpanTiles * kMmaKeys;
-  return (max_keys + per - 1) / per;
+  const int all = (max_keys + per - 1) / per;
+  if (reach <= 0) return all;
+  const long long keys = static_cast<long long>(reach) + tile_rows - 1;
+  const long long near = (keys + per - 2) / per + 1;
+  return near < all ? static_cast<int>(near) : all;
 }
 #endif  // BW_ACT_BF16

@@ -1,0 +1,704 @@
+// Mixers whose memory is one matrix per head: three recurrences over the tokens of a sequence on one
+// kernel, what prepares their operands, and what finishes their outputs. Per head the state S is
+// dim x vdim float32 numbers of a request (zero before its first token):
+//
+//   delta    S <- g S (g per key channel), then S <- S + k (beta (v - S^T k))^T, then o = S^T q
+//   bonus    o = (S + diag(u) k v^T)^T q, then S <- diag(w) S + k v^T, w = exp(-exp(z + z0))
+//   memory   m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, the normaliser n alike with
+//            k alone, o = S^T q (divided later by max(|n . q|, e^-m) + 1e-6)
+//
+// The columns of S (one per value channel) do not meet inside a token, so a block walks the rows of one
+// sequence of the step for one head and a few columns, from the state that the request's slot holds.
+// LP lanes of a warp share a column; a lane holds V groups of four consecutive rows (group p + LP i).
+// A sum over a column's rows is a chain per lane and a butterfly over the LP lanes, in an order given
+// by dim alone. The tokens' operands are copied into shared memory a chunk ahead (cp.async, two buffers);
+// the chunk is a staging unit only: every S and o is the same chain of operations wherever the step's
+// rows begin and end, so a position's result does not depend on how its prompt was cut.
+// Everything here is float32 in both precisions; only what enters the next product changes type.
+#include "bw_act.cuh"
+#include "bw_mma.cuh"
+
+#include <math.h>
+
+namespace {
+
+constexpr int kThreads = 128;
+enum { kDelta = 0, kBonus = 1, kMemory = 2 };
+
+// The serving precision takes the hardware's exponential (relative error about 1e-7 times the exponent's size, far
+// below that of the bfloat16 operands of the products before it).
+__device__ __forceinline__ float exp_f(float x) {
+#if BW_ACT_BF16
+  return __expf(x);
+#else
+  return expf(x);
+#endif
+}
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z))); }
+// ln(1 + e^z) without overflow
+__device__ __forceinline__ float softplus_f(float z) { return __fadd_rn(fmaxf(z, 0.0f), log1pf(expf(-fabsf(z)))); }
+
+__device__ __forceinline__ void copy4_async(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(bw::smem_addr(dst)), "l"(src));
+}
+__device__ __forceinline__ void copy16_async(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(bw::smem_addr(dst)), "l"(src));
+}
+
+struct ScanArgs {
+  const float* q;          // row r, head h / rep: q + r * q_stride + (h / rep) * dim
+  const float* k;
+  const float* v;          // row r, head h: v + r * v_stride + h * vdim
+  int q_stride, k_stride, v_stride;
+  int rep;                 // heads that share a q/k head
+  const float* decay;      // delta: g; bonus: z. Row r, head h: decay + r * decay_stride + h * dim
+  int decay_stride;
+  const float* decay_bias;  // bonus: z0 [heads * dim]
+  const float* bonus;      // bonus: u [heads * dim]
+  const float* s0;         // delta: beta; memory: the forget gate's projection. Row r, head h: s0 + r * s_stride + h
+  const float* s1;         // memory: the input gate's projection
+  int s_stride;
+  const float* s0_bias;    // memory: [heads]
+  const float* s1_bias;
+  float cap;               // memory: gates are cap * tanh(. / cap)
+  float* state;            // [slots, heads, columns, column]: delta, bonus: vdim columns of dim; memory: vdim + 1
+                           // columns of dim + 4 (the last column is n; entry dim of every column is m)
+  float* o;                // [n, heads * vdim]
+  float* aux;              // memory: [n, heads, 2]: n . q and m
+  const int* tile_seq;
+  const int* tile_row0;
+  const int* tile_rows;
+  const int* seq_pos0;
+  const int* seq_slot;
+  int heads, dim, vdim, chunk, wide;
+};
+
+// Sums x[0 .. G - 1] over the LP lanes of a column at once: afterwards lane p holds the sum of x[p / (LP / G)]. Each
+// sum is the butterfly over lane distances LP / 2, LP / 4, .. 1 (a + b and b + a are the same bits), as below.
+template <int LP, int G>
+__device__ __forceinline__ float group_sum(float (&x)[G], int p) {
+  int off = LP / 2;
+#pragma unroll
+  for (int n = G; n > 1; n /= 2) {
+    const bool up = (p & off) != 0;
+#pragma unroll
+    for (int i = 0; i < n / 2; ++i) {
+      const float send = up ? x[i] : x[i + n / 2], keep = up ? x[i + n / 2] : x[i];
+      x[i] = __fadd_rn(keep, __shfl_xor_sync(0xffffffffu, send, off));
+    }
+    off /= 2;
+  }
+#pragma unroll
+  for (; off > 0; off /= 2) x[0] = __fadd_rn(x[0], __shfl_xor_sync(0xffffffffu, x[0], off));
+  return x[0];
+}
+template <int LP>
+__device__ __forceinline__ float column_sum(float x) {
+#pragma unroll
+  for (int off = LP / 2; off > 0; off /= 2) x = __fadd_rn(x, __shfl_xor_sync(0xffffffffu, x, off));
+  return x;
+}
+
+template <int MODE, int LP, int V>
+struct Shape {
+  static constexpr int CB = kThreads / LP;   // columns of a block
+  static constexpr int DP = LP * 4 * V;      // rows held; those from dim on are zero
+  static constexpr int VECS = MODE == kMemory ? 2 : 3;
+  static constexpr int SC = VECS * DP + CB;  // where a token's scalars start
+  static constexpr int W = SC + 4;           // a staged token: k | q | decay | values | scalars
+  static constexpr int G = LP < 8 ? LP : 8;  // tokens whose outputs are summed together
+};
+
+template <int V>
+struct Rows {
+  float v[4 * V];
+};
+template <int LP, int V>
+__device__ __forceinline__ Rows<V> load_rows(const float* at, int p) {
+  Rows<V> r;
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const float4 f = *reinterpret_cast<const float4*>(at + 4 * (p + LP * i));
+    r.v[4 * i] = f.x, r.v[4 * i + 1] = f.y, r.v[4 * i + 2] = f.z, r.v[4 * i + 3] = f.w;
+  }
+  return r;
+}
+// Two chains (even and odd entries) and their sum.
+template <int V>
+__device__ __forceinline__ float dot(const Rows<V>& a, const Rows<V>& b) {
+  float e = 0.0f, o = 0.0f;
+#pragma unroll
+  for (int i = 0; i < 4 * V; i += 2) {
+    e = __fmaf_rn(a.v[i], b.v[i], e);
+    o = __fmaf_rn(a.v[i + 1], b.v[i + 1], o);
+  }
+  return __fadd_rn(e, o);
+}
+
+template <int MODE, int LP, int V>
+__global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) {
+  typedef Shape<MODE, LP, V> T;
+  const bool few = gridDim.x * gridDim.y * gridDim.z <= 296;
+  if (few) bw::pdl_launch();
+  extern __shared__ __align__(16) float sm[];
+  const int dim = a.dim, vdim = a.vdim, chunk = a.chunk;
+  float* stage = sm;                            // [2][chunk][W]
+  float* outs = sm + 2 * chunk * T::W;          // [chunk][CB]
+  const int t = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * T::CB;
+  const int seq = a.tile_seq[t], row0 = a.tile_row0[t], cnt = a.tile_rows[t];
+  const int tid = threadIdx.x;
+  const int p = tid & (LP - 1), c = c0 + tid / LP;
+  constexpr bool kMem = MODE == kMemory;
+  const int cols = kMem ? vdim + 1 : vdim, col_size = kMem ? dim + 4 : dim;
+  const bool col_ok = c < cols;
+  float* head_state = a.state + (static_cast<size_t>(a.seq_slot[seq]) * a.heads + h) * cols * col_size;
+  float* sp = head_state + static_cast<size_t>(c) * col_size;
+  const bool fresh = a.seq_pos0[seq] == 0;      // a slot is handed out as its last holder left it
+  // The state of this run was written by the step before, so it is asked for before the wait for this step's kernels.
+  Rows<V> S;
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const int row = 4 * (p + LP * i);
+    float4 f = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (!fresh && col_ok) {
+      if (a.wide) {
+        if (row < dim) f = *reinterpret_cast<const float4*>(sp + row);
+      } else {
+        if (row < dim) f.x = sp[row];
+        if (row + 1 < dim) f.y = sp[row + 1];
+        if (row + 2 < dim) f.z = sp[row + 2];
+        if (row + 3 < dim) f.w = sp[row + 3];
+      }
+    }
+    S.v[4 * i] = f.x, S.v[4 * i + 1] = f.y, S.v[4 * i + 2] = f.z, S.v[4 * i + 3] = f.w;
+  }
+  float m = 0.0f;  // memory: the running maximum (held by every thread of warp 0)
+  if (kMem && !fresh) m = head_state[static_cast<size_t>(c0) * col_size + dim];
+  Rows<V> bonus;
+  if (MODE == kBonus) {
+#pragma unroll
+    for (int i = 0; i < V; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int row = 4 * (p + LP * i) + e;
+        bonus.v[4 * i + e] = row < dim ? a.bonus[h * dim + row] : 0.0f;
+      }
+  }
+  for (int i = tid; i < 2 * chunk * T::W; i += kThreads) stage[i] = 0.0f;  // rows from dim on stay zero
+  bw::pdl_wait();
+  if (!few) bw::pdl_launch();
+  __syncthreads();
+  const int kh = h / a.rep;
+  auto request = [&](int first, float* buf) {
+    const int len = min(chunk, cnt - first);
+    if (a.wide) {
+      constexpr int Ws = T::SC / 4;
+      for (int i = tid; i < len * Ws; i += kThreads) {
+        const int tt = i / Ws, e = (i - tt * Ws) * 4;
+        const size_t r = static_cast<size_t>(row0 + first + tt);
+        const float* src;
+        if (e < T::VECS * T::DP) {
+          const int d = e % T::DP;
+          if (d >= dim) continue;
+          if (e < T::DP) src = a.k + r * a.k_stride + kh * dim + d;
+          else if (e < 2 * T::DP) src = a.q + r * a.q_stride + kh * dim + d;
+          else src = a.decay + r * a.decay_stride + h * dim + d;
+        } else {
+          const int cc = c0 + e - T::VECS * T::DP;
+          if (cc >= vdim) continue;
+          src = a.v + r * a.v_stride + h * vdim + cc;
+        }
+        copy16_async(buf + tt * T::W + e, src);
+      }
+    } else {
+      constexpr int Ws = T::SC;
+      for (int i = tid; i < len * Ws; i += kThreads) {
+        const int tt = i / Ws, e = i - tt * Ws;
+        const size_t r = static_cast<size_t>(row0 + first + tt);
+        const float* src;
+        if (e < T::VECS * T::DP) {
+          const int d = e % T::DP;
+          if (d >= dim) continue;
+          if (e < T::DP) src = a.k + r * a.k_stride + kh * dim + d;
+          else if (e < 2 * T::DP) src = a.q + r * a.q_stride + kh * dim + d;
+          else src = a.decay + r * a.decay_stride + h * dim + d;
+        } else {
+          const int cc = c0 + e - T::VECS * T::DP;
+          if (cc >= vdim) continue;
+          src = a.v + r * a.v_stride + h * vdim + cc;
+        }
+        copy4_async(buf + tt * T::W + e, src);
+      }
+    }
+    if (MODE != kBonus) {
+      for (int tt = tid; tt < len; tt += kThreads) {
+        const size_t r = static_cast<size_t>(row0 + first + tt);
+        copy4_async(buf + tt * T::W + T::SC, a.s0 + r * a.s_stride + h);
+        if (kMem) copy4_async(buf + tt * T::W + T::SC + 1, a.s1 + r * a.s_stride + h);
+      }
+    }
+    bw::copies_commit();
+  };
+  // One token: S moves on; returns this lane's share of the output.
+  auto token = [&](const float* tok) -> float {
+    const Rows<V> k = load_rows<LP, V>(tok, p), q = load_rows<LP, V>(tok + T::DP, p);
+    const float* vals = tok + T::VECS * T::DP;
+    float v = vals[tid / LP];
+    if (MODE == kDelta) {
+      const Rows<V> g = load_rows<LP, V>(tok + 2 * T::DP, p);
+      const float beta = tok[T::SC];
+#pragma unroll
+      for (int i = 0; i < 4 * V; ++i) S.v[i] = __fmul_rn(g.v[i], S.v[i]);
+      const float u = __fmul_rn(beta, __fsub_rn(v, column_sum<LP>(dot<V>(k, S))));
+#pragma unroll
+      for (int i = 0; i < 4 * V; ++i) S.v[i] = __fmaf_rn(k.v[i], u, S.v[i]);
+      return dot<V>(q, S);
+    } else if (MODE == kBonus) {
+      const Rows<V> w = load_rows<LP, V>(tok + 2 * T::DP, p);
+      Rows<V> seen;
+#pragma unroll
+      for (int i = 0; i < 4 * V; ++i) {
+        const float kv = __fmul_rn(k.v[i], v);
+        seen.v[i] = __fmaf_rn(bonus.v[i], kv, S.v[i]);
+        S.v[i] = __fmaf_rn(w.v[i], S.v[i], kv);
+      }
+      return dot<V>(q, seen);
+    } else {
+      if (c == vdim) v = 1.0f;  // the normaliser's column
+      const float keep = tok[T::SC], add = __fmul_rn(tok[T::SC + 1], v);
+#pragma unroll
+      for (int i = 0; i < 4 * V; ++i) S.v[i] = __fmaf_rn(k.v[i], add, __fmul_rn(keep, S.v[i]));
+      return dot<V>(q, S);
+    }
+  };
+  request(0, stage);
+  for (int first = 0, b = 0; first < cnt; first += chunk, b ^= 1) {
+    const int len = min(chunk, cnt - first);
+    float* buf = stage + b * chunk * T::W;
+    if (first) __syncthreads();  // the other buffer and `outs` have been used
+    if (first + chunk < cnt) {
+      request(first + chunk, stage + (b ^ 1) * chunk * T::W);
+      bw::copies_wait<1>();
+    } else {
+      bw::copies_wait<0>();
+    }
+    __syncthreads();
+    if (MODE == kBonus) {
+      for (int i = tid; i < len * T::DP; i += kThreads) {
+        const int tt = i / T::DP, d = i % T::DP;
+        if (d >= dim) continue;
+        float* at = buf + tt * T::W + 2 * T::DP + d;
+        *at = exp_f(-exp_f(__fadd_rn(*at, a.decay_bias[h * dim + d])));
+      }
+      __syncthreads();
+    }
+    if (kMem) {
+      if (tid < 32) {
+        // lane l forms the gates of tokens l, l + 32, ..; the maxima follow one after the other
+        const float bf = a.s0_bias[h], bi = a.s1_bias[h];
+        for (int t0 = 0; t0 < len; t0 += 32) {
+          float f = 0.0f, g = 0.0f;
+          float* sc = buf + (t0 + tid) * T::W + T::SC;
+          if (t0 + tid < len) {
+            // ln(sigmoid(y)) = -softplus(-y)
+            f = -softplus_f(-__fmul_rn(a.cap, tanhf(__fdiv_rn(__fadd_rn(sc[0], bf), a.cap))));
+            g = __fmul_rn(a.cap, tanhf(__fdiv_rn(__fadd_rn(sc[1], bi), a.cap)));
+          }
+          float mine = 0.0f, before = 0.0f;
+          const int end = min(32, len - t0);
+          for (int l = 0; l < end; ++l) {
+            const float fm = __fadd_rn(__shfl_sync(0xffffffffu, f, l), m);
+            m = fmaxf(fm, __shfl_sync(0xffffffffu, g, l));
+            if (tid == l) mine = m, before = fm;
+          }
+          if (t0 + tid < len) {
+            sc[0] = exp_f(__fsub_rn(before, mine));
+            sc[1] = exp_f(__fsub_rn(g, mine));
+            sc[2] = mine;
+          }
+        }
+      }
+      __syncthreads();
+    }
+    int tt = 0;
+    for (; tt + T::G <= len; tt += T::G) {
+      float part[T::G];
+#pragma unroll
+      for (int j = 0; j < T::G; ++j) part[j] = token(buf + (tt + j) * T::W);
+      const float s = group_sum<LP, T::G>(part, p);
+      if (p % (LP / T::G) == 0) outs[(tt + p / (LP / T::G)) * T::CB + tid / LP] = s;
+    }
+    for (; tt < len; ++tt) {
+      const float s = column_sum<LP>(token(buf + tt * T::W));
+      if (p == 0) outs[tt * T::CB + tid / LP] = s;
+    }
+    __syncthreads();
+    for (int i = tid; i < len * T::CB; i += kThreads) {
+      const int ti = i / T::CB, cc = c0 + i % T::CB;
+      const size_t r = static_cast<size_t>(row0 + first + ti);
+      if (cc < vdim) {
+        a.o[r * a.heads * vdim + h * vdim + cc] = outs[i];
+      } else if (kMem && cc == vdim) {
+        float* x = a.aux + (r * a.heads + h) * 2;
+        x[0] = outs[i], x[1] = buf[ti * T::W + T::SC + 2];
+      }
+    }
+  }
+  if (!col_ok) return;
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const int row = 4 * (p + LP * i);
+    if (a.wide) {
+      if (row < dim) *reinterpret_cast<float4*>(sp + row) = make_float4(S.v[4 * i], S.v[4 * i + 1], S.v[4 * i + 2], S.v[4 * i + 3]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (row + e < dim) sp[row + e] = S.v[4 * i + e];
+    }
+  }
+  // every column keeps the maximum of its own: the blocks of a head do not read what another one writes
+  if (kMem && p == 0) {
+    const int last = (cnt - 1) / chunk, slot = (cnt - 1) - last * chunk;
+    sp[dim] = stage[(last & 1) * chunk * T::W + slot * T::W + T::SC + 2];
+  }
+}
+
+// out[r, h] = y / sqrt(mean(y^2) + eps) * w * gate(g) for every head, y the recurrence's output; with `aux` y is first
+// divided: y <- s y / (max(|s n.q|, e^-m) + 1e-6), s the queries' scale. A warp per row and head.
+struct FinishArgs {
+  const float* o;
+  const float* aux;    // [n, heads, 2] or null
+  float q_scale;
+  const float* w;      // [vdim] (w_stride 0) or [heads * vdim] (w_stride vdim)
+  int w_stride;
+  const float* gate;   // row r, head h: gate + r * gate_stride + h * vdim
+  int gate_stride;
+  int gate_silu;       // 0: sigmoid(g); 1: g sigmoid(g)
+  float eps;
+  act_t* out;
+  int heads, vdim;
+};
+
+__global__ void __launch_bounds__(kThreads) scan_finish_kernel(const FinishArgs a) {
+  bw::pdl_enter();
+  const size_t r = blockIdx.x;
+  const int h = blockIdx.y * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= a.heads) return;
+  const float* o = a.o + (r * a.heads + h) * a.vdim;
+  const float* g = a.gate + r * a.gate_stride + h * a.vdim;
+  const float* w = a.w + static_cast<size_t>(h) * a.w_stride;
+  act_t* out = a.out + (r * a.heads + h) * a.vdim;
+  float f = 1.0f;
+  if (a.aux) {
+    const float nq = a.aux[(r * a.heads + h) * 2], m = a.aux[(r * a.heads + h) * 2 + 1];
+    const float den = __fadd_rn(fmaxf(fabsf(__fmul_rn(nq, a.q_scale)), expf(-m)), 1e-6f);
+    f = __fdiv_rn(a.q_scale, den);
+  }
+  constexpr int kKeep = 8;  // entries of a lane that stay in registers (vdim up to 256)
+  float y[kKeep];
+  float ss = 0.0f;
+#pragma unroll
+  for (int j = 0; j < kKeep; ++j) {
+    const int d = lane + 32 * j;
+    y[j] = d < a.vdim ? __fmul_rn(o[d], f) : 0.0f;
+    ss = __fmaf_rn(y[j], y[j], ss);
+  }
+  for (int d = lane + 32 * kKeep; d < a.vdim; d += 32) {
+    const float v = __fmul_rn(o[d], f);
+    ss = __fmaf_rn(v, v, ss);
+  }
+  const float inv = bw::rms_scale(bw::warp_sum(ss), a.vdim, a.eps);
+  auto finish = [&](int d, float v) {
+    const float z = g[d];
+    const float s = sigmoid_f(z);
+    out[d] = bw::from_f<act_t>(__fmul_rn(bw::rms_apply(v, inv, w[d]), a.gate_silu ? __fmul_rn(z, s) : s));
+  };
+#pragma unroll
+  for (int j = 0; j < kKeep; ++j) {
+    const int d = lane + 32 * j;
+    if (d < a.vdim) finish(d, y[j]);
+  }
+  for (int d = lane + 32 * kKeep; d < a.vdim; d += 32) finish(d, __fmul_rn(o[d], f));
+}
+
+// ---------------------------------------------------------------------------------------
+// What the delta recurrence reads: per row, a warp per head. q, k and v pass a causal convolution over time on
+// every channel (inputs before the step's first row of a sequence from the request's state, zeros before position 0)
+// and SiLU; q and k become unit vectors, q times a scale; the decays g = exp(-exp(A_h) softplus(z + bias)) replace z;
+// beta = sigmoid(b). With `keep` (steps of one row per sequence) the state is brought up to date here as well.
+struct DeltaPrepArgs {
+  const float* u;         // [n, u_stride]: q heads | k heads | v heads, beta's projections from beta_col on
+  int u_stride, beta_col;
+  const float* conv_t;    // [taps, channels]
+  int taps;
+  float* conv_state;      // [slots, taps - 1, channels] or null
+  int keep;
+  float* z;               // [n, z_stride]: heads * dim columns
+  int z_stride;
+  const float* dt_bias;   // [heads * dim]
+  const float* a_log;     // [heads]
+  float* out;             // [n, out_stride]: q | k | v | beta
+  int out_stride;
+  const int* pos;
+  const int* row_seq;
+  const int* seq_row0;
+  const int* seq_slot;
+  int heads, kv_heads, dim, vdim;
+  float q_scale;
+};
+
+constexpr int kMaxPer = 16;  // entries of a head per lane: sizes up to 512
+
+__global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const DeltaPrepArgs a) {
+  bw::pdl_enter();
+  const int r = blockIdx.x;
+  const int lane = threadIdx.x & 31;
+  const int unit = blockIdx.y * (kThreads / 32) + (threadIdx.x >> 5);
+  const int qk = 2 * a.kv_heads, convs = qk + a.heads;
+  float* out = a.out + static_cast<size_t>(r) * a.out_stride;
+  const int channels = qk * a.dim + a.heads * a.vdim;
+  if (unit < convs) {
+    const int size = unit < qk ? a.dim : a.vdim;
+    const int col0 = unit < qk ? unit * a.dim : qk * a.dim + (unit - qk) * a.vdim;
+    const int p = a.pos[r], seq = a.row_seq[r], row0 = a.seq_row0[seq];
+    float* st = a.conv_state ? a.conv_state + static_cast<size_t>(a.seq_slot[seq]) * (a.taps - 1) * channels : nullptr;
+    const float* u = a.u + static_cast<size_t>(r) * a.u_stride;
+    float val[kMaxPer];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kMaxPer; ++j) {
+      const int e = lane + 32 * j;
+      float y = 0.0f;
+      if (e < size) {
+        const int c = col0 + e;
+        for (int t = 0; t < a.taps; ++t) {  // taps ascending
+          const int back = a.taps - 1 - t;
+          if (p - back < 0) continue;
+          const float x = r - back >= row0 ? u[c - static_cast<ptrdiff_t>(back) * a.u_stride]
+                                           : st[static_cast<size_t>(a.taps - 1 - (row0 - (r - back))) * channels + c];
+          y = __fmaf_rn(a.conv_t[static_cast<size_t>(t) * channels + c], x, y);
+        }
+        if (a.keep && st) {  // the sequence's only row: the inputs move up by one
+          for (int t = 0; t + 1 < a.taps - 1; ++t)
+            st[static_cast<size_t>(t) * channels + c] = p - (a.taps - 2 - t) >= 0 ? st[static_cast<size_t>(t + 1) * channels + c] : 0.0f;
+          st[static_cast<size_t>(a.taps - 2) * channels + c] = u[c];
+        }
+        y = __fmul_rn(y, sigmoid_f(y));
+        ss = __fmaf_rn(y, y, ss);
+      }
+      val[j] = y;
+    }
+    float f = 1.0f;
+    if (unit < qk) {
+      f = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(bw::warp_sum(ss), 1e-6f)));
+      if (unit < a.kv_heads) f = __fmul_rn(f, a.q_scale);
+    }
+#pragma unroll
+    for (int j = 0; j < kMaxPer; ++j) {
+      const int e = lane + 32 * j;
+      if (e < size) out[col0 + e] = __fmul_rn(val[j], f);
+    }
+  } else if (unit < convs + a.heads) {
+    const int h = unit - convs;
+    const float rate = expf(a.a_log[h]);
+    float* z = a.z + static_cast<size_t>(r) * a.z_stride + h * a.dim;
+    for (int d = lane; d < a.dim; d += 32) z[d] = expf(-__fmul_rn(rate, softplus_f(__fadd_rn(z[d], a.dt_bias[h * a.dim + d]))));
+  } else if (unit == convs + a.heads) {
+    for (int h = lane; h < a.heads; h += 32) out[channels + h] = sigmoid_f(a.u[static_cast<size_t>(r) * a.u_stride + a.beta_col + h]);
+  }
+}
+
+// Token shift: mix_s = x + (x' - x) mu_s for `mixes` vectors mu, x' the row before of the same sequence (from the
+// state for the step's first row, zero for a sequence's first token). out: [mixes, n, width], as the products read them.
+// With `keep` (steps of one row per sequence) the state becomes the row.
+__global__ void __launch_bounds__(256)
+shift_mix_kernel(const float* __restrict__ x, const float* __restrict__ mu, int mixes, float* last, int keep, act_t* out, int n,
+                 int width, const int* __restrict__ pos, const int* __restrict__ row_seq, const int* __restrict__ seq_row0,
+                 const int* __restrict__ seq_slot) {
+  bw::pdl_enter();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= width) return;
+  const int r = blockIdx.x;
+  const int seq = row_seq[r];
+  float* st = last + static_cast<size_t>(seq_slot[seq]) * width + c;
+  const float v = x[static_cast<size_t>(r) * width + c];
+  float before = 0.0f;
+  if (r > seq_row0[seq]) before = x[static_cast<size_t>(r - 1) * width + c];
+  else if (pos[r] > 0) before = *st;
+  if (keep) *st = v;
+  const float d = __fsub_rn(before, v);
+  for (int s = 0; s < mixes; ++s)
+    out[(static_cast<size_t>(s) * n + r) * width + c] = bw::from_f<act_t>(__fmaf_rn(d, mu[static_cast<size_t>(s) * width + c], v));
+}
+
+// Two sublayers side by side and the block's norm behind them, one block per row:
+//   y = (a / rms(a) * wa + b / rms(b) * wb) / 2
+// and either y into `y`, or x += layernorm(y) * w with the summed row rounded into `xn`.
+__global__ void __launch_bounds__(256)
+pair_mean_kernel(const float* __restrict__ a, const float* __restrict__ wa, const float* __restrict__ b,
+                 const float* __restrict__ wb, float eps, float* y, int width, const float* __restrict__ w, float norm_eps,
+                 float* x, act_t* xn) {
+  bw::pdl_enter();
+  extern __shared__ float row[];
+  __shared__ float red[32];
+  const size_t base = static_cast<size_t>(blockIdx.x) * width;
+  float sa = 0.0f, sb = 0.0f;
+  for (int i = threadIdx.x; i < width; i += 256) {
+    const float va = a[base + i], vb = b[base + i];
+    sa = __fmaf_rn(va, va, sa), sb = __fmaf_rn(vb, vb, sb);
+  }
+  const float ia = bw::rms_scale(bw::block_sum(sa, red), width, eps), ib = bw::rms_scale(bw::block_sum(sb, red), width, eps);
+  float s = 0.0f;
+  for (int i = threadIdx.x; i < width; i += 256) {
+    const float v = __fmul_rn(0.5f, __fadd_rn(bw::rms_apply(a[base + i], ia, wa[i]), bw::rms_apply(b[base + i], ib, wb[i])));
+    if (x) {
+      row[i] = v;
+      s = __fadd_rn(s, v);
+    } else {
+      y[base + i] = v;
+    }
+  }
+  if (!x) return;
+  const float fw = static_cast<float>(width);
+  const float mean = __fdiv_rn(bw::block_sum(s, red), fw);
+  float q = 0.0f;
+  for (int i = threadIdx.x; i < width; i += 256) {
+    const float d = __fsub_rn(row[i], mean);
+    q = __fmaf_rn(d, d, q);
+  }
+  const float inv = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(bw::block_sum(q, red), fw), norm_eps)));
+  for (int i = threadIdx.x; i < width; i += 256) {
+    const float v = __fadd_rn(x[base + i], __fmul_rn(__fmul_rn(__fsub_rn(row[i], mean), inv), w[i]));
+    x[base + i] = v;
+    if (xn) xn[base + i] = bw::from_f<act_t>(v);
+  }
+}
+
+template <int MODE, int LP, int V>
+int launch_scan(ScanArgs a, int tiles, int longest, cudaStream_t stream) {
+  typedef Shape<MODE, LP, V> T;
+  // Tokens staged at a time: no more than the longest sequence of the step can have (a step of single rows stages
+  // one, so that many of its small blocks share an SM), at most 16, and no more than 100 KB.
+  a.chunk = 1;
+  while (a.chunk < 16 && a.chunk < longest) a.chunk *= 2;
+  auto bytes = [](int chunk) { return static_cast<size_t>(2 * chunk * T::W + chunk * T::CB) * sizeof(float); };
+  while (a.chunk > 1 && bytes(a.chunk) > 100 * 1024) a.chunk /= 2;
+  const size_t smem = bytes(a.chunk);
+  static size_t allowed = 48 * 1024;
+  if (smem > allowed) {
+    cudaError_t e = cudaFuncSetAttribute(state_scan_kernel<MODE, LP, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) {
+      bw::set_error("state_scan: %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+      return static_cast<int>(e);
+    }
+    allowed = smem;
+  }
+  const int cols = MODE == kMemory ? a.vdim + 1 : a.vdim;
+  bw::launch_pdl(state_scan_kernel<MODE, LP, V>, dim3(tiles, a.heads, (cols + T::CB - 1) / T::CB), dim3(kThreads), smem, stream, a);
+  return bw::launch_status();
+}
+
+template <int MODE>
+int launch_mode(const ScanArgs& a, int tiles, int longest, cudaStream_t stream) {
+  if (a.dim <= 16) return launch_scan<MODE, 4, 1>(a, tiles, longest, stream);
+  if (a.dim <= 32) return launch_scan<MODE, 4, 2>(a, tiles, longest, stream);
+  if (a.dim <= 64) return launch_scan<MODE, 8, 2>(a, tiles, longest, stream);
+  if (a.dim <= 128) return launch_scan<MODE, 16, 2>(a, tiles, longest, stream);
+  if (a.dim <= 256) return launch_scan<MODE, 32, 2>(a, tiles, longest, stream);
+  if (a.dim <= 512) return launch_scan<MODE, 32, 4>(a, tiles, longest, stream);
+  bw::set_error("state_scan: key size %d (up to 512)", a.dim);
+  return -1;
+}
+
+bool on16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace
+
+// mode 0: the delta rule (decay = g, s0 = beta); 1: the bonus form (decay = z with decay_bias, bonus = u); 2: the matrix memory
+// (s0, s1 = the projections of the forget and the input gate with their biases, cap; aux [n, heads, 2]). q and k
+// rows hold heads / rep heads. o: [n, heads * vdim]. tiles: one per sequence (sequence, first row, rows).
+BW_API int BW_FN(state_scan)(int mode, const float* q, int q_stride, const float* k, int k_stride, const float* v,
+                             int v_stride, int rep, const float* decay, int decay_stride, const float* decay_bias,
+                             const float* bonus, const float* s0, const float* s1, int s_stride, const float* s0_bias,
+                             const float* s1_bias, float cap, float* state, float* o, float* aux, const int* tile_seq,
+                             const int* tile_row0, const int* tile_rows, int tiles, const int* seq_pos0, const int* seq_slot,
+                             int n, int heads, int dim, int vdim, cudaStream_t stream) {
+  if (tiles <= 0 || n <= 0) return 0;
+  if (heads <= 0 || dim <= 0 || vdim <= 0 || rep <= 0 || heads % rep) {
+    bw::set_error("state_scan: %d heads, %d to a query head, sizes %d / %d", heads, rep, dim, vdim);
+    return -1;
+  }
+  ScanArgs a;
+  a.q = q, a.k = k, a.v = v, a.q_stride = q_stride, a.k_stride = k_stride, a.v_stride = v_stride, a.rep = rep;
+  a.decay = decay, a.decay_stride = decay_stride, a.decay_bias = decay_bias, a.bonus = bonus;
+  a.s0 = s0, a.s1 = s1, a.s_stride = s_stride, a.s0_bias = s0_bias, a.s1_bias = s1_bias, a.cap = cap;
+  a.state = state, a.o = o, a.aux = aux, a.tile_seq = tile_seq, a.tile_row0 = tile_row0, a.tile_rows = tile_rows;
+  a.seq_pos0 = seq_pos0, a.seq_slot = seq_slot, a.heads = heads, a.dim = dim, a.vdim = vdim, a.chunk = 1;
+  // 16 bytes at a time where every row and head starts on 16 bytes
+  a.wide = dim % 4 == 0 && vdim % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && v_stride % 4 == 0 &&
+           (mode == kMemory || decay_stride % 4 == 0) && on16(q) && on16(k) && on16(v) && on16(decay) && on16(state);
+  const int longest = n - tiles + 1;
+  switch (mode) {
+    case kDelta: return launch_mode<kDelta>(a, tiles, longest, stream);
+    case kBonus: return launch_mode<kBonus>(a, tiles, longest, stream);
+    case kMemory: return launch_mode<kMemory>(a, tiles, longest, stream);
+  }
+  bw::set_error("state_scan: unknown mode %d", mode);
+  return -1;
+}
+
+// gate_kind 0: sigmoid(g); 1: g sigmoid(g). w_per_head: w holds heads * vdim numbers (else vdim). aux may be null.
+BW_API int BW_FN(scan_finish)(const float* o, const float* aux, float q_scale, const float* w, int w_per_head,
+                              const float* gate, int gate_stride, int gate_kind, float eps, void* out, int n, int heads,
+                              int vdim, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  FinishArgs a;
+  a.o = o, a.aux = aux, a.q_scale = q_scale, a.w = w, a.w_stride = w_per_head ? vdim : 0, a.gate = gate;
+  a.gate_stride = gate_stride, a.gate_silu = gate_kind, a.eps = eps, a.out = static_cast<act_t*>(out), a.heads = heads, a.vdim = vdim;
+  bw::launch_pdl(scan_finish_kernel, dim3(n, (heads + kThreads / 32 - 1) / (kThreads / 32)), dim3(kThreads), 0, stream, a);
+  return bw::launch_status();
+}
+
+BW_API int BW_FN(delta_prepare)(const float* u, int u_stride, int beta_col, const float* conv_t, int taps, float* conv_state,
+                                int keep, float* z, int z_stride, const float* dt_bias, const float* a_log, float* out,
+                                int out_stride, const int* pos, const int* row_seq, const int* seq_row0, const int* seq_slot,
+                                int n, int heads, int kv_heads, int dim, int vdim, float q_scale, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (dim > 32 * kMaxPer || vdim > 32 * kMaxPer) {
+    bw::set_error("delta_prepare: head sizes %d / %d (up to %d)", dim, vdim, 32 * kMaxPer);
+    return -1;
+  }
+  if (taps > 1 && !conv_state) {
+    bw::set_error("delta_prepare: a convolution of %d taps needs the requests' state", taps);
+    return -1;
+  }
+  DeltaPrepArgs a;
+  a.u = u, a.u_stride = u_stride, a.beta_col = beta_col, a.conv_t = conv_t, a.taps = taps;
+  a.conv_state = taps > 1 ? conv_state : nullptr, a.keep = keep, a.z = z, a.z_stride = z_stride, a.dt_bias = dt_bias, a.a_log = a_log;
+  a.out = out, a.out_stride = out_stride, a.pos = pos, a.row_seq = row_seq, a.seq_row0 = seq_row0, a.seq_slot = seq_slot;
+  a.heads = heads, a.kv_heads = kv_heads, a.dim = dim, a.vdim = vdim, a.q_scale = q_scale;
+  const int units = 2 * kv_heads + 2 * heads + 1;
+  bw::launch_pdl(delta_prepare_kernel, dim3(n, (units + kThreads / 32 - 1) / (kThreads / 32)), dim3(kThreads), 0, stream, a);
+  return bw::launch_status();
+}
+
+BW_API int BW_FN(shift_mix)(const float* x, const float* mu, int mixes, float* last, int keep, void* out, int n, int width,
+                            const int* pos, const int* row_seq, const int* seq_row0, const int* seq_slot, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  bw::launch_pdl(shift_mix_kernel, dim3(n, (width + 255) / 256), dim3(256), 0, stream, x, mu, mixes, last, keep,
+                 static_cast<act_t*>(out), n, width, pos, row_seq, seq_row0, seq_slot);
+  return bw::launch_status();
+}
+
+// x null: y = the mean of the two normed rows. Otherwise x += layernorm(that) * w, and the summed row into xn (if given).
+BW_API int BW_FN(pair_mean)(const float* a, const float* wa, const float* b, const float* wb, float eps, float* y, int n,
+                            int width, const float* w, float norm_eps, float* x, void* xn, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (width <= 0 || width > 48 * 1024 / 4) {
+    bw::set_error("pair_mean: width %d (1 .. 12288)", width);
+    return -1;
+  }
+  bw::launch_pdl(pair_mean_kernel, dim3(n), dim3(256), x ? static_cast<size_t>(width) * sizeof(float) : 0, stream, a, wa, b, wb,
+                 eps, y, width, w, norm_eps, x, static_cast<act_t*>(xn));
+  return bw::launch_status();
+}

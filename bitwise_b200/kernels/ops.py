@@ -59,6 +59,7 @@ class KernelOps:
     """Operations of one precision.  ``act_dtype`` is the dtype of activations between
     kernels (the residual stream, logits and norm weights are float32 in both)."""
 
+    OUT_ACTIVATIONS = (None, "relu2", "tanh")  # what a product's outputs can pass before they are stored, by index
     FUSED_ACTIVATIONS = ("silu", "gelu_tanh")  # what the gate/up product can apply in its epilogue, by index
 
     def __init__(self, dtype: str, verbose_build: bool = True):
@@ -185,9 +186,16 @@ class KernelOps:
                    _c_float(eps), self._stream())
 
     def linear(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
-               residual: Optional[torch.Tensor] = None, legacy: bool = False) -> None:
+               residual: Optional[torch.Tensor] = None, legacy: bool = False, activation: Optional[str] = None) -> None:
         """out = x @ w.T (+ residual).  x [M,K] and w [N,K] in act_dtype; out act_dtype or
-        float32; with a float32 residual the sum is formed in 32-bit (out float32, may alias)."""
+        float32; with a float32 residual the sum is formed in 32-bit (out float32, may alias).
+        ``activation`` (of OUT_ACTIVATIONS; out act_dtype, no residual): out = act(x @ w.T), applied to the
+        32-bit sums in the product's epilogue on the serving precision."""
+        act = 0
+        if activation is not None:
+            if activation not in self.OUT_ACTIVATIONS or residual is not None or out.dtype != self.act_dtype:
+                raise KernelError(f"linear: activation {activation!r} wants an output of the activation type and no residual")
+            act = self.OUT_ACTIVATIONS.index(activation)
         m, k = x.shape
         n = w.shape[0]
         _need(x, self.act_dtype, "linear x", 2)
@@ -203,6 +211,8 @@ class KernelOps:
             _need(out, torch.float32, "linear out", 2)
             self._call("bw_f32_linear", _p(x), _p(w), _p(out), _p(residual), _c_int(m), _c_int(n), _c_int(k),
                        self._stream())
+            if act:
+                self.activate_rows(out, out, activation)
         else:
             if out.dtype not in (torch.float32, torch.bfloat16):
                 raise KernelError("linear: out must be float32 or bfloat16")
@@ -210,7 +220,7 @@ class KernelOps:
             partials = counters = None
             if m <= self._split_rows:
                 partials, counters = self._linear_scratch(x.device, n, k)
-            self._call("bw_bf16_linear", _p(x), _p(w), _p(out), _c_int(int(out.dtype == torch.float32)),
+            self._call("bw_bf16_linear", _p(x), _p(w), _p(out), _c_int(2 * act + int(out.dtype == torch.float32)),
                        _p(residual), _c_int(m), _c_int(n), _c_int(k), _p(partials), _p(counters),
                        _c_int(int(legacy)), self._stream(),
                        launches=1 if legacy else self._linear_kernels(m, n, k, False, partials is not None))
@@ -650,19 +660,21 @@ class KernelOps:
                            next_out: Optional[torch.Tensor] = None) -> None:
         """x[r] += (d[r] - mean) / sqrt(var + eps) * weight with the row statistics of d; d, weight and x
         float32.  With ``next_weight`` and ``next_out`` (act_dtype) also the layer norm of the summed row, with
-        that weight and ``next_eps``: the norm before the next sublayer, in the same kernel."""
+        that weight and ``next_eps``: the norm before the next sublayer, in the same kernel.  ``next_out`` alone
+        receives the summed row itself, rounded: a sublayer that reads the stream without a norm."""
         n, width = x.shape
         _need(d, torch.float32, "layernorm_residual d", 2)
         _need(x, torch.float32, "layernorm_residual x", 2)
         _need(weight, torch.float32, "layernorm_residual weight", 1)
         if tuple(d.shape) != (n, width) or weight.shape[0] != width:
             raise KernelError("layernorm_residual: shapes differ")
-        if (next_weight is None) != (next_out is None):
-            raise KernelError("layernorm_residual: the next norm needs a weight and an output")
+        if next_weight is not None and next_out is None:
+            raise KernelError("layernorm_residual: the next norm needs an output")
         if next_out is not None:
-            _need(next_weight, torch.float32, "layernorm_residual next_weight", 1)
             _need(next_out, self.act_dtype, "layernorm_residual next_out", 2)
-            if tuple(next_out.shape) != (n, width) or next_weight.shape[0] != width:
+            if next_weight is not None:
+                _need(next_weight, torch.float32, "layernorm_residual next_weight", 1)
+            if tuple(next_out.shape) != (n, width) or (next_weight is not None and next_weight.shape[0] != width):
                 raise KernelError("layernorm_residual: the next norm's shapes differ")
         self._pcall("layernorm_residual", _p(d), _p(weight), _p(x), _c_int(n), _c_int(width), _c_float(eps),
                     _p(next_weight), _c_float(next_eps), _p(next_out), self._stream())
@@ -1002,6 +1014,16 @@ class KernelOps:
             raise KernelError("glu_gelu: input is not [rows, 2 * inner]")
         self._gcall("glu_gelu", _p(gate_up), _p(out), _c_int(n), _c_int(inter), self._stream())
 
+    def activate_rows(self, x: torch.Tensor, out: torch.Tensor, activation: Optional[str] = None) -> None:
+        """out = act(x) for float32 rows x (which may be columns of wider rows), out in act_dtype (in float32 it may be
+        x); without an activation the rows are only rounded."""
+        _need_rows(x, torch.float32, "activate_rows x")
+        _need(out, self.act_dtype, "activate_rows out", 2)
+        if activation not in self.OUT_ACTIVATIONS or x.shape != out.shape:
+            raise KernelError(f"activate_rows: activation {activation!r}, shapes {tuple(x.shape)} and {tuple(out.shape)}")
+        self._gcall("activate_rows", _p(x), _c_int(x.shape[0]), _c_int(x.shape[1]), _c_int(x.stride(0)), _p(out),
+                    _c_int(self.OUT_ACTIVATIONS.index(activation)), self._stream())
+
     def softcap_rows(self, z: torch.Tensor, cap: float) -> None:
         """z <- cap * tanh(z / cap) in place on float32 rows."""
         _need(z, torch.float32, "softcap_rows z")
@@ -1041,19 +1063,21 @@ class KernelOps:
                          next_out: Optional[torch.Tensor] = None) -> None:
         """x[r] += d[r] / sqrt(mean(d[r]^2) + eps) * weight; d, weight and x float32.  With ``next_weight``
         and ``next_out`` (act_dtype) also next_out[r] = x[r] / sqrt(mean(x[r]^2) + next_eps) * next_weight of
-        the summed row: the norm before the next sublayer, in the same kernel."""
+        the summed row: the norm before the next sublayer, in the same kernel.  ``next_out`` alone receives the
+        summed row itself, rounded: a sublayer that reads the stream without a norm."""
         n, width = x.shape
         _need(d, torch.float32, "rmsnorm_residual d", 2)
         _need(x, torch.float32, "rmsnorm_residual x", 2)
         _need(weight, torch.float32, "rmsnorm_residual weight", 1)
         if tuple(d.shape) != (n, width) or weight.shape[0] != width:
             raise KernelError("rmsnorm_residual: shapes differ")
-        if (next_weight is None) != (next_out is None):
-            raise KernelError("rmsnorm_residual: the next norm needs a weight and an output")
+        if next_weight is not None and next_out is None:
+            raise KernelError("rmsnorm_residual: the next norm needs an output")
         if next_out is not None:
-            _need(next_weight, torch.float32, "rmsnorm_residual next_weight", 1)
             _need(next_out, self.act_dtype, "rmsnorm_residual next_out", 2)
-            if tuple(next_out.shape) != (n, width) or next_weight.shape[0] != width:
+            if next_weight is not None:
+                _need(next_weight, torch.float32, "rmsnorm_residual next_weight", 1)
+            if tuple(next_out.shape) != (n, width) or (next_weight is not None and next_weight.shape[0] != width):
                 raise KernelError("rmsnorm_residual: the next norm's shapes differ")
         self._mcall("rmsnorm_residual", _p(d), _p(weight), _p(x), _c_int(n), _c_int(width), _c_float(eps), _p(next_weight),
                     _c_float(next_eps), _p(next_out), self._stream())
@@ -1086,7 +1110,8 @@ class KernelOps:
                     kcache: torch.Tensor, vcache: Optional[torch.Tensor], q_out: torch.Tensor, heads: int,
                     write_kv_heads: int, dim: int, vdim: int, conv_wt: Optional[torch.Tensor] = None,
                     bias: Optional[torch.Tensor] = None, vmix_src: Optional[torch.Tensor] = None,
-                    vmix_lambda: Optional[torch.Tensor] = None, v_keep: Optional[torch.Tensor] = None) -> None:
+                    vmix_lambda: Optional[torch.Tensor] = None, v_keep: Optional[torch.Tensor] = None,
+                    half_layout: bool = False) -> None:
         """From the projected rows ``u`` (float32 [n, cols]: ``heads`` query heads of ``dim``, then, when
         ``write_kv_heads`` > 0, that many key heads of ``dim`` and, with ``vcache``, value heads of
         ``vdim``): the convolution over time with ``conv_w`` [cols, taps] (inputs before the step's
@@ -1097,7 +1122,8 @@ class KernelOps:
         transposed ([taps, cols]); with them, and sizes that are multiples of 4, the kernel reads four
         channels at a time.  ``bias`` [cols] is added to every projected row first.  ``vmix_src`` (float32 [n,
         kv_heads * vdim]) and ``vmix_lambda`` (one float32): the values become (1 - lambda) v + lambda vmix_src
-        before they are stored; ``v_keep`` (same shape) receives the values as stored, in float32."""
+        before they are stored; ``v_keep`` (same shape) receives the values as stored, in float32.  ``half_layout``:
+        the rotation's pair i is made of entries i and i + pairs of a head instead of 2i and 2i + 1."""
         n, cols = u.shape
         _need_rows(u, torch.float32, "qkv_prepare u")
         _need(q_out, self.act_dtype, "qkv_prepare q_out", 2)
@@ -1150,7 +1176,7 @@ class KernelOps:
                     _p(batch.seq_pos0), _p(batch.seq_slot), _p(block_table), _c_int(block_table.shape[1]), _p(kcache),
                     _p(vcache if write_kv_heads else None), _p(q_out), _c_int(n), _c_int(heads), _c_int(write_kv_heads),
                     _c_int(dim), _c_int(vdim), _c_int(kcache.shape[2]), _p(bias), _p(vmix_src), _p(vmix_lambda), _p(v_keep),
-                    _c_int(u.stride(0)), self._stream())
+                    _c_int(u.stride(0)), _c_int(int(half_layout)), self._stream())
 
     def conv_state_update(self, u: torch.Tensor, state: torch.Tensor, batch, taps: int, seq_tiles) -> None:
         """state[slot of s][i] = the projected row of position end_s - (taps - 1) + i for every sequence s
@@ -1168,14 +1194,15 @@ class KernelOps:
                          block_table: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
                          scale: float, softcap: float, sink: bool, slopes: Optional[torch.Tensor], window: int,
                          batch, dist_a: Optional[torch.Tensor] = None, dist_b: Optional[torch.Tensor] = None,
-                         sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                         sinks: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0) -> None:
         """out[r, h] = sum_j p_j v_j over the cached positions j <= pos[r] of row r's sequence (from pos -
         window + 1 on when window > 0) with s_j = (q[r, h] . k_j) * scale, then s_j <- softcap * tanh(s_j /
         softcap) when softcap > 0, then s_j <- s_j - slopes[h] * (pos[r] - j) when slopes are given, and
         p_j = exp(s_j) / (sum exp(s) + (1 if sink else 0)).  ``vcache`` None: the values are the keys.
         ``dist_a``, ``dist_b`` [heads]: s_j <- s_j - dist_a[h] * ln(1 + dist_b[h] * (pos[r] - j)) as well.  ``sinks``
         [heads]: with ``sink``, exp(sinks[h]) joins the denominator instead of 1.  ``keep_first``: with a window,
-        the keys j < keep_first are seen too."""
+        the keys j < keep_first are seen too.  ``chunk`` > 0 (and no window): only the keys of the row's own chunk of
+        that many positions are seen, j // chunk == pos[r] // chunk."""
         n = q.shape[0]
         _need(q, self.act_dtype, "scored_attention q", 2)
         _need(out, self.act_dtype, "scored_attention out", 2)
@@ -1199,7 +1226,9 @@ class KernelOps:
                 _need(t_, torch.float32, "scored_attention " + what, 1)
                 if t_.shape[0] != heads:
                     raise KernelError(f"scored_attention: {what} is not one number per head")
-        tail = (_p(dist_a), _p(dist_b), _p(sinks), _c_int(int(keep_first)))
+        if chunk and window:
+            raise KernelError("scored_attention: chunks or a window, not both")
+        tail = (_p(dist_a), _p(dist_b), _p(sinks), _c_int(int(keep_first)), _c_int(int(chunk or 0)))
         tc_rows = self._scored_mma_rows(heads // kv_heads, dim, vdim)
         if tc_rows and (not hasattr(batch, "tile_sets") or tc_rows in batch.tile_sets):
             # The serving precision's tensor-core kernel.  Contexts beyond 256 keys are walked in spans
@@ -1210,7 +1239,9 @@ class KernelOps:
             t_seq, t_row0, t_rows, t_count = batch.query_tiles(tc_rows)
             spans, scratch, launches = 1, None, 1
             if batch.max_keys > 256:
-                spans = int(self._mixers_lib().bw_bf16_scored_attention_spans(_c_int(batch.max_keys)))
+                reach = int(chunk or (0 if keep_first else window) or 0)
+                spans = int(self._mixers_lib().bw_bf16_scored_attention_spans(_c_int(batch.max_keys), _c_int(reach),
+                                                                              _c_int(tc_rows)))
                 scratch, launches = self._latent_scratch(n * heads * spans * (vdim + 2), q.device), 2
             self._mcall("scored_attention_mma", _p(q), _c_int(q.shape[1]), _p(kcache), _p(vcache), _p(block_table),
                         _c_int(block_table.shape[1]), _p(t_seq), _p(t_row0), _p(t_rows), _c_int(t_count), _p(batch.seq_pos0),
@@ -1255,6 +1286,207 @@ class KernelOps:
                     _c_float(eps), _p(scratch), _p(out), _p(t_seq), _p(t_row0), _p(t_rows), _c_int(t_count),
                     _p(batch.seq_pos0), _p(batch.seq_slot), _c_int(n), _c_int(heads), _c_int(dim), _c_int(vdim),
                     _c_float(q_scale), self._stream(), launches=2)
+
+    # -- recurrences over a matrix of state per head (their library is loaded at first use) ---------------
+    SCAN_MODES = ("delta", "bonus", "memory")
+
+    def _scan_lib(self):
+        lib = getattr(self, "_scanlib", None)
+        if lib is None:
+            path = build.ensure_built(f"{self.kind}_scan", (), self._verbose_build)
+            try:
+                lib = ctypes.CDLL(path)
+            except OSError as e:
+                raise KernelError(f"cannot load the kernel library {path}: {e}") from None
+            lib.bw_last_error.restype = ctypes.c_char_p
+            if self._failure_word is not None:
+                lib.bw_set_failure_word(_p(self._failure_word))
+            self._scanlib = lib
+            self._scan_fns = {}
+        return lib
+
+    def _sccall(self, name: str, *args) -> None:
+        lib = self._scan_lib()
+        fn = self._scan_fns.get(name)
+        if fn is None:
+            fn = getattr(lib, f"bw_{self.kind}_{name}")
+            fn.restype = _c_int
+            self._scan_fns[name] = fn
+        rc = fn(*args)
+        if rc != 0:
+            raise KernelError(f"{name} failed ({rc}): " + lib.bw_last_error().decode("utf-8", "replace"))
+        self.launches += 1
+
+    @staticmethod
+    def scan_state_shape(mode: str, heads: int, dim: int, vdim: int):
+        """The float32 state of one request as ``state_scan`` lays it out: a head's value columns one after the
+        other, ``dim`` numbers each; with "memory" one more column (the normaliser) and behind every column four
+        numbers of which the first is the running maximum."""
+        return (heads, vdim + 1, dim + 4) if mode == "memory" else (heads, vdim, dim)
+
+    def state_scan(self, mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, o: torch.Tensor,
+                   batch, seq_tiles, heads: int, dim: int, vdim: int, decay: Optional[torch.Tensor] = None,
+                   decay_bias: Optional[torch.Tensor] = None, bonus: Optional[torch.Tensor] = None,
+                   beta: Optional[torch.Tensor] = None, forget: Optional[torch.Tensor] = None,
+                   inp: Optional[torch.Tensor] = None, forget_bias: Optional[torch.Tensor] = None,
+                   inp_bias: Optional[torch.Tensor] = None, cap: float = 0.0, aux: Optional[torch.Tensor] = None) -> None:
+        """One recurrence over the rows of every sequence of the step (``seq_tiles``: one tile per sequence), from and
+        into ``state`` [slots, *scan_state_shape] (zero at a request's first position); the outputs before their norm
+        into ``o`` [n, heads * vdim].  q, k [n, heads' * dim] (heads a multiple of heads'; head h reads head h // (heads
+        / heads')), v [n, heads * vdim]: float32, rows may be columns of wider rows.  Per head:
+
+        * "delta": S <- g S, S <- S + k (beta (v - S^T k))^T, o = S^T q; ``decay`` [n, heads * dim] = g, ``beta`` [n, heads];
+        * "bonus": o = (S + diag(u) k v^T)^T q, S <- diag(w) S + k v^T, w = exp(-exp(z + z0)); ``decay`` = z, ``decay_bias``
+          = z0 and ``bonus`` = u [heads * dim];
+        * "memory": m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, n alike, o = S^T q; i = cap tanh((inp +
+          inp_bias) / cap), f = ln sigmoid(cap tanh((forget + forget_bias) / cap)); ``inp``, ``forget`` [n, heads]; ``aux`` [n,
+          heads, 2] receives n . q and m'."""
+        n = q.shape[0]
+        if mode not in self.SCAN_MODES:
+            raise KernelError(f"state_scan: mode {mode!r}")
+        for t_, what in ((q, "q"), (k, "k"), (v, "v")):
+            _need_rows(t_, torch.float32, "state_scan " + what)
+        if q.shape[1] % dim or k.shape != q.shape or not q.shape[1] or heads % (q.shape[1] // dim) or tuple(v.shape) != (n, heads * vdim):
+            raise KernelError("state_scan: q, k and v do not fit the heads")
+        _need(state, torch.float32, "state_scan state", 4)
+        if tuple(state.shape[1:]) != self.scan_state_shape(mode, heads, dim, vdim):
+            raise KernelError(f"state_scan: the state is not [slots, *{self.scan_state_shape(mode, heads, dim, vdim)}]")
+        _need(o, torch.float32, "state_scan o", 2)
+        if tuple(o.shape) != (n, heads * vdim):
+            raise KernelError("state_scan: the output is not [rows, heads * vdim]")
+        vectors, rows = [], []
+        if mode in ("delta", "bonus"):
+            rows.append((decay, heads * dim, "decay"))
+        if mode == "delta":
+            rows.append((beta, heads, "beta"))
+        elif mode == "bonus":
+            vectors += [(decay_bias, heads * dim, "decay_bias"), (bonus, heads * dim, "bonus")]
+        else:
+            rows += [(forget, heads, "forget"), (inp, heads, "inp")]
+            vectors += [(forget_bias, heads, "forget_bias"), (inp_bias, heads, "inp_bias")]
+            if not cap > 0:
+                raise KernelError("state_scan: the gates' cap must be positive")
+            if aux is None:
+                raise KernelError("state_scan: the matrix memory needs a place for its normaliser")
+            _need(aux, torch.float32, "state_scan aux")
+            if aux.numel() != n * heads * 2:
+                raise KernelError("state_scan: aux is not [rows, heads, 2]")
+            if forget is not None and inp is not None and forget.stride(0) != inp.stride(0):
+                raise KernelError("state_scan: both gates' rows must lie equally far apart")
+        for t_, cols, what in rows:
+            if t_ is None:
+                raise KernelError(f"state_scan: {mode} needs {what}")
+            _need_rows(t_, torch.float32, "state_scan " + what)
+            if tuple(t_.shape) != (n, cols):
+                raise KernelError(f"state_scan: {what} is not [rows, {cols}]")
+        for t_, count, what in vectors:
+            if t_ is None:
+                raise KernelError(f"state_scan: {mode} needs {what}")
+            _need(t_, torch.float32, "state_scan " + what)
+            if t_.numel() != count:
+                raise KernelError(f"state_scan: {what} does not hold {count} numbers")
+        t_seq, t_row0, t_rows, t_count = seq_tiles
+        s0 = beta if mode == "delta" else forget if mode == "memory" else None
+        s1 = inp if mode == "memory" else None
+        self._sccall("state_scan", _c_int(self.SCAN_MODES.index(mode)), _p(q), _c_int(q.stride(0)), _p(k), _c_int(k.stride(0)),
+                     _p(v), _c_int(v.stride(0)), _c_int(heads // (q.shape[1] // dim)), _p(decay),
+                     _c_int(decay.stride(0) if decay is not None else 0), _p(decay_bias), _p(bonus), _p(s0), _p(s1),
+                     _c_int(s0.stride(0) if s0 is not None else 0), _p(forget_bias), _p(inp_bias), _c_float(cap), _p(state), _p(o),
+                     _p(aux), _p(t_seq), _p(t_row0), _p(t_rows), _c_int(t_count), _p(batch.seq_pos0), _p(batch.seq_slot),
+                     _c_int(n), _c_int(heads), _c_int(dim), _c_int(vdim), self._stream())
+
+    def scan_finish(self, o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: torch.Tensor, heads: int,
+                    vdim: int, gate_kind: str = "sigmoid", aux: Optional[torch.Tensor] = None, q_scale: float = 1.0) -> None:
+        """out[r, h] = y / sqrt(mean(y^2) + eps) * weight * g(gate[r, h]) with y = o[r, h], or, with ``aux`` [n, heads, 2]
+        (n . q and m), y = q_scale o / (max(|q_scale n . q|, e^-m) + 1e-6).  ``weight``: [vdim] for all heads or [heads *
+        vdim]; ``gate_kind``: "sigmoid" or "silu"; gate: float32 [n, heads * vdim], rows may be columns of wider rows."""
+        n = o.shape[0]
+        _need(o, torch.float32, "scan_finish o", 2)
+        _need(weight, torch.float32, "scan_finish weight", 1)
+        _need_rows(gate, torch.float32, "scan_finish gate")
+        _need(out, self.act_dtype, "scan_finish out", 2)
+        if gate_kind not in ("sigmoid", "silu"):
+            raise KernelError(f"scan_finish: gate {gate_kind!r}")
+        if tuple(o.shape) != (n, heads * vdim) or o.shape != gate.shape or o.shape != out.shape or \
+                weight.shape[0] not in (vdim, heads * vdim):
+            raise KernelError("scan_finish: shapes do not fit the heads")
+        if aux is not None:
+            _need(aux, torch.float32, "scan_finish aux")
+            if aux.numel() != n * heads * 2:
+                raise KernelError("scan_finish: aux is not [rows, heads, 2]")
+        self._sccall("scan_finish", _p(o), _p(aux), _c_float(q_scale), _p(weight), _c_int(int(weight.shape[0] == heads * vdim)),
+                     _p(gate), _c_int(gate.stride(0)), _c_int(int(gate_kind == "silu")), _c_float(eps), _p(out), _c_int(n),
+                     _c_int(heads), _c_int(vdim), self._stream())
+
+    def delta_prepare(self, u: torch.Tensor, beta_col: int, conv_t: torch.Tensor, conv_state: Optional[torch.Tensor],
+                      z: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, out: torch.Tensor, batch, heads: int,
+                      kv_heads: int, dim: int, vdim: int, q_scale: float, keep: bool = False) -> None:
+        """What the delta recurrence reads.  ``u`` (float32 rows): q heads, k heads (``kv_heads`` each of ``dim``), v heads
+        (``heads`` of ``vdim``), and from ``beta_col`` on the projections of beta.  q, k and v pass the convolution over time
+        with ``conv_t`` [taps, channels] (earlier inputs from ``conv_state`` [slots, taps - 1, channels], zeros before position
+        0) and SiLU; q and k heads are divided by sqrt(sum of squares + 1e-6), q times ``q_scale``; ``out`` (float32 [n, >=
+        channels + heads]) receives q | k | v | sigmoid(beta).  ``z`` (float32 rows of heads * dim) becomes exp(-exp(a_log_h)
+        softplus(z + dt_bias)).  ``keep``: every sequence of the step has one row, and its state is brought up to date here."""
+        n = u.shape[0]
+        _need_rows(u, torch.float32, "delta_prepare u")
+        _need_rows(z, torch.float32, "delta_prepare z")
+        _need_rows(out, torch.float32, "delta_prepare out")
+        _need(conv_t, torch.float32, "delta_prepare conv_t", 2)
+        _need(dt_bias, torch.float32, "delta_prepare dt_bias", 1)
+        _need(a_log, torch.float32, "delta_prepare a_log", 1)
+        taps, channels = conv_t.shape
+        if channels != 2 * kv_heads * dim + heads * vdim or beta_col < channels or u.shape[1] < beta_col + heads or \
+                tuple(z.shape) != (n, heads * dim) or dt_bias.shape[0] != heads * dim or a_log.shape[0] != heads or \
+                out.shape[0] != n or out.shape[1] < channels + heads or heads % kv_heads:
+            raise KernelError("delta_prepare: shapes do not fit the heads")
+        if conv_state is not None:
+            _need(conv_state, torch.float32, "delta_prepare conv_state", 3)
+            if tuple(conv_state.shape[1:]) != (taps - 1, channels):
+                raise KernelError("delta_prepare: the state is not [slots, taps - 1, channels]")
+        self._sccall("delta_prepare", _p(u), _c_int(u.stride(0)), _c_int(beta_col), _p(conv_t), _c_int(taps), _p(conv_state),
+                     _c_int(int(keep)), _p(z), _c_int(z.stride(0)), _p(dt_bias), _p(a_log), _p(out), _c_int(out.stride(0)),
+                     _p(batch.pos), _p(batch.row_seq), _p(batch.seq_row0), _p(batch.seq_slot), _c_int(n), _c_int(heads),
+                     _c_int(kv_heads), _c_int(dim), _c_int(vdim), _c_float(q_scale), self._stream())
+
+    def shift_mix(self, x: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, out: torch.Tensor, batch, keep: bool = False) -> None:
+        """out[s, r] = x[r] + (x'[r] - x[r]) * mu[s], x' the row before of the same sequence: from the step, from ``last``
+        [slots, ..., width], or zero at a request's first position.  x float32 [n, width], out act_dtype [mixes, n, width].
+        ``keep``: every sequence of the step has one row, which becomes its ``last``."""
+        n, width = x.shape
+        _need(x, torch.float32, "shift_mix x", 2)
+        _need(mu, torch.float32, "shift_mix mu", 2)
+        _need(last, torch.float32, "shift_mix last")
+        _need(out, self.act_dtype, "shift_mix out")
+        mixes = mu.shape[0]
+        if mu.shape[1] != width or last.numel() != last.shape[0] * width or out.numel() != mixes * n * width:
+            raise KernelError("shift_mix: shapes differ")
+        self._sccall("shift_mix", _p(x), _p(mu), _c_int(mixes), _p(last), _c_int(int(keep)), _p(out), _c_int(n), _c_int(width),
+                     _p(batch.pos), _p(batch.row_seq), _p(batch.seq_row0), _p(batch.seq_slot), self._stream())
+
+    def pair_mean(self, a: torch.Tensor, wa: torch.Tensor, b: torch.Tensor, wb: torch.Tensor, eps: float,
+                  y: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
+                  x: Optional[torch.Tensor] = None, rounded: Optional[torch.Tensor] = None) -> None:
+        """y = (a / rms(a) * wa + b / rms(b) * wb) / 2 row by row (float32).  With ``x`` instead of ``y``: x += layernorm(that
+        mean) * norm_weight, and ``rounded`` (act_dtype) receives the summed rows."""
+        n, width = a.shape
+        for t_, what in ((a, "a"), (b, "b"), (y, "y"), (x, "x")):
+            if t_ is not None:
+                _need(t_, torch.float32, "pair_mean " + what, 2)
+                if tuple(t_.shape) != (n, width):
+                    raise KernelError("pair_mean: shapes differ")
+        for t_, what in ((wa, "wa"), (wb, "wb"), (norm_weight, "norm_weight")):
+            if t_ is not None:
+                _need(t_, torch.float32, "pair_mean " + what, 1)
+                if t_.shape[0] != width:
+                    raise KernelError("pair_mean: a weight is not of the rows' width")
+        if (x is None) == (y is None) or (x is None) != (norm_weight is None):
+            raise KernelError("pair_mean: either the mean is stored, or it is normed into the stream")
+        if rounded is not None:
+            _need(rounded, self.act_dtype, "pair_mean rounded", 2)
+            if x is None or tuple(rounded.shape) != (n, width):
+                raise KernelError("pair_mean: the rounded rows are the stream's")
+        self._sccall("pair_mean", _p(a), _p(wa), _p(b), _p(wb), _c_float(eps), _p(y), _c_int(n), _c_int(width), _p(norm_weight),
+                     _c_float(norm_eps), _p(x), _p(rounded), self._stream())
 
     # -- kernels on the residual stream that only some blocks use (their library is loaded at first use) -------
     def _stream_lib(self):

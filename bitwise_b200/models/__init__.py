@@ -4,5 +4,6 @@ from . import nuderax  # noqa: F401  (registers Nuderax)
 from . import favudra  # noqa: F401  (registers Favudra)
 from . import sebavik  # noqa: F401  (registers Sebavik)
 from . import kezuvik  # noqa: F401  (registers Kezuvik)
+from . import zuzupel  # noqa: F401  (registers Zuzupel)
 
 __all__ = ["DecoderModel", "LayerRun", "sequential_schedule"]

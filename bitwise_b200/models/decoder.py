@@ -14,7 +14,7 @@ from typing import Dict, List, Optional, Sequence
 
 import torch
 
-from ..parts.base import PositionEncoding, StepContext
+from ..parts.base import PositionEncoding, SlotStateView, StepContext
 from ..parts.embedding import OutputHead, TokenEmbedding
 from ..weights.loader import ParamSpec
 
@@ -36,11 +36,12 @@ class DecoderModel:
                  schedule: Optional[Sequence[LayerRun]] = None,
                  position_encodings: Sequence[PositionEncoding] = (),
                  block_prefix: str = "model.layers.{}", embed_prefix: str = "model", shared_parts: Sequence = (),
-                 ignorable=None):
+                 ignorable=None, block_prefixes: Optional[Sequence[str]] = None):
         """``shared_parts``: parts with weights that several blocks use (a table that every layer reads a
         slice of); their tensors are declared and loaded once, with ``embed_prefix``.  ``ignorable``: a
         predicate on names of stored tensors that this model has no use for (tensors of a sublayer that a
-        layer's configuration leaves out)."""
+        layer's configuration leaves out).  ``block_prefixes``: the blocks' prefixes one by one, where a block's
+        tensors are not numbered as the block is (a model some of whose layers run another layer's block)."""
         self.config = config
         self._ignorable = ignorable
         self.embedding = embedding
@@ -48,7 +49,11 @@ class DecoderModel:
         self.head = head
         self.schedule = list(schedule) if schedule is not None else sequential_schedule(len(self.blocks))
         self.position_encodings = list(position_encodings) + list(shared_parts)
-        self.block_prefix, self.embed_prefix = block_prefix, embed_prefix
+        self.embed_prefix = embed_prefix
+        self.block_prefixes = list(block_prefixes) if block_prefixes is not None else [
+            block_prefix.format(i) for i in range(len(self.blocks))]
+        if len(self.block_prefixes) != len(self.blocks):
+            raise ValueError(f"{len(self.block_prefixes)} prefixes for {len(self.blocks)} blocks")
         self.dtype: Optional[str] = None
         self.device = None
         self._check_schedule()
@@ -106,7 +111,7 @@ class DecoderModel:
         for pe in self.position_encodings:  # encodings with weights of their own (a learned table)
             specs += pe.param_specs(self.embed_prefix)
         for i, b in enumerate(self.blocks):
-            specs += b.param_specs(self.block_prefix.format(i))
+            specs += b.param_specs(self.block_prefixes[i])
         specs += self.head.param_specs()
         return specs
 
@@ -115,7 +120,7 @@ class DecoderModel:
         for pe in self.position_encodings:
             pe.load_params(state, self.embed_prefix)
         for i, b in enumerate(self.blocks):
-            b.load_params(state, self.block_prefix.format(i))
+            b.load_params(state, self.block_prefixes[i])
         self.head.load_params(state)
         self.dtype, self.device = dtype, device
 
@@ -171,6 +176,7 @@ class DecoderModel:
             if not run.owns_cache and hasattr(view, "writable"):
                 view = type(view)(**{**view.__dict__, "writable": False})
             if run.state is not None:
-                view = type(view)(**{**view.__dict__, "state": cache_views[run.state]})
+                field = "beside" if isinstance(view, SlotStateView) else "state"
+                view = type(view)(**{**view.__dict__, field: cache_views[run.state]})
             self.blocks[run.block].forward(ctx, x, view)
         return self.head.forward(ctx, x)

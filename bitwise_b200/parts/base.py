@@ -29,12 +29,14 @@ class PagedKVNeed:
     ``window`` = None keeps every key; an integer keeps the last ``window`` positions.
     ``v_dim``: the size of a value where it differs from a key's (None: ``head_dim``); 0 keeps no
     values at all (a mixer whose values are its keys).  ``keep_first``: with a window, the first
-    ``keep_first`` positions of a request stay in the cache as well."""
+    ``keep_first`` positions of a request stay in the cache as well.  ``chunk`` (instead of a window): positions
+    see the positions of their own chunk of ``chunk`` positions only, counted from a request's first."""
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_dim: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -83,6 +85,7 @@ class PagedLatentView:
 class SlotStateView:
     state: torch.Tensor        # [slots, *shape]
     seq_slot: torch.Tensor     # int32 [step sequences]
+    beside: Optional["SlotStateView"] = None  # the run's second slot state (Mixer.state_need)
 
 
 class Workspace:
@@ -206,6 +209,9 @@ class PositionEncoding(Part):
 class Mixer(Part):
     """Mixes information between the positions of a sequence."""
 
+    # True: the mixer takes the float32 stream itself where its block reads without a norm (``forward``'s ``xn``)
+    reads_stream = False
+
     def cache_need(self):
         return None
 
@@ -213,7 +219,8 @@ class Mixer(Part):
         """A :class:`SlotStateNeed` that the mixer wants BESIDE its ``cache_need`` (a paged cache and
         a little state per request, as a convolution's last inputs), or None.  Every run of the
         mixer owns such state itself, also a run that reads another run's pages; it arrives as
-        the ``state`` field of the run's cache view."""
+        the ``state`` field of the run's cache view, or, where ``cache_need`` is slot state itself (a
+        recurrence with a convolution's inputs), as the ``beside`` field."""
         return None
 
     def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, cache) -> None:

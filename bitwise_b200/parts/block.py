@@ -131,6 +131,51 @@ class SandwichBlock(PreNormBlock):
         self.ffn_post.forward_residual(ctx, out, x)
 
 
+class PostNormBlock(PreNormBlock):
+    """A norm on the sublayer's output only: ``x += norm1(mixer(x))``, ``x += norm2(feed_forward(x))``.  The
+    sublayers read the stream itself: rounded to the activation type where their products take that (a buffer that
+    the norm before fills with the rows it has just summed), or as it is (``Mixer.reads_stream``).  A mixer
+    that has ``forward_into_norm`` hands its output to the norm in a kernel of its own.
+
+    ``opens``: the block is the first that runs, nobody has rounded the stream before it.  ``feed_forward``
+    None: the layer is its mixer alone.  ``names``: mixer, mixer_post, feed_forward, ffn_post."""
+
+    def __init__(self, width: int, mixer: Mixer, feed_forward, mixer_post: Norm, ffn_post, names: Dict[str, str],
+                 opens: bool = False):
+        super().__init__(width, mixer, feed_forward, None, None, names)
+        self.mixer_post, self.ffn_post, self.opens = mixer_post, ffn_post, opens
+
+    def _children(self, prefix: str):
+        kids = [(self.mixer, f"{prefix}.{self.names['mixer']}"), (self.mixer_post, f"{prefix}.{self.names['mixer_post']}"),
+                (self.feed_forward, f"{prefix}.{self.names['feed_forward']}"), (self.ffn_post, f"{prefix}.{self.names['ffn_post']}")]
+        return [(p, n) for p, n in kids if p is not None]
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, cache) -> None:
+        rounded, h = None, x
+        if ctx.act_dtype != torch.float32:
+            rounded = h = ctx.workspace.rows("stream_rounded", ctx.n, self.width, ctx.act_dtype)
+            if self.opens and not self.mixer.reads_stream:
+                ctx.ops.activate_rows(x, rounded)
+        out = ctx.workspace.rows("sublayer_out", ctx.n, self.width, torch.float32)
+        into = getattr(self.mixer, "forward_into_norm", None)
+        if into is not None:
+            into(ctx, h, x, cache, self.mixer_post, rounded)
+        else:
+            self.mixer.forward(ctx, x if self.mixer.reads_stream else h, out, cache, accumulate=False)
+            self._add(ctx, self.mixer_post, out, x, rounded)
+        if self.feed_forward is None:
+            return
+        self.feed_forward.forward(ctx, h, out, accumulate=False)
+        self._add(ctx, self.ffn_post, out, x, rounded)
+
+    @staticmethod
+    def _add(ctx: StepContext, norm: Norm, d, x, rounded) -> None:
+        if rounded is None:
+            norm.forward_residual(ctx, d, x)
+        else:
+            norm.forward_residual_round(ctx, d, x, rounded)
+
+
 class DepthMix:
     """What a block hands on is a weighted sum of the embedding's output and of every block's result so
     far: with X_0 the embedding's output and X_(j+1) the result of block j, block i hands on ``sum_j a[j]

@@ -78,4 +78,36 @@ class SwiGLU(FeedForward):
         ops.linear(h, self.w_down, x, residual=x if accumulate else None)
 
 
+class DenseFFN(FeedForward):
+    """``x += W_down act(W_up xn)``: no gate, no biases.  ``activation``: "relu2", the square of relu.  On the serving
+    precision the activation is applied in the up product's epilogue."""
+    graph_safe = True  # kernels only
+
+    def __init__(self, width: int, intermediate: int, names=("up", "down"), suffix: str = "", activation: str = "relu2"):
+        if activation != "relu2":
+            raise ValueError(f"feed-forward: activation {activation!r} (known: relu2)")
+        self.width, self.intermediate, self.names, self.suffix, self.activation = width, intermediate, names, suffix, activation
+        self.w_up: Optional[torch.Tensor] = None
+        self.w_down: Optional[torch.Tensor] = None
+
+    def param_specs(self, prefix: str) -> List[ParamSpec]:
+        u, d = self.names
+        return [ParamSpec(f"{prefix}.{u}{self.suffix}", (self.intermediate, self.width), MATRIX),
+                ParamSpec(f"{prefix}.{d}{self.suffix}", (self.width, self.intermediate), MATRIX)]
+
+    def load_params(self, state: Dict[str, torch.Tensor], prefix: str) -> None:
+        u, d = self.names
+        self.w_up, self.w_down = state[f"{prefix}.{u}{self.suffix}"], state[f"{prefix}.{d}{self.suffix}"]
+
+    def param_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down))
+
+    def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, accumulate: bool = True) -> None:
+        """``accumulate`` False: the output is written to ``x`` (float32) instead of added to it."""
+        h = ctx.workspace.rows("ffn_h", ctx.n, self.intermediate, ctx.act_dtype)
+        ctx.ops.linear(xn, self.w_up, h, activation=self.activation)
+        ctx.ops.linear(h, self.w_down, x, residual=x if accumulate else None)
+
+
 register_feed_forward("swiglu", SwiGLU)
+register_feed_forward("dense", DenseFFN)

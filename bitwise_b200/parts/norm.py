@@ -47,6 +47,11 @@ class RMSNorm(Norm):
         """x += norm(d): the norm of a sublayer's output ``d`` (float32) on its way into the stream."""
         ctx.ops.rmsnorm_residual(d, self.weight, self.eps, x)
 
+    def forward_residual_round(self, ctx: StepContext, d, x, rounded) -> None:
+        """``forward_residual(d, x)``; the summed rows also go into ``rounded`` in the activation type, for a sublayer
+        that reads the stream without a norm."""
+        ctx.ops.rmsnorm_residual(d, self.weight, self.eps, x, next_out=rounded)
+
     def forward_residual_then(self, ctx: StepContext, d, x, nxt: "RMSNorm", out) -> None:
         """``forward_residual(d, x)`` followed by ``nxt.forward(x, out)``, in one kernel where ``nxt`` is a
         norm of this kind."""
@@ -76,6 +81,9 @@ class LayerNorm(RMSNorm):
         """x += norm(d) with the row statistics of the sublayer's output ``d`` (float32); a constant factor on
         what is added is this norm's ``gain``."""
         ctx.ops.layernorm_residual(d, self.weight, self.eps, x)
+
+    def forward_residual_round(self, ctx: StepContext, d, x, rounded) -> None:
+        ctx.ops.layernorm_residual(d, self.weight, self.eps, x, next_out=rounded)
 
     def forward_residual_then(self, ctx: StepContext, d, x, nxt: "LayerNorm", out) -> None:
         if type(nxt) is not LayerNorm or nxt.width != self.width:

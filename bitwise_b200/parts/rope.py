@@ -138,14 +138,32 @@ class RampScaling:
         return f / self.factor * ramp + f * (1.0 - ramp)
 
 
+class LinearScaling:
+    """The other rescaling: every frequency divided by one ``factor`` (positions count that much slower)."""
+
+    def __init__(self, factor: float):
+        if not factor > 0:
+            raise ValueError("a rescaling of rotary frequencies needs a positive factor")
+        self.factor = float(factor)
+
+    def key(self):
+        return ("linear", self.factor)
+
+    def gain(self) -> float:
+        return 1.0
+
+    def frequencies(self, dims: int, base: float) -> np.ndarray:
+        return np.array([base ** (-2.0 * i / dims) / self.factor for i in range(dims // 2)], dtype=np.float64)
+
+
 class HalfRotaryEncoding(RotaryEncoding):
     """Tables for a rotation whose pair i is made of entries i and i + dims / 2 of the turned part (the
     kernels are told the layout; the tables are [positions, dims / 2] either way), with an optional
-    :class:`RampScaling`.  Frequencies and angles are formed in 64-bit and rounded once, to the 32-bit
+    :class:`RampScaling` or :class:`LinearScaling`.  Frequencies and angles are formed in 64-bit and rounded once, to the 32-bit
     tables that the kernels read; the tables carry the scaling's gain."""
     layout = "half"
 
-    def __init__(self, dims: int, base: float, scaling: Optional[RampScaling] = None, positions: int = 0):
+    def __init__(self, dims: int, base: float, scaling=None, positions: int = 0):
         if dims % 2 or dims <= 0:
             raise ValueError(f"rotary encoding needs an even number of turned entries, got {dims}")
         if not base > 0:

@@ -12,7 +12,8 @@ Before the scores, each on or off by a constructor argument:
 * a root-mean-square norm of every head of q and of k, with one weight of the head's size each
   (``qk_norm="unit"``: without weights, the head is only divided by its root mean square);
 * a rotation of the first ``rot_dims`` entries of every head of q and k: entries 2i and 2i + 1
-  form pair i, turned by ``pos * base ** (-2i / rot_dims)`` (tables from a ``RotaryEncoding``).
+  form pair i, turned by ``pos * base ** (-2i / rot_dims)`` (tables from a ``RotaryEncoding``), or entries i
+  and i + rot_dims / 2 (a ``HalfRotaryEncoding``, whose tables may carry rescaled frequencies).
 
 On the scores ``s = (q . k) * scale``:
 
@@ -21,6 +22,8 @@ On the scores ``s = (q . k) * scale``:
 * ``distance_log``: ``s <- s - a_h * ln(1 + b_h * (i - j))`` with two learned numbers per head;
 * ``window``: position i sees the keys j with ``0 <= i - j < window`` (every j <= i without), and
   with ``keep_first`` also the keys ``j < keep_first``, at their true distance;
+* ``chunk`` (instead of a window): position i sees the keys j <= i of its own chunk, ``j // chunk == i //
+  chunk``, counted from the sequence's first position;
 * ``sink``: one is added to the softmax's denominator (a key of score 0 that has no value);
   ``sink="learned"``: ``exp(sink_h)`` with a learned number per head instead.
 
@@ -54,6 +57,7 @@ def distance_slopes(heads: int, exponent: float = 8.0) -> List[float]:
 
 class ScoredAttention(Mixer):
     graph_safe = True  # kernels only; launches depend on the step's sizes and ctx.max_keys
+    stacks_input = True  # ``w_in`` is one product of the mixer's input, and ``forward`` takes its result ready-made
 
     NAMES = {"q": "q", "k": "k", "v": "v", "out": "o", "conv": ".conv", "norm": ".norm", "bias": ".b", "vmix": "vmix",
              "dist_a": "r1", "dist_b": "r2", "sink": "sink", "gate": "g"}
@@ -63,7 +67,10 @@ class ScoredAttention(Mixer):
                  softcap: Optional[float] = None, sink: bool = False, slopes: Optional[Sequence[float]] = None,
                  window: Optional[int] = None, values_are_keys: bool = False, shares_cache: bool = False,
                  names: Optional[Dict[str, str]] = None, bias: bool = False, distance_log: bool = False,
-                 keep_first: int = 0, value_mix: Optional[str] = None, gate: Optional[str] = None):
+                 keep_first: int = 0, value_mix: Optional[str] = None, gate: Optional[str] = None,
+                 chunk: Optional[int] = None):
+        if chunk is not None and (window is not None or chunk <= 0):
+            raise ValueError("chunks have a positive size and stand instead of a window")
         if heads % kv_heads:
             raise ValueError(f"{heads} heads are not a multiple of {kv_heads} key/value heads")
         if values_are_keys and vdim != dim:
@@ -81,7 +88,8 @@ class ScoredAttention(Mixer):
         self.taps = int(conv_taps or 0)  # 0: no convolution; 1: a factor per channel and no state
         self.qk_norm, self.position, self.rot_dims = bool(qk_norm), position, rot_dims
         self.unit_norm = qk_norm == "unit"  # no weights: a head is divided by its root mean square and no more
-        self.softcap, self.sink, self.window = softcap, bool(sink), window
+        self.softcap, self.sink, self.window, self.chunk = softcap, bool(sink), window, chunk
+        self.half_layout = getattr(position, "layout", "pairs") == "half"
         self.learned_sink = sink == "learned"
         self.bias, self.distance_log, self.value_mix = bool(bias), bool(distance_log), value_mix
         self.keep_first = int(keep_first or 0) if window else 0
@@ -99,7 +107,7 @@ class ScoredAttention(Mixer):
     # -- what the cache keeps --------------------------------------------------------------
     def cache_need(self):
         return PagedKVNeed(self.kv_heads, self.dim, self.window, v_dim=0 if self.values_are_keys else self.vdim,
-                           keep_first=self.keep_first)
+                           keep_first=self.keep_first, chunk=self.chunk)
 
     def state_need(self):
         """The convolution's inputs of the last ``taps - 1`` positions, for every channel it runs on."""
@@ -187,14 +195,19 @@ class ScoredAttention(Mixer):
 
     # -- one step --------------------------------------------------------------------------
     def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, cache: PagedKVView,
-                accumulate: bool = True) -> None:
-        """``accumulate`` False: the output is written to ``x`` instead of added to it."""
+                accumulate: bool = True, projected: Optional[torch.Tensor] = None) -> None:
+        """``accumulate`` False: the output is written to ``x`` instead of added to it.  ``projected``: the product
+        of ``xn`` with ``w_in`` (float32 rows) where the caller has formed it."""
         ops, ws, n = ctx.ops, ctx.workspace, ctx.n
         gate_logits = None
         if self.gate is not None:
-            wide = ws.rows("scored_qkv32", n, self.cols + self.gate.cols, torch.float32)
-            ops.linear(xn, self.w_in, wide)
+            wide = projected
+            if wide is None:
+                wide = ws.rows("scored_qkv32", n, self.cols + self.gate.cols, torch.float32)
+                ops.linear(xn, self.w_in, wide)
             u, gate_logits = wide[:, :self.cols], wide[:, self.cols:]
+        elif projected is not None:
+            u = projected
         else:
             u = ws.rows("scored_qkv32", n, self.cols, torch.float32)
             ops.linear(xn, self.w_in, u)
@@ -204,6 +217,8 @@ class ScoredAttention(Mixer):
         state = cache.state if self.taps > 1 else None
         writes = cache.writable and not self.shares_cache
         extra = {}
+        if self.half_layout and cos is not None:
+            extra["half_layout"] = True
         if self.bias:
             extra["bias"] = self.b_in
         if self.value_mix and writes:
@@ -221,7 +236,8 @@ class ScoredAttention(Mixer):
         mixed = ws.rows("scored_mixed", n, self.heads * self.vdim, ctx.act_dtype)
         ops.scored_attention(q, cache.k, cache.v, cache.block_table, mixed, self.heads, self.kv_heads, self.dim, self.vdim,
                              self.scale, self.softcap or 0.0, self.sink, self.slopes, self.window or 0, ctx,
-                             dist_a=self.dist_a, dist_b=self.dist_b, sinks=self.sinks, keep_first=self.keep_first)
+                             dist_a=self.dist_a, dist_b=self.dist_b, sinks=self.sinks, keep_first=self.keep_first,
+                             **({"chunk": self.chunk} if self.chunk else {}))
         if self.gate is not None:
             self.gate.apply(ctx, xn, mixed, gate_logits)
         ops.linear(mixed, self.w_o, x, residual=x if accumulate else None)

@@ -25,7 +25,9 @@ class CpuOps:
 
     def rmsnorm_residual(self, d, weight, eps, x, next_weight=None, next_eps=0.0, next_out=None):
         x += (d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps)) * weight
-        if next_out is not None:
+        if next_out is not None and next_weight is None:
+            next_out.copy_(x.to(next_out.dtype))
+        elif next_out is not None:
             self.rmsnorm(x, next_weight, next_eps, next_out)
 
     # -- scored attention and the linear recurrence (stand-ins shaped like the kernels' interface) --
@@ -33,7 +35,8 @@ class CpuOps:
         return [max(1, 32 // group)]
 
     def qkv_prepare(self, u, conv_w, conv_state, q_norm, k_norm, eps, cos, sin, ctx, block_table, kcache, vcache, q_out,
-                    heads, write_kv_heads, dim, vdim, conv_wt=None, bias=None, vmix_src=None, vmix_lambda=None, v_keep=None):
+                    heads, write_kv_heads, dim, vdim, conv_wt=None, bias=None, vmix_src=None, vmix_lambda=None, v_keep=None,
+                    half_layout=False):
         n, cols = u.shape
         page = kcache.shape[2]
         if bias is not None:
@@ -59,7 +62,9 @@ class CpuOps:
             t = t.reshape(n, -1, size)
             if w is not None:
                 t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
-            if cos is not None:
+            if cos is not None and half_layout:
+                t = self._turn(t, p, cos, sin, True)
+            elif cos is not None:
                 pairs = cos.shape[1]
                 c, sn = cos[p][:, None, :], sin[p][:, None, :]
                 a, b = t[..., 0:2 * pairs:2].clone(), t[..., 1:2 * pairs:2].clone()
@@ -101,13 +106,13 @@ class CpuOps:
                     state[slot, j] = old[pos - pos0 + taps - 1]
 
     def scored_attention(self, q, kcache, vcache, block_table, out, heads, kv_heads, dim, vdim, scale, softcap, sink,
-                         slopes, window, ctx, dist_a=None, dist_b=None, sinks=None, keep_first=0):
+                         slopes, window, ctx, dist_a=None, dist_b=None, sinks=None, keep_first=0, chunk=0):
         n = q.shape[0]
         page = kcache.shape[2]
         grp = heads // kv_heads
         for r in range(n):
             p = int(ctx.pos[r])
-            lo = max(0, p - window + 1) if window else 0
+            lo = max(0, p - window + 1) if window else p // chunk * chunk if chunk else 0
             idx = torch.arange(lo, p + 1)
             if window and keep_first and lo > 0:
                 idx = torch.cat([torch.arange(0, min(keep_first, lo)), idx])
@@ -248,11 +253,124 @@ class CpuOps:
         inv = torch.rsqrt(src.pow(2).mean(-1, keepdim=True) + eps)
         out.copy_(((src * inv) * weight).to(out.dtype))
 
-    def linear(self, x, w, out, residual=None):
+    def linear(self, x, w, out, residual=None, activation=None):
         y = x.float() @ w.float().t()
+        if activation is not None:
+            y = self._activated(y, activation)
         if residual is not None:
             y = residual + y
         out.copy_(y.to(out.dtype))
+
+    # -- recurrences over a matrix of state per head, the token shift, two mixers side by side ------------
+    @staticmethod
+    def _activated(y, activation):
+        return {None: lambda t: t, "relu2": lambda t: torch.relu(t) ** 2, "tanh": torch.tanh}[activation](y)
+
+    def activate_rows(self, x, out, activation=None):
+        out.copy_(self._activated(x, activation).to(out.dtype))
+
+    def shift_mix(self, x, mu, last, out, ctx, keep=False):
+        n, width = x.shape
+        for r in range(n):
+            s = int(ctx.row_seq[r])
+            slot = last[int(ctx.seq_slot[s])].view(-1)
+            if r > int(ctx.seq_row0[s]):
+                before = x[r - 1]
+            else:
+                before = slot.clone() if int(ctx.pos[r]) > 0 else torch.zeros(width)
+            out.view(-1, n, width)[:, r] = (x[r] + (before - x[r]) * mu).to(out.dtype)
+            if keep:
+                slot.copy_(x[r])
+
+    def delta_prepare(self, u, beta_col, conv_t, conv_state, z, dt_bias, a_log, out, ctx, heads, kv_heads, dim, vdim, q_scale,
+                      keep=False):
+        n, (taps, channels) = u.shape[0], conv_t.shape
+        y = torch.zeros(n, channels)
+        for r in range(n):
+            s = int(ctx.row_seq[r])
+            row0, slot = int(ctx.seq_row0[s]), int(ctx.seq_slot[s])
+            for j in range(taps):
+                back = taps - 1 - j
+                if int(ctx.pos[r]) - back < 0:
+                    continue
+                src = u[r - back, :channels] if r - back >= row0 else conv_state[slot, taps - 1 - (row0 - (r - back))]
+                y[r] += conv_t[j] * src
+            if keep and conv_state is not None:
+                old = conv_state[slot].clone() if int(ctx.pos[r]) > 0 else torch.zeros(taps - 1, channels)
+                if 0 < int(ctx.pos[r]) < taps - 1:
+                    old[:taps - 1 - int(ctx.pos[r])] = 0
+                conv_state[slot] = torch.cat([old[1:], u[r:r + 1, :channels]], 0)
+        y = y * torch.sigmoid(y)
+        qk = y[:, :2 * kv_heads * dim].reshape(n, 2 * kv_heads, dim)
+        qk = qk / torch.sqrt(qk.pow(2).sum(-1, keepdim=True) + 1e-6)
+        qk[:, :kv_heads] *= q_scale
+        out[:, :2 * kv_heads * dim] = qk.reshape(n, -1)
+        out[:, 2 * kv_heads * dim:channels] = y[:, 2 * kv_heads * dim:]
+        out[:, channels:channels + heads] = torch.sigmoid(u[:, beta_col:beta_col + heads])
+        soft = torch.nn.functional.softplus(z + dt_bias).view(n, heads, dim)
+        z.copy_(torch.exp(-torch.exp(a_log).view(1, -1, 1) * soft).reshape(n, -1))
+
+    def state_scan(self, mode, q, k, v, state, o, ctx, tiles, heads, dim, vdim, decay=None, decay_bias=None, bonus=None,
+                   beta=None, forget=None, inp=None, forget_bias=None, inp_bias=None, cap=0.0, aux=None):
+        n = q.shape[0]
+        rep = heads // (q.shape[1] // dim)
+        qh = q.reshape(n, -1, dim).repeat_interleave(rep, 1)
+        kh = k.reshape(n, -1, dim).repeat_interleave(rep, 1)
+        vh = v.reshape(n, heads, vdim)
+        t_seq, t_row0, t_rows, count = tiles
+        for i in range(count):
+            s, row0, cnt = int(t_seq[i]), int(t_row0[i]), int(t_rows[i])
+            st = state[int(ctx.seq_slot[s])]
+            if int(ctx.seq_pos0[s]) == 0:
+                st.zero_()
+            S = st[:, :vdim, :dim]                                    # [heads, value column, key row]
+            for r in range(row0, row0 + cnt):
+                kv = vh[r][:, :, None] * kh[r][:, None, :]
+                if mode == "delta":
+                    S.mul_(decay[r].view(heads, 1, dim))
+                    w = beta[r][:, None] * (vh[r] - torch.einsum("hvd,hd->hv", S, kh[r]))
+                    S.add_(w[:, :, None] * kh[r][:, None, :])
+                    out = torch.einsum("hvd,hd->hv", S, qh[r])
+                elif mode == "bonus":
+                    out = torch.einsum("hvd,hd->hv", S + bonus.view(heads, 1, dim) * kv, qh[r])
+                    w = torch.exp(-torch.exp(decay[r] + decay_bias)).view(heads, 1, dim)
+                    S.mul_(w).add_(kv)
+                else:
+                    f = torch.nn.functional.logsigmoid(cap * torch.tanh((forget[r] + forget_bias) / cap))
+                    g = cap * torch.tanh((inp[r] + inp_bias) / cap)
+                    m = st[:, 0, dim].clone()
+                    new = torch.maximum(f + m, g)
+                    keep, add = torch.exp(f + m - new), torch.exp(g - new)
+                    S.mul_(keep[:, None, None]).add_(add[:, None, None] * kv)
+                    st[:, vdim, :dim] = keep[:, None] * st[:, vdim, :dim] + add[:, None] * kh[r]
+                    st[:, :, dim] = new[:, None]
+                    aux.view(n, heads, 2)[r, :, 0] = (st[:, vdim, :dim] * qh[r]).sum(-1)
+                    aux.view(n, heads, 2)[r, :, 1] = new
+                    out = torch.einsum("hvd,hd->hv", S, qh[r])
+                o[r] = out.reshape(-1)
+
+    def scan_finish(self, o, weight, gate, eps, out, heads, vdim, gate_kind="sigmoid", aux=None, q_scale=1.0):
+        n = o.shape[0]
+        y = o.view(n, heads, vdim)
+        if aux is not None:
+            a = aux.view(n, heads, 2)
+            y = y * q_scale / (torch.maximum((a[..., 0] * q_scale).abs(), torch.exp(-a[..., 1])) + 1e-6)[..., None]
+        y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight.view(-1, vdim)
+        g = torch.sigmoid(gate) * (gate if gate_kind == "silu" else 1.0)
+        out.copy_((y.reshape(n, -1) * g).to(out.dtype))
+
+    def pair_mean(self, a, wa, b, wb, eps, y=None, norm_weight=None, norm_eps=0.0, x=None, rounded=None):
+        unit = lambda t: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+        mean = 0.5 * (unit(a) * wa + unit(b) * wb)
+        if y is not None:
+            y.copy_(mean)
+            return
+        x += self._layer_normed(mean, norm_eps) * norm_weight
+        if rounded is not None:
+            rounded.copy_(x.to(rounded.dtype))
+
+    def add_rows(self, x, d):
+        x += d
 
     def fuses_swiglu(self, width, intermediate, activation="silu"):
         return False
@@ -272,7 +390,9 @@ class CpuOps:
 
     def layernorm_residual(self, d, weight, eps, x, next_weight=None, next_eps=0.0, next_out=None):
         x += self._layer_normed(d, eps) * weight
-        if next_out is not None:
+        if next_out is not None and next_weight is None:
+            next_out.copy_(x.to(next_out.dtype))
+        elif next_out is not None:
             self.layernorm(x, next_weight, next_eps, next_out)
 
     @staticmethod
