@@ -1089,6 +1089,221 @@ def compare_kezuvik(args, pk):
     return line
 
 
+# ---- the Zuzupel design beside Favudra at equal size (--compare zuzupel) ------------------------
+ZUZUPEL_SIZES = {
+    # width, layers; wkv heads x dim; delta rule: heads on kv_heads, dim, vdim, taps, low ranks; attention: heads on
+    # kv_heads of dim, chunk; matrix memory: heads, dim, vdim; ff, vocab
+    "small": dict(width=1024, layers=4, r_heads=16, r_dim=64, d_heads=8, d_kv_heads=8, d_dim=128, d_vdim=128, taps=4, rank=64,
+                  heads=8, kv_heads=2, dim=128, chunk=512, m_heads=4, m_dim=128, m_vdim=256, ff=4096, vocab=32768),
+    "medium": dict(width=2048, layers=4, r_heads=32, r_dim=64, d_heads=16, d_kv_heads=16, d_dim=128, d_vdim=128, taps=4, rank=128,
+                   heads=16, kv_heads=4, dim=128, chunk=1024, m_heads=8, m_dim=128, m_vdim=256, ff=8192, vocab=32768),
+}
+
+
+def zuzupel_config(z):
+    """Layers in the order token-shift recurrence, delta rule, attention in chunks beside a matrix memory, delta rule, and so
+    on; every layer with a feed-forward and weights of its own."""
+    from bitwise_b200.config import (ChannelDeltaConfig, ChunkAttentionConfig, MatrixMemoryConfig, ParallelConfig, WkvConfig,
+                                     ZuzupelConfig, ZuzupelLayerConfig)
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 == 0:
+            m = WkvConfig(z["r_heads"], z["r_dim"], decay_rank=z["rank"])
+        elif i % 4 == 2:
+            m = ParallelConfig(ChunkAttentionConfig(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, 1e6, z["dim"], 4.0,
+                                                    z["chunk"]),
+                               MatrixMemoryConfig(z["m_heads"], z["m_dim"], z["m_vdim"], 15.0))
+        else:
+            m = ChannelDeltaConfig(z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"], z["taps"], decay_rank=z["rank"],
+                                   gate_rank=z["rank"])
+        layers.append(ZuzupelLayerConfig(m, z["ff"]))
+    return ZuzupelConfig(vocab=z["vocab"], width=z["width"], eps=1e-5, layers=tuple(layers))
+
+
+def zuzupel_twin(z):
+    """Favudra with the same width, layers, vocabulary and weights per feed-forward (three matrices of two thirds of the inner
+    size): gated linear attention where Zuzupel has a recurrence (the heads of its delta rule), window attention of the chunk's
+    size, with the same heads, where it has attention beside a matrix memory."""
+    from bitwise_b200.config import FavudraConfig, FavudraLayerConfig, FavudraMixerConfig
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 == 2:
+            m = FavudraMixerConfig("attention_2", z["heads"], z["dim"], z["dim"], kv_heads=z["kv_heads"], scale=z["dim"] ** -0.5,
+                                   window=z["chunk"])
+        else:
+            m = FavudraMixerConfig("gla", z["d_heads"], z["d_dim"], z["d_vdim"], tau=16.0, decay_rank=z["rank"])
+        layers.append(FavudraLayerConfig(m, z["ff"] * 2 // 3 // 64 * 64))
+    return FavudraConfig(vocab=z["vocab"], width=z["width"], eps=1e-5, embedding_scale=z["width"] ** 0.5, logit_scale=0.25,
+                         layers=tuple(layers))
+
+
+def zuzupel_kernel_table(z, pk, page=16):
+    """Every kernel that the design added or changed, alone at the size's shapes, beside the like kernel of an
+    earlier design: milliseconds and the fraction of its roofline (measured copy bandwidth, bf16 peak, or the CUDA cores'
+    float32 rate for the walks along a prompt)."""
+    import torch
+    from bitwise_b200.kernels.ops import get_ops
+    from bitwise_b200.parts.rope import HalfRotaryEncoding, LinearScaling, RotaryEncoding
+    from bitwise_b200.parts.scored_attention import SEQUENCE_TILE, distance_slopes
+    ops = get_ops("bfloat16")
+    dev, bf = "cuda:0", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    H, G, hd, chunk, width, ff, taps = z["heads"], z["kv_heads"], z["dim"], z["chunk"], z["width"], z["ff"], z["taps"]
+    out = {}
+    fp32 = pk.get("fp32_tflops", 74.0)
+
+    def frac_flops(flops, ms, peak=None):
+        return round(flops / (ms / 1e3) / 1e12 / (peak or pk["bf16_tflops"]), 4)
+
+    def frac_bytes(nbytes, ms):
+        return round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4)
+
+    def put(name, ms, frac, twin_ms, twin_frac, bound, twin):
+        out[name] = {"ms": round(ms, 4), "frac": frac, "twin_ms": round(twin_ms, 4), "twin_frac": twin_frac, "bound": bound,
+                     "twin": twin, "gap_ratio": round(twin_frac / frac, 2) if frac else None}
+
+    rnd = lambda *s: torch.randn(*s, device=dev)
+    ones = lambda *s: torch.ones(*s, device=dev)
+    cos_h, sin_h = HalfRotaryEncoding(hd, 1e6, LinearScaling(4.0), positions=2048).rotary_tables(dev)
+    cos_p, sin_p = RotaryEncoding(hd, 1e6, positions=2048).rotary_tables(dev)
+    slopes = torch.tensor(distance_slopes(H), dtype=torch.float32, device=dev)
+    for label, seqs in (("prefill_2048", [(0, 2048)]), ("decode_b8_ctx2048", [(2047, 1)] * 8)):
+        keys = max(p0 + c for p0, c in seqs)
+        blocks = (keys + page - 1) // page
+        nseq = len(seqs)
+        table = torch.arange(nseq * blocks, dtype=torch.int32, device=dev).reshape(nseq, blocks)
+        b = KernelBatch(seqs, sorted(set(ops.scored_attention_tile_heights(H // G, hd, hd)) | {SEQUENCE_TILE}), dev)
+        b.seq_slot = torch.arange(nseq, dtype=torch.int32, device=dev)
+        n = b.n
+        prefill = n > nseq
+        tiles = b.query_tiles(SEQUENCE_TILE)
+        # the recurrences with what finishes their outputs, beside gated linear attention of the same heads and sizes
+        for mode, heads, kvh, dim, vdim, work in (("bonus", z["r_heads"], z["r_heads"], z["r_dim"], z["r_dim"], 4.0),
+                                                  ("delta", z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"], 6.0),
+                                                  ("memory", z["m_heads"], z["m_heads"], z["m_dim"], z["m_vdim"], 4.0)):
+            q, k, v, gate = rnd(n, kvh * dim), rnd(n, kvh * dim) * dim ** -0.5, rnd(n, heads * vdim), rnd(n, heads * vdim)
+            state = torch.zeros(nseq + 1, *ops.scan_state_shape(mode, heads, dim, vdim), device=dev)
+            o32, og = torch.empty(n, heads * vdim, device=dev), torch.empty(n, heads * vdim, dtype=bf, device=dev)
+            aux = torch.empty(n, heads * 2, device=dev) if mode == "memory" else None
+            extra = {"delta": dict(decay=torch.rand(n, heads * dim, device=dev), beta=torch.rand(n, heads, device=dev), qk=torch.rand(n, kvh, device=dev)),
+                     "bonus": dict(decay=rnd(n, heads * dim), decay_bias=rnd(heads * dim), bonus=rnd(heads * dim)),
+                     "memory": dict(inp=rnd(n, heads), forget=rnd(n, heads), inp_bias=rnd(heads), forget_bias=rnd(heads), cap=15.0,
+                                    aux=aux)}[mode]
+            w = ones(vdim) if mode == "delta" else ones(heads * vdim)
+            run = lambda: (ops.state_scan(mode, q, k, v, state, o32, b, tiles, heads, dim, vdim, **extra),
+                           ops.scan_finish(o32, w, gate, 1e-5, og, heads, vdim, aux=aux))
+            ms = timed_device(run, flush=flush)
+            ms_alone = timed_device(lambda: ops.state_scan(mode, q, k, v, state, o32, b, tiles, heads, dim, vdim, **extra), flush=flush)
+            uu, zz = rnd(n, 2 * heads * (dim + vdim)), rnd(n, heads * dim)
+            gst = torch.zeros(nseq + 1, heads, dim, vdim, device=dev)
+            gb, gw = torch.zeros(heads * dim, device=dev), ones(vdim)
+            tms = timed_device(lambda: ops.gla_scan(uu, zz, gb, 16.0, gst, gw, 1e-5, og, heads, dim, vdim, dim ** -0.5, b, tiles,
+                                                    scratch=o32), flush=flush)
+            per = n * heads * dim * vdim
+            if prefill:
+                put(f"{mode}_scan_{label}", ms, frac_flops(work * per, ms, fp32), tms, frac_flops(4.0 * per, tms, fp32),
+                    "float32 on the CUDA cores", "gated linear attention")
+            else:
+                put(f"{mode}_scan_{label}", ms, frac_bytes(8 * per, ms), tms, frac_bytes(8 * per, tms), "copy bandwidth",
+                    "gated linear attention")
+            out[f"{mode}_scan_{label}"]["scan_alone_ms"] = round(ms_alone, 4)
+            del q, k, v, gate, state, uu, zz, gst
+        # attention inside chunks beside attention inside a window of the chunk's size
+        kc, vc = rnd(nseq * blocks + 1, G, page, hd).to(bf), rnd(nseq * blocks + 1, G, page, hd).to(bf)
+        wq, wo = rnd(n, H * hd).to(bf), torch.empty(n, H * hd, dtype=bf, device=dev)
+        cpairs = sum(sum(p % chunk + 1 for p in range(p0, p0 + c)) for p0, c in seqs)
+        wpairs = sum(sum(min(p + 1, chunk) for p in range(p0, p0 + c)) for p0, c in seqs)
+        ms = timed_device(lambda: ops.scored_attention(wq, kc, vc, table, wo, H, G, hd, hd, hd ** -0.5, 0.0, False, None, 0, b, chunk=chunk),
+                          flush=flush)
+        tms = timed_device(lambda: ops.scored_attention(wq, kc, None, table, wo, H, G, hd, hd, hd ** -0.5, 0.0, False, slopes, chunk, b),
+                           flush=flush)
+        if prefill:
+            put(f"chunk_attention_{label}", ms, frac_flops(4.0 * H * hd * cpairs, ms), tms, frac_flops(4.0 * H * hd * wpairs, tms),
+                "bf16 peak", "window attention with slopes")
+        else:
+            put(f"chunk_attention_{label}", ms, frac_bytes(cpairs * G * hd * 4, ms), tms, frac_bytes(wpairs * G * hd * 2, tms),
+                "copy bandwidth", "window attention with slopes (keys only)")
+        # biases, weighted norm, half-layout rotation, store beside convolution, norm, rotation of pairs, store
+        cols = (H + 2 * G) * hd
+        u, nw, bias, cw = rnd(n, cols), ones(hd), rnd(cols), rnd(cols, taps)
+        cwt, st = cw.t().contiguous(), torch.zeros(nseq + 1, taps - 1, cols, device=dev)
+        ms = timed_device(lambda: ops.qkv_prepare(u, None, None, nw, nw, 1e-5, cos_h, sin_h, b, table, kc, vc, wq, H, G, hd, hd, bias=bias,
+                                                  half_layout=True), flush=flush)
+        tms = timed_device(lambda: (ops.qkv_prepare(u, cw, st, nw, nw, 1e-5, cos_p, sin_p, b, table, kc, vc, wq, H, G, hd, hd, conv_wt=cwt),
+                                    ops.conv_state_update(u, st, b, taps, tiles)), flush=flush)
+        put(f"bias_norm_rotate_store_{label}", ms, frac_bytes(n * cols * 6, ms), tms, frac_bytes(n * cols * 6, tms), "copy bandwidth",
+            "convolution, norm, rotation, store")
+        del kc, vc
+        # what the delta rule reads (convolution, SiLU, unit vectors, decays, beta) beside the same twin kernels
+        DH, DG, dd, dv = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"]
+        ch = 2 * DG * dd + DH * dv
+        u, zz, ready = rnd(n, ch + DH), rnd(n, DH * dd), torch.empty(n, ch + DH + DG + (-DH - DG) % 4, device=dev)
+        ct, dst = rnd(taps, ch), torch.zeros(nseq + 1, taps - 1, ch, device=dev)
+        db, al = rnd(DH * dd), rnd(DH)
+        run = lambda: (ops.delta_prepare(u, ch, ct, dst, zz, db, al, ready, b, DH, DG, dd, dv, dd ** -0.5, keep=not prefill),
+                       ops.conv_state_update(u[:, :ch], dst, b, taps, tiles) if prefill else None)
+        ms = timed_device(run, flush=flush)
+        by = n * (ch * 8 + DH * dd * 8)
+        put(f"delta_prepare_{label}", ms, frac_bytes(by, ms), tms, frac_bytes(n * cols * 6, tms), "copy bandwidth",
+            "convolution, norm, rotation, store")
+        # the token shift beside the norm with a convolution over rows
+        x, mu, last = rnd(n, width), rnd(5, width), torch.zeros(nseq + 1, 1, width, device=dev)
+        mixes = torch.empty(5, n, width, dtype=bf, device=dev)
+        run = lambda: (ops.shift_mix(x, mu, last, mixes, b, keep=not prefill),
+                       ops.conv_state_update(x, last, b, 2, tiles) if prefill else None)
+        ms = timed_device(run, flush=flush)
+        ww, wt, cst = ones(width), rnd(taps, width), torch.zeros(nseq + 1, taps - 1, width, device=dev)
+        xn, normed = torch.empty(n, width, dtype=bf, device=dev), torch.empty(n, width, device=dev)
+        tms = timed_device(lambda: (ops.norm_conv(x, ww, 1e-5, wt, cst, 0, b, xn, normed, 0),
+                                    ops.conv_state_update(normed, cst, b, taps, tiles)), flush=flush)
+        put(f"token_shift_{label}", ms, frac_bytes(n * width * 14, ms), tms, frac_bytes(n * width * 6, tms), "copy bandwidth",
+            "norm with a convolution over rows")
+        # the norms behind a sublayer: rounding the stream, and the mean of two mixers, beside the norm with the next norm
+        a, c = rnd(n, width), rnd(n, width)
+        tms = timed_device(lambda: ops.layernorm_residual(a, ww, 1e-5, x, next_weight=ww, next_eps=1e-5, next_out=xn), flush=flush)
+        tf = frac_bytes(n * width * 14, tms)
+        ms = timed_device(lambda: ops.layernorm_residual(a, ww, 1e-5, x, next_out=xn), flush=flush)
+        put(f"norm_after_sublayer_{label}", ms, frac_bytes(n * width * 14, ms), tms, tf, "copy bandwidth", "layer norm with the next norm")
+        ms = timed_device(lambda: ops.pair_mean(a, ww, c, ww, 1e-5, norm_weight=ww, norm_eps=1e-5, x=x, rounded=xn), flush=flush)
+        put(f"pair_mean_norm_{label}", ms, frac_bytes(n * width * 18, ms), tms, tf, "copy bandwidth", "layer norm with the next norm")
+        # the up product with the square of relu in its epilogue beside the same product without
+        xb, wu, hh = rnd(n, width).to(bf), (rnd(ff, width) * 0.02).to(bf), torch.empty(n, ff, dtype=bf, device=dev)
+        ms = timed_device(lambda: ops.linear(xb, wu, hh, activation="relu2"), flush=flush)
+        tms = timed_device(lambda: ops.linear(xb, wu, hh), flush=flush)
+        if prefill:
+            fl = 2.0 * n * ff * width
+            put(f"up_relu2_{label}", ms, frac_flops(fl, ms), tms, frac_flops(fl, tms), "bf16 peak", "the product alone")
+        else:
+            by = ff * width * 2
+            put(f"up_relu2_{label}", ms, frac_bytes(by, ms), tms, frac_bytes(by, tms), "copy bandwidth", "the product alone")
+        torch.cuda.empty_cache()
+    return out
+
+
+def compare_zuzupel(args, pk):
+    import torch
+    from bitwise_b200 import Model
+    z = ZUZUPEL_SIZES[args.size]
+    line = {"metric": f"Zuzupel beside Favudra at equal size ({args.size}): prefill of 2,048 tokens and decode at batch "
+                      f"{args.batch}, {args.ctx or 2048:,}-token contexts", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16",
+            "data": "synthetic: random N(0,0.02) weights, prompt ids uniform over the vocabulary", "size": z,
+            "peaks": "of " + pk["source"], "l2": "whole models: weights and cache exceed L2; kernels alone: L2 flushed "
+            "before every repetition"}
+    ctx = args.ctx or 2048
+    for name, cfg in (("zuzupel", zuzupel_config(z)), ("favudra_twin", zuzupel_twin(z))):
+        model = Model.random(cfg, seed=0, dtype="bfloat16", device="cuda:0", fast=True)
+        with ClockSampler() as clocks:
+            ms, launches = run_decode(model, args.batch, ctx, args.steps, max(3, args.warmup), args.page)
+        pms = run_prefill(model, 2048, reps=5, warmup=3, page=args.page)
+        line[name] = {"decode_tok_s": round(args.batch / (ms / 1e3), 1), "decode_ms_per_step": round(ms, 4),
+                      "prefill_tok_s": round(2048 / (pms / 1e3), 1), "prefill_ms": round(pms, 3),
+                      "weight_bytes": model.weight_bytes, "gpu_launches": launches, "clocks": clocks.summary()}
+        del model
+        torch.cuda.empty_cache()
+    line["kernels"] = zuzupel_kernel_table(z, pk, args.page)
+    return line
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1107,9 +1322,10 @@ def main():
     ap.add_argument("--page", type=int, default=16)
     ap.add_argument("--skip-points", action="store_true", help="only the headline decode (for profiling runs)")
     ap.add_argument("--skip-prefill", action="store_true")
-    ap.add_argument("--compare", default="", choices=["", "nuderax", "favudra", "sebavik", "kezuvik"],
+    ap.add_argument("--compare", default="", choices=["", "nuderax", "favudra", "sebavik", "kezuvik", "zuzupel"],
                     help="instead of the headline: this design beside its closest earlier architecture at equal size")
-    ap.add_argument("--size", default="small", choices=sorted(set(NUDERAX_SIZES) | set(FAVUDRA_SIZES) | set(SEBAVIK_SIZES) | set(KEZUVIK_SIZES)),
+    ap.add_argument("--size", default="small", choices=sorted(set(NUDERAX_SIZES) | set(FAVUDRA_SIZES) | set(SEBAVIK_SIZES) | set(KEZUVIK_SIZES) |
+                                                                set(ZUZUPEL_SIZES)),
                     help="layer sizes for --compare")
     args = ap.parse_args()
 
@@ -1132,6 +1348,9 @@ def main():
         return 0
     if args.compare == "kezuvik":
         print(json.dumps(compare_kezuvik(args, pk)))
+        return 0
+    if args.compare == "zuzupel":
+        print(json.dumps(compare_zuzupel(args, pk)))
         return 0
     if args.compare == "sebavik":
         print(json.dumps(compare_sebavik(args, pk)))

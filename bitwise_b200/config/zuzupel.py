@@ -106,15 +106,15 @@ class ChunkAttentionConfig:
         _whole_groups(heads, kv_heads, where)
         rot, mask = d.get("rot"), d.get("mask")
         base = dims = factor = None
-        if rot:
+        if rot is not None:
             base = _positive(_get(rot, "base", where + ".rot"), where + ".rot.base")
             dims = _int_of(rot, "dims", where + ".rot")
             if dims > dim or dims % 2:
                 raise ConfigError(f"config.json: {where}.rot.dims = {dims} must be even and at most dim = {dim}")
-            if rot.get("scaling"):
+            if rot.get("scaling") is not None:
                 factor = _positive(_get(rot["scaling"], "factor", where + ".rot.scaling"), where + ".rot.scaling.factor")
         return ChunkAttentionConfig(heads, kv_heads, dim, vdim, float(_get(d, "scale", where)), base, dims, factor,
-                                    _int_of(mask, "size", where + ".mask") if mask else None)
+                                    _int_of(mask, "size", where + ".mask") if mask is not None else None)
 
     def to_json(self) -> dict:
         d = {"dim": self.dim, "heads": self.heads, "kv_heads": self.kv_heads, "scale": self.scale, "vdim": self.vdim}

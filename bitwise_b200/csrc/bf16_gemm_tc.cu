@@ -665,9 +665,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         }
         continue;
       }
-      if (EPI == 0 && !GROUPED && y_is_f32) {
+      if (EPI == 0 && !GROUPED && y_is_f32 == 2 * bw::kOutRelu2) {
 #pragma unroll
-        for (int j = 0; j < 2 * PW; ++j) total[j] = bw::out_act(total[j], y_is_f32 >> 1);
+        for (int j = 0; j < 2 * PW; ++j) total[j] = bw::out_act(total[j], bw::kOutRelu2);
+      } else if (EPI == 0 && !GROUPED && y_is_f32 == 2 * bw::kOutTanh) {
+#pragma unroll
+        for (int j = 0; j < 2 * PW; ++j) total[j] = bw::out_act(total[j], bw::kOutTanh);
       }
 #pragma unroll
       for (int piece = 0; piece < 2; ++piece) {

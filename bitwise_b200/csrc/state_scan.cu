@@ -2,16 +2,17 @@
 // kernel, what prepares their operands, and what finishes their outputs. Per head the state S is
 // dim x vdim float32 numbers of a request (zero before its first token):
 //
-//   delta    S <- g S (g per key channel), then S <- S + k (beta (v - S^T k))^T, then o = S^T q
+//   delta    S <- g S (g per key channel), then S <- S + k u^T with u = beta (v - S^T k), then o = S^T q; the last
+//            two as o = (g S)^T q + (q . k) u, so that both sums over g S are formed together
 //   bonus    o = (S + diag(u) k v^T)^T q, then S <- diag(w) S + k v^T, w = exp(-exp(z + z0))
 //   memory   m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, the normaliser n alike with
 //            k alone, o = S^T q (divided later by max(|n . q|, e^-m) + 1e-6)
 //
 // The columns of S (one per value channel) do not meet inside a token, so a block walks the rows of one
 // sequence of the step for one head and a few columns, from the state that the request's slot holds.
-// LP lanes of a warp share a column; a lane holds V groups of four consecutive rows (group p + LP i).
-// A sum over a column's rows is a chain per lane and a butterfly over the LP lanes, in an order given
-// by dim alone. The tokens' operands are copied into shared memory a chunk ahead (cp.async, two buffers);
+// LP lanes of a warp share two neighbouring columns (what a lane reads of a token then serves both); a
+// lane holds V groups of four consecutive rows (group p + LP i). A sum over a column's rows is four chains
+// per lane and a butterfly over the LP lanes, in an order given by dim alone. The tokens' operands are copied into shared memory a chunk ahead (cp.async, two buffers);
 // the chunk is a staging unit only: every S and o is the same chain of operations wherever the step's
 // rows begin and end, so a position's result does not depend on how its prompt was cut.
 // Everything here is float32 in both precisions; only what enters the next product changes type.
@@ -23,6 +24,8 @@
 namespace {
 
 constexpr int kThreads = 128;
+constexpr int kWarps = kThreads / 32;
+constexpr int kCols = 2;  // columns of a lane
 enum { kDelta = 0, kBonus = 1, kMemory = 2 };
 
 // The serving precision takes the hardware's exponential (relative error about 1e-7 times the exponent's size, far
@@ -56,7 +59,7 @@ struct ScanArgs {
   const float* decay_bias;  // bonus: z0 [heads * dim]
   const float* bonus;      // bonus: u [heads * dim]
   const float* s0;         // delta: beta; memory: the forget gate's projection. Row r, head h: s0 + r * s_stride + h
-  const float* s1;         // memory: the input gate's projection
+  const float* s1;         // delta: q . k, one per query head (h / rep); memory: the input gate's projection, one per head
   int s_stride;
   const float* s0_bias;    // memory: [heads]
   const float* s1_bias;
@@ -101,7 +104,7 @@ __device__ __forceinline__ float column_sum(float x) {
 
 template <int MODE, int LP, int V>
 struct Shape {
-  static constexpr int CB = kThreads / LP;   // columns of a block
+  static constexpr int CB = kThreads / LP * kCols;  // columns of a block
   static constexpr int DP = LP * 4 * V;      // rows held; those from dim on are zero
   static constexpr int VECS = MODE == kMemory ? 2 : 3;
   static constexpr int SC = VECS * DP + CB;  // where a token's scalars start
@@ -123,17 +126,23 @@ __device__ __forceinline__ Rows<V> load_rows(const float* at, int p) {
   }
   return r;
 }
-// Two chains (even and odd entries) and their sum.
+// Four chains (the entries of equal place in the groups of four) and their sum.
 template <int V>
 __device__ __forceinline__ float dot(const Rows<V>& a, const Rows<V>& b) {
-  float e = 0.0f, o = 0.0f;
+  float s[4];
 #pragma unroll
-  for (int i = 0; i < 4 * V; i += 2) {
-    e = __fmaf_rn(a.v[i], b.v[i], e);
-    o = __fmaf_rn(a.v[i + 1], b.v[i + 1], o);
-  }
-  return __fadd_rn(e, o);
+  for (int e = 0; e < 4; ++e) s[e] = __fmul_rn(a.v[e], b.v[e]);
+#pragma unroll
+  for (int i = 4; i < 4 * V; ++i) s[i & 3] = __fmaf_rn(a.v[i], b.v[i], s[i & 3]);
+  return __fadd_rn(__fadd_rn(s[0], s[1]), __fadd_rn(s[2], s[3]));
 }
+// What a lane reads of a staged token.
+template <int V>
+struct Token {
+  Rows<V> k, q, d;
+  float v[kCols];
+  float s0, s1;
+};
 
 template <int MODE, int LP, int V>
 __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) {
@@ -147,30 +156,33 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
   const int t = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * T::CB;
   const int seq = a.tile_seq[t], row0 = a.tile_row0[t], cnt = a.tile_rows[t];
   const int tid = threadIdx.x;
-  const int p = tid & (LP - 1), c = c0 + tid / LP;
+  const int p = tid & (LP - 1), col = tid / LP * kCols;  // this lane's rows and its first column in the block
   constexpr bool kMem = MODE == kMemory;
   const int cols = kMem ? vdim + 1 : vdim, col_size = kMem ? dim + 4 : dim;
-  const bool col_ok = c < cols;
   float* head_state = a.state + (static_cast<size_t>(a.seq_slot[seq]) * a.heads + h) * cols * col_size;
-  float* sp = head_state + static_cast<size_t>(c) * col_size;
+  float* sp = head_state + static_cast<size_t>(c0 + col) * col_size;
   const bool fresh = a.seq_pos0[seq] == 0;      // a slot is handed out as its last holder left it
   // The state of this run was written by the step before, so it is asked for before the wait for this step's kernels.
-  Rows<V> S;
+  Rows<V> S[kCols];
 #pragma unroll
-  for (int i = 0; i < V; ++i) {
-    const int row = 4 * (p + LP * i);
-    float4 f = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    if (!fresh && col_ok) {
-      if (a.wide) {
-        if (row < dim) f = *reinterpret_cast<const float4*>(sp + row);
-      } else {
-        if (row < dim) f.x = sp[row];
-        if (row + 1 < dim) f.y = sp[row + 1];
-        if (row + 2 < dim) f.z = sp[row + 2];
-        if (row + 3 < dim) f.w = sp[row + 3];
+  for (int j = 0; j < kCols; ++j) {
+    const float* from = sp + j * col_size;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const int row = 4 * (p + LP * i);
+      float4 f = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (!fresh && c0 + col + j < cols) {
+        if (a.wide) {
+          if (row < dim) f = *reinterpret_cast<const float4*>(from + row);
+        } else {
+          if (row < dim) f.x = from[row];
+          if (row + 1 < dim) f.y = from[row + 1];
+          if (row + 2 < dim) f.z = from[row + 2];
+          if (row + 3 < dim) f.w = from[row + 3];
+        }
       }
+      S[j].v[4 * i] = f.x, S[j].v[4 * i + 1] = f.y, S[j].v[4 * i + 2] = f.z, S[j].v[4 * i + 3] = f.w;
     }
-    S.v[4 * i] = f.x, S.v[4 * i + 1] = f.y, S.v[4 * i + 2] = f.z, S.v[4 * i + 3] = f.w;
   }
   float m = 0.0f;  // memory: the running maximum (held by every thread of warp 0)
   if (kMem && !fresh) m = head_state[static_cast<size_t>(c0) * col_size + dim];
@@ -184,91 +196,117 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
         bonus.v[4 * i + e] = row < dim ? a.bonus[h * dim + row] : 0.0f;
       }
   }
-  for (int i = tid; i < 2 * chunk * T::W; i += kThreads) stage[i] = 0.0f;  // rows from dim on stay zero
+  if (dim < T::DP)  // rows from dim on stay zero
+    for (int i = tid; i < 2 * chunk * T::W; i += kThreads) stage[i] = 0.0f;
   bw::pdl_wait();
   if (!few) bw::pdl_launch();
   __syncthreads();
   const int kh = h / a.rep;
+  const int warp = tid >> 5, lane = tid & 31;
+  // where entry e of a staged token's vectors and values comes from: its address in row 0 and the distance between rows
+  auto source = [&](int e, int& stride) -> const float* {
+    if (e < T::VECS * T::DP) {
+      const int d = e % T::DP;
+      if (d >= dim) return nullptr;
+      if (e < T::DP) return stride = a.k_stride, a.k + kh * dim + d;
+      if (e < 2 * T::DP) return stride = a.q_stride, a.q + kh * dim + d;
+      return stride = a.decay_stride, a.decay + h * dim + d;
+    }
+    const int cc = c0 + e - T::VECS * T::DP;
+    if (e >= T::SC || cc >= vdim) return nullptr;
+    return stride = a.v_stride, a.v + h * vdim + cc;
+  };
+  // A warp copies every fourth token, a lane the same 16-byte pieces of each: addresses only move on by rows.
+  constexpr int NP = (T::SC / 4 + 31) / 32;
+  const float* piece[NP];
+  int step[NP];
+  if (a.wide) {
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      step[i] = 0;
+      piece[i] = source(4 * (lane + 32 * i), step[i]);
+      if (piece[i]) piece[i] += static_cast<size_t>(row0 + warp) * step[i];
+      step[i] *= kWarps;
+    }
+  }
   auto request = [&](int first, float* buf) {
     const int len = min(chunk, cnt - first);
     if (a.wide) {
-      constexpr int Ws = T::SC / 4;
-      for (int i = tid; i < len * Ws; i += kThreads) {
-        const int tt = i / Ws, e = (i - tt * Ws) * 4;
-        const size_t r = static_cast<size_t>(row0 + first + tt);
-        const float* src;
-        if (e < T::VECS * T::DP) {
-          const int d = e % T::DP;
-          if (d >= dim) continue;
-          if (e < T::DP) src = a.k + r * a.k_stride + kh * dim + d;
-          else if (e < 2 * T::DP) src = a.q + r * a.q_stride + kh * dim + d;
-          else src = a.decay + r * a.decay_stride + h * dim + d;
-        } else {
-          const int cc = c0 + e - T::VECS * T::DP;
-          if (cc >= vdim) continue;
-          src = a.v + r * a.v_stride + h * vdim + cc;
-        }
-        copy16_async(buf + tt * T::W + e, src);
+      for (int tt = warp; tt < len; tt += kWarps) {
+        float* dst = buf + tt * T::W + 4 * lane;
+#pragma unroll
+        for (int i = 0; i < NP; ++i)
+          if (piece[i]) copy16_async(dst + 128 * i, piece[i]), piece[i] += step[i];
       }
     } else {
-      constexpr int Ws = T::SC;
-      for (int i = tid; i < len * Ws; i += kThreads) {
-        const int tt = i / Ws, e = i - tt * Ws;
-        const size_t r = static_cast<size_t>(row0 + first + tt);
-        const float* src;
-        if (e < T::VECS * T::DP) {
-          const int d = e % T::DP;
-          if (d >= dim) continue;
-          if (e < T::DP) src = a.k + r * a.k_stride + kh * dim + d;
-          else if (e < 2 * T::DP) src = a.q + r * a.q_stride + kh * dim + d;
-          else src = a.decay + r * a.decay_stride + h * dim + d;
-        } else {
-          const int cc = c0 + e - T::VECS * T::DP;
-          if (cc >= vdim) continue;
-          src = a.v + r * a.v_stride + h * vdim + cc;
-        }
-        copy4_async(buf + tt * T::W + e, src);
+      for (int i = tid; i < len * T::SC; i += kThreads) {
+        const int tt = i / T::SC, e = i - tt * T::SC;
+        int stride = 0;
+        const float* src = source(e, stride);
+        if (src) copy4_async(buf + tt * T::W + e, src + static_cast<size_t>(row0 + first + tt) * stride);
       }
     }
     if (MODE != kBonus) {
       for (int tt = tid; tt < len; tt += kThreads) {
         const size_t r = static_cast<size_t>(row0 + first + tt);
         copy4_async(buf + tt * T::W + T::SC, a.s0 + r * a.s_stride + h);
-        if (kMem) copy4_async(buf + tt * T::W + T::SC + 1, a.s1 + r * a.s_stride + h);
+        copy4_async(buf + tt * T::W + T::SC + 1, a.s1 + r * a.s_stride + (kMem ? h : kh));
       }
     }
     bw::copies_commit();
   };
-  // One token: S moves on; returns this lane's share of the output.
-  auto token = [&](const float* tok) -> float {
-    const Rows<V> k = load_rows<LP, V>(tok, p), q = load_rows<LP, V>(tok + T::DP, p);
-    const float* vals = tok + T::VECS * T::DP;
-    float v = vals[tid / LP];
+  auto load = [&](const float* tok) -> Token<V> {
+    Token<V> x;
+    x.k = load_rows<LP, V>(tok, p), x.q = load_rows<LP, V>(tok + T::DP, p);
+    if (!kMem) x.d = load_rows<LP, V>(tok + 2 * T::DP, p);
+#pragma unroll
+    for (int j = 0; j < kCols; ++j) x.v[j] = tok[T::VECS * T::DP + col + j];
+    x.s0 = MODE == kBonus ? 0.0f : tok[T::SC], x.s1 = MODE == kBonus ? 0.0f : tok[T::SC + 1];
+    return x;
+  };
+  // One token: S moves on; this lane's share of both columns' outputs into o (delta: one column's whole output, see below).
+  auto move = [&](const Token<V>& x, float (&o)[kCols]) {
     if (MODE == kDelta) {
-      const Rows<V> g = load_rows<LP, V>(tok + 2 * T::DP, p);
-      const float beta = tok[T::SC];
+      // All four sums (of k and of q, both columns) in one butterfly: lane p ends up with the sum p / (LP / 4).
+      float d[2 * kCols];
 #pragma unroll
-      for (int i = 0; i < 4 * V; ++i) S.v[i] = __fmul_rn(g.v[i], S.v[i]);
-      const float u = __fmul_rn(beta, __fsub_rn(v, column_sum<LP>(dot<V>(k, S))));
+      for (int j = 0; j < kCols; ++j) {
 #pragma unroll
-      for (int i = 0; i < 4 * V; ++i) S.v[i] = __fmaf_rn(k.v[i], u, S.v[i]);
-      return dot<V>(q, S);
-    } else if (MODE == kBonus) {
-      const Rows<V> w = load_rows<LP, V>(tok + 2 * T::DP, p);
-      Rows<V> seen;
-#pragma unroll
-      for (int i = 0; i < 4 * V; ++i) {
-        const float kv = __fmul_rn(k.v[i], v);
-        seen.v[i] = __fmaf_rn(bonus.v[i], kv, S.v[i]);
-        S.v[i] = __fmaf_rn(w.v[i], S.v[i], kv);
+        for (int i = 0; i < 4 * V; ++i) S[j].v[i] = __fmul_rn(x.d.v[i], S[j].v[i]);
+        d[j] = dot<V>(x.k, S[j]);
+        d[kCols + j] = dot<V>(x.q, S[j]);
       }
-      return dot<V>(q, seen);
-    } else {
-      if (c == vdim) v = 1.0f;  // the normaliser's column
-      const float keep = tok[T::SC], add = __fmul_rn(tok[T::SC + 1], v);
+      const float sum = group_sum<LP, 2 * kCols>(d, p);
+      const float mine = __fmul_rn(x.s0, __fsub_rn((p & (LP / 4)) ? x.v[1] : x.v[0], sum));
+      const int base = lane & ~(LP - 1);
+      float u[kCols];
 #pragma unroll
-      for (int i = 0; i < 4 * V; ++i) S.v[i] = __fmaf_rn(k.v[i], add, __fmul_rn(keep, S.v[i]));
-      return dot<V>(q, S);
+      for (int j = 0; j < kCols; ++j) u[j] = __shfl_sync(0xffffffffu, mine, base + j * (LP / 4));
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) {
+#pragma unroll
+        for (int i = 0; i < 4 * V; ++i) S[j].v[i] = __fmaf_rn(x.k.v[i], u[j], S[j].v[i]);
+      }
+      o[0] = __fmaf_rn(x.s1, (p & (LP / 4)) ? u[1] : u[0], sum);  // in the lanes of q's sums: a column's output
+    } else {
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) {
+        if (MODE == kBonus) {
+          Rows<V> seen;
+#pragma unroll
+          for (int i = 0; i < 4 * V; ++i) {
+            const float kv = __fmul_rn(x.k.v[i], x.v[j]);
+            seen.v[i] = __fmaf_rn(bonus.v[i], kv, S[j].v[i]);
+            S[j].v[i] = __fmaf_rn(x.d.v[i], S[j].v[i], kv);
+          }
+          o[j] = dot<V>(x.q, seen);
+        } else {
+          const float add = __fmul_rn(x.s1, c0 + col + j == vdim ? 1.0f : x.v[j]);  // (the normaliser's column takes ones)
+#pragma unroll
+          for (int i = 0; i < 4 * V; ++i) S[j].v[i] = __fmaf_rn(x.k.v[i], add, __fmul_rn(x.s0, S[j].v[i]));
+          o[j] = dot<V>(x.q, S[j]);
+        }
+      }
     }
   };
   request(0, stage);
@@ -284,11 +322,12 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
     }
     __syncthreads();
     if (MODE == kBonus) {
-      for (int i = tid; i < len * T::DP; i += kThreads) {
-        const int tt = i / T::DP, d = i % T::DP;
-        if (d >= dim) continue;
-        float* at = buf + tt * T::W + 2 * T::DP + d;
-        *at = exp_f(-exp_f(__fadd_rn(*at, a.decay_bias[h * dim + d])));
+      constexpr int kTokens = T::DP < kThreads ? kThreads / T::DP : 1;  // tokens that the block's threads cover at a time
+      for (int d = tid % T::DP; d < dim; d += kThreads) {
+        const float bias = a.decay_bias[h * dim + d];
+        float* at = buf + tid / T::DP * T::W + 2 * T::DP + d;
+        for (int tt = tid / T::DP; tt < len; tt += kTokens, at += kTokens * T::W)
+          *at = exp_f(-exp_f(__fadd_rn(*at, bias)));
       }
       __syncthreads();
     }
@@ -321,20 +360,52 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
       __syncthreads();
     }
     int tt = 0;
+    if (MODE == kDelta) {
+      // lane p = LP / 2 holds the first column's output, lane p = LP / 2 + LP / 4 the second's
+      float* to = outs + col + ((p & (LP / 4)) ? 1 : 0);
+      const bool stores = p == LP / 2 || p == LP / 2 + LP / 4;
+      Token<V> x = load(buf);
+#pragma unroll 4
+      for (; tt < len; ++tt) {  // the next token's operands are asked for before this one's are used
+        const Token<V> y = load(buf + min(tt + 1, len - 1) * T::W);
+        float o[kCols];
+        move(x, o);
+        if (stores) to[tt * T::CB] = o[0];
+        x = y;
+      }
+    }
     for (; tt + T::G <= len; tt += T::G) {
-      float part[T::G];
+      float part[kCols][T::G];
+      const float* tok = buf + tt * T::W;
+      Token<V> x = load(tok);
 #pragma unroll
-      for (int j = 0; j < T::G; ++j) part[j] = token(buf + (tt + j) * T::W);
-      const float s = group_sum<LP, T::G>(part, p);
-      if (p % (LP / T::G) == 0) outs[(tt + p / (LP / T::G)) * T::CB + tid / LP] = s;
+      for (int i = 0; i < T::G; ++i) {  // the next token's operands are asked for before this one's are used
+        const Token<V> y = load(tok + min(i + 1, T::G - 1) * T::W);
+        float o[kCols];
+        move(x, o);
+#pragma unroll
+        for (int j = 0; j < kCols; ++j) part[j][i] = o[j];
+        x = y;
+      }
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) {
+        const float s = group_sum<LP, T::G>(part[j], p);
+        if (p % (LP / T::G) == 0) outs[(tt + p / (LP / T::G)) * T::CB + col + j] = s;
+      }
     }
     for (; tt < len; ++tt) {
-      const float s = column_sum<LP>(token(buf + tt * T::W));
-      if (p == 0) outs[tt * T::CB + tid / LP] = s;
+      float o[kCols];
+      move(load(buf + tt * T::W), o);
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) {
+        const float s = column_sum<LP>(o[j]);
+        if (p == 0) outs[tt * T::CB + col + j] = s;
+      }
     }
     __syncthreads();
+    const int cc = c0 + tid % T::CB;
     for (int i = tid; i < len * T::CB; i += kThreads) {
-      const int ti = i / T::CB, cc = c0 + i % T::CB;
+      const int ti = i / T::CB;
       const size_t r = static_cast<size_t>(row0 + first + ti);
       if (cc < vdim) {
         a.o[r * a.heads * vdim + h * vdim + cc] = outs[i];
@@ -344,22 +415,27 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
       }
     }
   }
-  if (!col_ok) return;
 #pragma unroll
-  for (int i = 0; i < V; ++i) {
-    const int row = 4 * (p + LP * i);
-    if (a.wide) {
-      if (row < dim) *reinterpret_cast<float4*>(sp + row) = make_float4(S.v[4 * i], S.v[4 * i + 1], S.v[4 * i + 2], S.v[4 * i + 3]);
-    } else {
+  for (int j = 0; j < kCols; ++j) {
+    if (c0 + col + j >= cols) continue;
+    float* to = sp + j * col_size;
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (row + e < dim) sp[row + e] = S.v[4 * i + e];
+    for (int i = 0; i < V; ++i) {
+      const int row = 4 * (p + LP * i);
+      if (a.wide) {
+        if (row < dim)
+          *reinterpret_cast<float4*>(to + row) = make_float4(S[j].v[4 * i], S[j].v[4 * i + 1], S[j].v[4 * i + 2], S[j].v[4 * i + 3]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (row + e < dim) to[row + e] = S[j].v[4 * i + e];
+      }
     }
-  }
-  // every column keeps the maximum of its own: the blocks of a head do not read what another one writes
-  if (kMem && p == 0) {
-    const int last = (cnt - 1) / chunk, slot = (cnt - 1) - last * chunk;
-    sp[dim] = stage[(last & 1) * chunk * T::W + slot * T::W + T::SC + 2];
+    // every column keeps the maximum of its own: the blocks of a head do not read what another one writes
+    if (kMem && p == 0) {
+      const int last = (cnt - 1) / chunk, slot = (cnt - 1) - last * chunk;
+      to[dim] = stage[(last & 1) * chunk * T::W + slot * T::W + T::SC + 2];
+    }
   }
 }
 
@@ -422,10 +498,10 @@ __global__ void __launch_bounds__(kThreads) scan_finish_kernel(const FinishArgs 
 }
 
 // ---------------------------------------------------------------------------------------
-// What the delta recurrence reads: per row, a warp per head. q, k and v pass a causal convolution over time on
+// What the delta recurrence reads, row by row. q, k and v pass a causal convolution over time on
 // every channel (inputs before the step's first row of a sequence from the request's state, zeros before position 0)
 // and SiLU; q and k become unit vectors, q times a scale; the decays g = exp(-exp(A_h) softplus(z + bias)) replace z;
-// beta = sigmoid(b). With `keep` (steps of one row per sequence) the state is brought up to date here as well.
+// beta = sigmoid(b); q . k per query head. With `keep` (steps of one row per sequence) the state is brought up to date here as well.
 struct DeltaPrepArgs {
   const float* u;         // [n, u_stride]: q heads | k heads | v heads, beta's projections from beta_col on
   int u_stride, beta_col;
@@ -437,7 +513,7 @@ struct DeltaPrepArgs {
   int z_stride;
   const float* dt_bias;   // [heads * dim]
   const float* a_log;     // [heads]
-  float* out;             // [n, out_stride]: q | k | v | beta
+  float* out;             // [n, out_stride]: q | k | v | beta | q . k (one per query head)
   int out_stride;
   const int* pos;
   const int* row_seq;
@@ -449,61 +525,106 @@ struct DeltaPrepArgs {
 
 constexpr int kMaxPer = 16;  // entries of a head per lane: sizes up to 512
 
+// The convolution over time and SiLU of one head (`size` channels from col0 on) into the lane's registers: with VEC 4 four
+// neighbouring channels at a time (128 to a warp), else channels 32 apart. The order of a channel's sum is the taps', either way.
+template <int VEC>
+__device__ __forceinline__ void conv_head(const DeltaPrepArgs& a, int r, int p, int row0, float* st, int channels, int lane, int col0,
+                                          int size, float (&val)[kMaxPer]) {
+  constexpr int NG = kMaxPer / VEC;
+#pragma unroll
+  for (int j = 0; j < kMaxPer; ++j) val[j] = 0.0f;
+  const float* u = a.u + static_cast<size_t>(r) * a.u_stride + col0;
+  for (int t = 0; t < a.taps; ++t) {  // taps ascending
+    const int back = a.taps - 1 - t;
+    if (p - back < 0) continue;
+    const float* src = r - back >= row0 ? u - static_cast<ptrdiff_t>(back) * a.u_stride
+                                        : st + static_cast<size_t>(a.taps - 1 - (row0 - (r - back))) * channels + col0;
+    const float* w = a.conv_t + static_cast<size_t>(t) * channels + col0;
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int e = VEC * (lane + 32 * g);
+      if (e >= size) continue;
+      if (VEC == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(src + e), c = *reinterpret_cast<const float4*>(w + e);
+        val[4 * g] = __fmaf_rn(c.x, x.x, val[4 * g]), val[4 * g + 1] = __fmaf_rn(c.y, x.y, val[4 * g + 1]);
+        val[4 * g + 2] = __fmaf_rn(c.z, x.z, val[4 * g + 2]), val[4 * g + 3] = __fmaf_rn(c.w, x.w, val[4 * g + 3]);
+      } else {
+        val[g] = __fmaf_rn(w[e], src[e], val[g]);
+      }
+    }
+  }
+  if (a.keep && st) {  // the sequence's only row: the inputs move up by one
+#pragma unroll
+    for (int j = 0; j < kMaxPer; ++j) {
+      const int e = VEC * (lane + 32 * (j / VEC)) + j % VEC;
+      if (e >= size) continue;
+      float* at = st + col0 + e;
+      for (int t = 0; t + 1 < a.taps - 1; ++t)
+        at[static_cast<size_t>(t) * channels] = p - (a.taps - 2 - t) >= 0 ? at[static_cast<size_t>(t + 1) * channels] : 0.0f;
+      at[static_cast<size_t>(a.taps - 2) * channels] = u[e];
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < kMaxPer; ++j) val[j] = __fmul_rn(val[j], sigmoid_f(val[j]));
+}
+
+template <int VEC>
+__device__ __forceinline__ void store_head(float* out, int lane, int size, const float (&val)[kMaxPer], float f) {
+#pragma unroll
+  for (int g = 0; g < kMaxPer / VEC; ++g) {
+    const int e = VEC * (lane + 32 * g);
+    if (e >= size) continue;
+    if (VEC == 4)
+      *reinterpret_cast<float4*>(out + e) = make_float4(__fmul_rn(val[4 * g], f), __fmul_rn(val[4 * g + 1], f),
+                                                        __fmul_rn(val[4 * g + 2], f), __fmul_rn(val[4 * g + 3], f));
+    else
+      out[e] = __fmul_rn(val[g], f);
+  }
+}
+
+// A warp per query/key head (both), value head, head of decays; the last one forms beta.
+template <int VEC>
 __global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const DeltaPrepArgs a) {
   bw::pdl_enter();
   const int r = blockIdx.x;
   const int lane = threadIdx.x & 31;
-  const int unit = blockIdx.y * (kThreads / 32) + (threadIdx.x >> 5);
-  const int qk = 2 * a.kv_heads, convs = qk + a.heads;
+  int unit = blockIdx.y * kWarps + (threadIdx.x >> 5);
+  const int G = a.kv_heads, channels = 2 * G * a.dim + a.heads * a.vdim;
   float* out = a.out + static_cast<size_t>(r) * a.out_stride;
-  const int channels = qk * a.dim + a.heads * a.vdim;
-  if (unit < convs) {
-    const int size = unit < qk ? a.dim : a.vdim;
-    const int col0 = unit < qk ? unit * a.dim : qk * a.dim + (unit - qk) * a.vdim;
+  if (unit < G + a.heads) {
     const int p = a.pos[r], seq = a.row_seq[r], row0 = a.seq_row0[seq];
     float* st = a.conv_state ? a.conv_state + static_cast<size_t>(a.seq_slot[seq]) * (a.taps - 1) * channels : nullptr;
-    const float* u = a.u + static_cast<size_t>(r) * a.u_stride;
     float val[kMaxPer];
-    float ss = 0.0f;
+    if (unit >= G) {
+      const int col0 = 2 * G * a.dim + (unit - G) * a.vdim;
+      conv_head<VEC>(a, r, p, row0, st, channels, lane, col0, a.vdim, val);
+      store_head<VEC>(out + col0, lane, a.vdim, val, 1.0f);
+      return;
+    }
+    float other[kMaxPer];
+    conv_head<VEC>(a, r, p, row0, st, channels, lane, unit * a.dim, a.dim, val);
+    conv_head<VEC>(a, r, p, row0, st, channels, lane, (G + unit) * a.dim, a.dim, other);
+    float qq = 0.0f, kk = 0.0f;  // (entries beyond the head are zero)
 #pragma unroll
-    for (int j = 0; j < kMaxPer; ++j) {
-      const int e = lane + 32 * j;
-      float y = 0.0f;
-      if (e < size) {
-        const int c = col0 + e;
-        for (int t = 0; t < a.taps; ++t) {  // taps ascending
-          const int back = a.taps - 1 - t;
-          if (p - back < 0) continue;
-          const float x = r - back >= row0 ? u[c - static_cast<ptrdiff_t>(back) * a.u_stride]
-                                           : st[static_cast<size_t>(a.taps - 1 - (row0 - (r - back))) * channels + c];
-          y = __fmaf_rn(a.conv_t[static_cast<size_t>(t) * channels + c], x, y);
-        }
-        if (a.keep && st) {  // the sequence's only row: the inputs move up by one
-          for (int t = 0; t + 1 < a.taps - 1; ++t)
-            st[static_cast<size_t>(t) * channels + c] = p - (a.taps - 2 - t) >= 0 ? st[static_cast<size_t>(t + 1) * channels + c] : 0.0f;
-          st[static_cast<size_t>(a.taps - 2) * channels + c] = u[c];
-        }
-        y = __fmul_rn(y, sigmoid_f(y));
-        ss = __fmaf_rn(y, y, ss);
-      }
-      val[j] = y;
-    }
-    float f = 1.0f;
-    if (unit < qk) {
-      f = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(bw::warp_sum(ss), 1e-6f)));
-      if (unit < a.kv_heads) f = __fmul_rn(f, a.q_scale);
-    }
+    for (int j = 0; j < kMaxPer; ++j) qq = __fmaf_rn(val[j], val[j], qq), kk = __fmaf_rn(other[j], other[j], kk);
+    const float fq = __fmul_rn(__fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(bw::warp_sum(qq), 1e-6f))), a.q_scale);
+    const float fk = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(bw::warp_sum(kk), 1e-6f)));
+    float qk = 0.0f;
 #pragma unroll
-    for (int j = 0; j < kMaxPer; ++j) {
-      const int e = lane + 32 * j;
-      if (e < size) out[col0 + e] = __fmul_rn(val[j], f);
-    }
-  } else if (unit < convs + a.heads) {
-    const int h = unit - convs;
-    const float rate = expf(a.a_log[h]);
-    float* z = a.z + static_cast<size_t>(r) * a.z_stride + h * a.dim;
-    for (int d = lane; d < a.dim; d += 32) z[d] = expf(-__fmul_rn(rate, softplus_f(__fadd_rn(z[d], a.dt_bias[h * a.dim + d]))));
-  } else if (unit == convs + a.heads) {
+    for (int j = 0; j < kMaxPer; ++j) qk = __fmaf_rn(__fmul_rn(val[j], fq), __fmul_rn(other[j], fk), qk);
+    qk = bw::warp_sum(qk);
+    store_head<VEC>(out + unit * a.dim, lane, a.dim, val, fq);
+    store_head<VEC>(out + (G + unit) * a.dim, lane, a.dim, other, fk);
+    if (lane == 0) out[channels + a.heads + unit] = qk;
+    return;
+  }
+  unit -= G + a.heads;
+  if (unit < a.heads) {
+    const float rate = expf(a.a_log[unit]);
+    float* z = a.z + static_cast<size_t>(r) * a.z_stride + unit * a.dim;
+    const float* bias = a.dt_bias + unit * a.dim;
+    for (int d = lane; d < a.dim; d += 32) z[d] = exp_f(-__fmul_rn(rate, softplus_f(__fadd_rn(z[d], bias[d]))));
+  } else if (unit == a.heads) {
     for (int h = lane; h < a.heads; h += 32) out[channels + h] = sigmoid_f(a.u[static_cast<size_t>(r) * a.u_stride + a.beta_col + h]);
   }
 }
@@ -578,11 +699,12 @@ template <int MODE, int LP, int V>
 int launch_scan(ScanArgs a, int tiles, int longest, cudaStream_t stream) {
   typedef Shape<MODE, LP, V> T;
   // Tokens staged at a time: no more than the longest sequence of the step can have (a step of single rows stages
-  // one, so that many of its small blocks share an SM), at most 16, and no more than 100 KB.
+  // one, so that many of its small blocks share an SM), at most 32 (a chunk is a multiple of the warps beyond that), and no more
+  // than two blocks of an SM have room for.
   a.chunk = 1;
-  while (a.chunk < 16 && a.chunk < longest) a.chunk *= 2;
+  while (a.chunk < 32 && a.chunk < longest) a.chunk *= 2;
   auto bytes = [](int chunk) { return static_cast<size_t>(2 * chunk * T::W + chunk * T::CB) * sizeof(float); };
-  while (a.chunk > 1 && bytes(a.chunk) > 100 * 1024) a.chunk /= 2;
+  while (a.chunk > kWarps && bytes(a.chunk) > 108 * 1024) a.chunk /= 2;
   const size_t smem = bytes(a.chunk);
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
@@ -601,8 +723,8 @@ int launch_scan(ScanArgs a, int tiles, int longest, cudaStream_t stream) {
 template <int MODE>
 int launch_mode(const ScanArgs& a, int tiles, int longest, cudaStream_t stream) {
   if (a.dim <= 16) return launch_scan<MODE, 4, 1>(a, tiles, longest, stream);
-  if (a.dim <= 32) return launch_scan<MODE, 4, 2>(a, tiles, longest, stream);
-  if (a.dim <= 64) return launch_scan<MODE, 8, 2>(a, tiles, longest, stream);
+  if (a.dim <= 32) return launch_scan<MODE, 8, 1>(a, tiles, longest, stream);
+  if (a.dim <= 64) return launch_scan<MODE, 16, 1>(a, tiles, longest, stream);
   if (a.dim <= 128) return launch_scan<MODE, 16, 2>(a, tiles, longest, stream);
   if (a.dim <= 256) return launch_scan<MODE, 32, 2>(a, tiles, longest, stream);
   if (a.dim <= 512) return launch_scan<MODE, 32, 4>(a, tiles, longest, stream);
@@ -614,7 +736,7 @@ bool on16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 }  // namespace
 
-// mode 0: the delta rule (decay = g, s0 = beta); 1: the bonus form (decay = z with decay_bias, bonus = u); 2: the matrix memory
+// mode 0: the delta rule (decay = g, s0 = beta, s1 = q . k per query head); 1: the bonus form (decay = z with decay_bias, bonus = u); 2: the matrix memory
 // (s0, s1 = the projections of the forget and the input gate with their biases, cap; aux [n, heads, 2]). q and k
 // rows hold heads / rep heads. o: [n, heads * vdim]. tiles: one per sequence (sequence, first row, rows).
 BW_API int BW_FN(state_scan)(int mode, const float* q, int q_stride, const float* k, int k_stride, const float* v,
@@ -677,8 +799,11 @@ BW_API int BW_FN(delta_prepare)(const float* u, int u_stride, int beta_col, cons
   a.conv_state = taps > 1 ? conv_state : nullptr, a.keep = keep, a.z = z, a.z_stride = z_stride, a.dt_bias = dt_bias, a.a_log = a_log;
   a.out = out, a.out_stride = out_stride, a.pos = pos, a.row_seq = row_seq, a.seq_row0 = seq_row0, a.seq_slot = seq_slot;
   a.heads = heads, a.kv_heads = kv_heads, a.dim = dim, a.vdim = vdim, a.q_scale = q_scale;
-  const int units = 2 * kv_heads + 2 * heads + 1;
-  bw::launch_pdl(delta_prepare_kernel, dim3(n, (units + kThreads / 32 - 1) / (kThreads / 32)), dim3(kThreads), 0, stream, a);
+  const dim3 grid(n, (kv_heads + 2 * heads + 1 + kWarps - 1) / kWarps);
+  if (dim % 4 == 0 && vdim % 4 == 0 && u_stride % 4 == 0 && out_stride % 4 == 0 && on16(u) && on16(conv_t) && on16(conv_state) && on16(out))
+    bw::launch_pdl(delta_prepare_kernel<4>, grid, dim3(kThreads), 0, stream, a);
+  else
+    bw::launch_pdl(delta_prepare_kernel<1>, grid, dim3(kThreads), 0, stream, a);
   return bw::launch_status();
 }
 

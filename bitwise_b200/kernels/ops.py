@@ -1328,14 +1328,15 @@ class KernelOps:
                    batch, seq_tiles, heads: int, dim: int, vdim: int, decay: Optional[torch.Tensor] = None,
                    decay_bias: Optional[torch.Tensor] = None, bonus: Optional[torch.Tensor] = None,
                    beta: Optional[torch.Tensor] = None, forget: Optional[torch.Tensor] = None,
-                   inp: Optional[torch.Tensor] = None, forget_bias: Optional[torch.Tensor] = None,
+                   qk: Optional[torch.Tensor] = None, inp: Optional[torch.Tensor] = None, forget_bias: Optional[torch.Tensor] = None,
                    inp_bias: Optional[torch.Tensor] = None, cap: float = 0.0, aux: Optional[torch.Tensor] = None) -> None:
         """One recurrence over the rows of every sequence of the step (``seq_tiles``: one tile per sequence), from and
         into ``state`` [slots, *scan_state_shape] (zero at a request's first position); the outputs before their norm
         into ``o`` [n, heads * vdim].  q, k [n, heads' * dim] (heads a multiple of heads'; head h reads head h // (heads
         / heads')), v [n, heads * vdim]: float32, rows may be columns of wider rows.  Per head:
 
-        * "delta": S <- g S, S <- S + k (beta (v - S^T k))^T, o = S^T q; ``decay`` [n, heads * dim] = g, ``beta`` [n, heads];
+        * "delta": S <- g S, S <- S + k (beta (v - S^T k))^T, o = S^T q; ``decay`` [n, heads * dim] = g, ``beta`` [n, heads],
+          ``qk`` [n, heads'] the products q . k;
         * "bonus": o = (S + diag(u) k v^T)^T q, S <- diag(w) S + k v^T, w = exp(-exp(z + z0)); ``decay`` = z, ``decay_bias``
           = z0 and ``bonus`` = u [heads * dim];
         * "memory": m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, n alike, o = S^T q; i = cap tanh((inp +
@@ -1358,7 +1359,9 @@ class KernelOps:
         if mode in ("delta", "bonus"):
             rows.append((decay, heads * dim, "decay"))
         if mode == "delta":
-            rows.append((beta, heads, "beta"))
+            rows += [(beta, heads, "beta"), (qk, q.shape[1] // dim, "qk")]
+            if beta is not None and qk is not None and beta.stride(0) != qk.stride(0):
+                raise KernelError("state_scan: the rows of beta and of q . k must lie equally far apart")
         elif mode == "bonus":
             vectors += [(decay_bias, heads * dim, "decay_bias"), (bonus, heads * dim, "bonus")]
         else:
@@ -1387,7 +1390,7 @@ class KernelOps:
                 raise KernelError(f"state_scan: {what} does not hold {count} numbers")
         t_seq, t_row0, t_rows, t_count = seq_tiles
         s0 = beta if mode == "delta" else forget if mode == "memory" else None
-        s1 = inp if mode == "memory" else None
+        s1 = inp if mode == "memory" else qk if mode == "delta" else None
         self._sccall("state_scan", _c_int(self.SCAN_MODES.index(mode)), _p(q), _c_int(q.stride(0)), _p(k), _c_int(k.stride(0)),
                      _p(v), _c_int(v.stride(0)), _c_int(heads // (q.shape[1] // dim)), _p(decay),
                      _c_int(decay.stride(0) if decay is not None else 0), _p(decay_bias), _p(bonus), _p(s0), _p(s1),
@@ -1425,7 +1428,7 @@ class KernelOps:
         (``heads`` of ``vdim``), and from ``beta_col`` on the projections of beta.  q, k and v pass the convolution over time
         with ``conv_t`` [taps, channels] (earlier inputs from ``conv_state`` [slots, taps - 1, channels], zeros before position
         0) and SiLU; q and k heads are divided by sqrt(sum of squares + 1e-6), q times ``q_scale``; ``out`` (float32 [n, >=
-        channels + heads]) receives q | k | v | sigmoid(beta).  ``z`` (float32 rows of heads * dim) becomes exp(-exp(a_log_h)
+        channels + heads + kv_heads]) receives q | k | v | sigmoid(beta) | q . k per query head.  ``z`` (float32 rows of heads * dim) becomes exp(-exp(a_log_h)
         softplus(z + dt_bias)).  ``keep``: every sequence of the step has one row, and its state is brought up to date here."""
         n = u.shape[0]
         _need_rows(u, torch.float32, "delta_prepare u")
@@ -1437,7 +1440,7 @@ class KernelOps:
         taps, channels = conv_t.shape
         if channels != 2 * kv_heads * dim + heads * vdim or beta_col < channels or u.shape[1] < beta_col + heads or \
                 tuple(z.shape) != (n, heads * dim) or dt_bias.shape[0] != heads * dim or a_log.shape[0] != heads or \
-                out.shape[0] != n or out.shape[1] < channels + heads or heads % kv_heads:
+                out.shape[0] != n or out.shape[1] < channels + heads + kv_heads or heads % kv_heads:
             raise KernelError("delta_prepare: shapes do not fit the heads")
         if conv_state is not None:
             _need(conv_state, torch.float32, "delta_prepare conv_state", 3)

@@ -139,7 +139,7 @@ class ChannelDelta(_StateMixer):
         z = ws.rows("delta_low32", n, H * self.dim + self.v_cols, torch.float32)
         ops.linear(low, self.w_low, z)
         decay, gate = z[:, :H * self.dim], z[:, H * self.dim:]
-        ready = ws.rows("delta_ready32", n, _padded(self.channels + H), torch.float32)
+        ready = ws.rows("delta_ready32", n, _padded(self.channels + H + self.kv_heads), torch.float32)
         keep = one_row_each(ctx)
         ops.delta_prepare(u, self.beta0, self.conv_t, conv_state, decay, self.decay_bias, self.decay_log, ready, ctx, H,
                           self.kv_heads, self.dim, self.vdim, self.dim ** -0.5, keep=keep)
@@ -148,7 +148,7 @@ class ChannelDelta(_StateMixer):
         o = ws.rows("scan_out32", n, self.v_cols, torch.float32)
         a, b, c = self.qk_cols, 2 * self.qk_cols, self.channels
         ops.state_scan("delta", ready[:, :a], ready[:, a:b], ready[:, b:c], cache.state, o, ctx, tiles, H, self.dim, self.vdim,
-                       decay=decay, beta=ready[:, c:c + H])
+                       decay=decay, beta=ready[:, c:c + H], qk=ready[:, c + H:c + H + self.kv_heads])
         gated = ws.rows("scan_gated", n, self.v_cols, ctx.act_dtype)
         ops.scan_finish(o, self.norm, gate, self.eps, gated, H, self.vdim)
         ops.linear(gated, self.w_o, x, residual=x if accumulate else None)

@@ -307,11 +307,12 @@ class CpuOps:
         out[:, :2 * kv_heads * dim] = qk.reshape(n, -1)
         out[:, 2 * kv_heads * dim:channels] = y[:, 2 * kv_heads * dim:]
         out[:, channels:channels + heads] = torch.sigmoid(u[:, beta_col:beta_col + heads])
+        out[:, channels + heads:channels + heads + kv_heads] = (qk[:, :kv_heads] * qk[:, kv_heads:]).sum(-1)
         soft = torch.nn.functional.softplus(z + dt_bias).view(n, heads, dim)
         z.copy_(torch.exp(-torch.exp(a_log).view(1, -1, 1) * soft).reshape(n, -1))
 
     def state_scan(self, mode, q, k, v, state, o, ctx, tiles, heads, dim, vdim, decay=None, decay_bias=None, bonus=None,
-                   beta=None, forget=None, inp=None, forget_bias=None, inp_bias=None, cap=0.0, aux=None):
+                   beta=None, qk=None, forget=None, inp=None, forget_bias=None, inp_bias=None, cap=0.0, aux=None):
         n = q.shape[0]
         rep = heads // (q.shape[1] // dim)
         qh = q.reshape(n, -1, dim).repeat_interleave(rep, 1)
@@ -331,6 +332,7 @@ class CpuOps:
                     w = beta[r][:, None] * (vh[r] - torch.einsum("hvd,hd->hv", S, kh[r]))
                     S.add_(w[:, :, None] * kh[r][:, None, :])
                     out = torch.einsum("hvd,hd->hv", S, qh[r])
+                    assert torch.allclose((q.reshape(n, -1, dim)[r] * k.reshape(n, -1, dim)[r]).sum(-1), qk[r], atol=1e-5)
                 elif mode == "bonus":
                     out = torch.einsum("hvd,hd->hv", S + bonus.view(heads, 1, dim) * kv, qh[r])
                     w = torch.exp(-torch.exp(decay[r] + decay_bias)).view(heads, 1, dim)
