@@ -525,43 +525,52 @@ struct DeltaPrepArgs {
 
 constexpr int kMaxPer = 16;  // entries of a head per lane: sizes up to 512
 
+template <int VEC>
+struct VecOf {
+  typedef float4 type;
+};
+template <>
+struct VecOf<1> {
+  typedef float type;
+};
+
 // The convolution over time and SiLU of one head (`size` channels from col0 on) into the lane's registers: with VEC 4 four
 // neighbouring channels at a time (128 to a warp), else channels 32 apart. The order of a channel's sum is the taps', either way.
 template <int VEC>
 __device__ __forceinline__ void conv_head(const DeltaPrepArgs& a, int r, int p, int row0, float* st, int channels, int lane, int col0,
                                           int size, float (&val)[kMaxPer]) {
-  constexpr int NG = kMaxPer / VEC;
+  constexpr int NG = kMaxPer / VEC, kTapBatch = 4;  // taps whose inputs are asked for together
+  typedef typename VecOf<VEC>::type vec_t;
 #pragma unroll
   for (int j = 0; j < kMaxPer; ++j) val[j] = 0.0f;
   const float* u = a.u + static_cast<size_t>(r) * a.u_stride + col0;
-  for (int t = 0; t < a.taps; ++t) {  // taps ascending
-    const int back = a.taps - 1 - t;
-    if (p - back < 0) continue;
-    const float* src = r - back >= row0 ? u - static_cast<ptrdiff_t>(back) * a.u_stride
-                                        : st + static_cast<size_t>(a.taps - 1 - (row0 - (r - back))) * channels + col0;
-    const float* w = a.conv_t + static_cast<size_t>(t) * channels + col0;
+  const bool keep = a.keep && st;
 #pragma unroll
-    for (int g = 0; g < NG; ++g) {
-      const int e = VEC * (lane + 32 * g);
-      if (e >= size) continue;
-      if (VEC == 4) {
-        const float4 x = *reinterpret_cast<const float4*>(src + e), c = *reinterpret_cast<const float4*>(w + e);
-        val[4 * g] = __fmaf_rn(c.x, x.x, val[4 * g]), val[4 * g + 1] = __fmaf_rn(c.y, x.y, val[4 * g + 1]);
-        val[4 * g + 2] = __fmaf_rn(c.z, x.z, val[4 * g + 2]), val[4 * g + 3] = __fmaf_rn(c.w, x.w, val[4 * g + 3]);
-      } else {
-        val[g] = __fmaf_rn(w[e], src[e], val[g]);
+  for (int g = 0; g < NG; ++g) {
+    const int e = VEC * (lane + 32 * g);
+    if (e >= size) continue;
+    for (int t0 = 0; t0 < a.taps; t0 += kTapBatch) {  // taps ascending
+      vec_t x[kTapBatch], w[kTapBatch];
+#pragma unroll
+      for (int i = 0; i < kTapBatch; ++i) {
+        const int t = t0 + i, back = a.taps - 1 - t;
+        x[i] = vec_t{}, w[i] = vec_t{};
+        if (t >= a.taps || p - back < 0) continue;
+        const float* src = r - back >= row0 ? u - static_cast<ptrdiff_t>(back) * a.u_stride
+                                            : st + static_cast<size_t>(a.taps - 1 - (row0 - (r - back))) * channels + col0;
+        x[i] = *reinterpret_cast<const vec_t*>(src + e);
+        w[i] = *reinterpret_cast<const vec_t*>(a.conv_t + static_cast<size_t>(t) * channels + col0 + e);
       }
-    }
-  }
-  if (a.keep && st) {  // the sequence's only row: the inputs move up by one
 #pragma unroll
-    for (int j = 0; j < kMaxPer; ++j) {
-      const int e = VEC * (lane + 32 * (j / VEC)) + j % VEC;
-      if (e >= size) continue;
-      float* at = st + col0 + e;
-      for (int t = 0; t + 1 < a.taps - 1; ++t)
-        at[static_cast<size_t>(t) * channels] = p - (a.taps - 2 - t) >= 0 ? at[static_cast<size_t>(t + 1) * channels] : 0.0f;
-      at[static_cast<size_t>(a.taps - 2) * channels] = u[e];
+      for (int i = 0; i < kTapBatch; ++i) {  // (a tap before the sequence's start adds 0 * 0)
+        const float* xf = reinterpret_cast<const float*>(&x[i]);
+        const float* wf = reinterpret_cast<const float*>(&w[i]);
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) val[VEC * g + c] = __fmaf_rn(wf[c], xf[c], val[VEC * g + c]);
+        // the sequence's only row: the inputs move up by one (row t - 1 of the state was read as tap t - 1)
+        if (keep && t0 + i >= 1 && t0 + i < a.taps)
+          *reinterpret_cast<vec_t*>(st + static_cast<size_t>(t0 + i - 1) * channels + col0 + e) = x[i];
+      }
     }
   }
 #pragma unroll
