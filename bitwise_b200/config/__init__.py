@@ -6,10 +6,13 @@ from .nuderax import LatentMixerConfig, NuderaxConfig, NuderaxLayerConfig, Route
 from .sebavik import BigramConfig, SebavikConfig, SebavikLayerConfig, SebavikMixerConfig, SebavikMlpConfig
 from .zuzupel import (ChannelDeltaConfig, ChunkAttentionConfig, MatrixMemoryConfig, ParallelConfig, WkvConfig, ZuzupelConfig,
                       ZuzupelLayerConfig)
+from .sazisun import (ExpertsConfig, FeedForwardConfig, SazisunConfig, SazisunLayerConfig, StateSpaceConfig, TwoMapAttentionConfig,
+                      WavelengthScalingConfig)
 from .registry import (Architecture, architecture_of, config_from_folder, known_architectures,
                        lookup_architecture, register_architecture)
 
-__all__ = ["ChannelDeltaConfig", "ChunkAttentionConfig", "MatrixMemoryConfig", "ParallelConfig", "WkvConfig", "ZuzupelConfig",
+__all__ = ["ExpertsConfig", "FeedForwardConfig", "SazisunConfig", "SazisunLayerConfig", "StateSpaceConfig", "TwoMapAttentionConfig",
+           "WavelengthScalingConfig", "ChannelDeltaConfig", "ChunkAttentionConfig", "MatrixMemoryConfig", "ParallelConfig", "WkvConfig", "ZuzupelConfig",
            "ZuzupelLayerConfig", "KezuvikConfig", "KezuvikLayerConfig", "KezuvikMixerConfig", "RotScalingConfig", "BigramConfig", "SebavikConfig", "SebavikLayerConfig", "SebavikMixerConfig", "SebavikMlpConfig", "ConfigError", "FavudraConfig", "FavudraLayerConfig", "FavudraMixerConfig", "LlamaConfig", "RopeScaling", "NuderaxConfig", "NuderaxLayerConfig", "LatentMixerConfig",
            "RoutedMlpConfig", "read_config_json", "Architecture",
            "architecture_of", "config_from_folder", "known_architectures", "lookup_architecture",

@@ -73,3 +73,5 @@ def _ensure_builtin() -> None:
         from ..models import kezuvik  # noqa: F401
     if "Zuzupel" not in _ARCHITECTURES:
         from ..models import zuzupel  # noqa: F401
+    if "Sazisun" not in _ARCHITECTURES:
+        from ..models import sazisun  # noqa: F401

@@ -665,7 +665,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         }
         continue;
       }
-      if (EPI == 0 && !GROUPED && y_is_f32 == 2 * bw::kOutRelu2) {
+      if (EPI == 0 && y_is_f32 == 2 * bw::kOutRelu2) {
 #pragma unroll
         for (int j = 0; j < 2 * PW; ++j) total[j] = bw::out_act(total[j], bw::kOutRelu2);
       } else if (EPI == 0 && !GROUPED && y_is_f32 == 2 * bw::kOutTanh) {
@@ -1095,8 +1095,9 @@ BW_API int bw_bf16_linear_tc_grouped(const __nv_bfloat16* x, const __nv_bfloat16
   }
   int* word = bw::failure_word();
   if (!word) return -1;
-  if (y_is_f32) return launch_tc_grouped<2>(x, w, y, 1, rows, n, k, group_off, tile_prefix, groups, word, stream);
-  return launch_tc_grouped<0>(x, w, y, 0, rows, n, k, group_off, tile_prefix, groups, word, stream);
+  // y_is_f32: 1 float32; 2 * act (bw::out_act: nothing or the square of relu): bfloat16 after the activation
+  if (y_is_f32 == 1) return launch_tc_grouped<2>(x, w, y, 1, rows, n, k, group_off, tile_prefix, groups, word, stream);
+  return launch_tc_grouped<0>(x, w, y, y_is_f32, rows, n, k, group_off, tile_prefix, groups, word, stream);
 }
 
 // h[m][n / 2] = SwiGLU of x W^T for gate/up weights interleaved in blocks of 64 rows

@@ -232,6 +232,12 @@ __device__ __forceinline__ float out_act(float v, int act) {
   return v;
 }
 
+// One entry of the norm without statistics: tanh(alpha x) w + b. One definition for the stand-alone kernel and the products
+// that form it in their epilogue.
+__device__ __forceinline__ float tanh_norm_one(float x, float alpha, float w, float b) {
+  return __fmaf_rn(tanhf(__fmul_rn(alpha, x)), w, b);
+}
+
 // The tail of RMSNorm for one element, and the scale from the sum of squares: one definition
 // for the stand-alone kernel and the fused one.
 __device__ __forceinline__ float rms_scale(float sumsq, int width, float eps) {

@@ -2,7 +2,7 @@
 // feed-forward read the same input: y = (x - mean) / sqrt(var + eps) * w, var the mean of the
 // squared deviations (two passes over a row held in shared memory). Statistics and the stream
 // are float32 in both precisions. One block per row; a row's sums are formed in an order that
-// depends on the width only.
+// depends on the width only. Beside them a norm without statistics: y = tanh(alpha x) w + b.
 #include "bw_act.cuh"
 
 namespace {
@@ -92,6 +92,42 @@ layernorm_residual_kernel(const float* __restrict__ d, const float* __restrict__
     xn[base + i] = bw::from_f<act_t>(__fmul_rn(__fmul_rn(__fsub_rn(row[i], mean2), inv2), w_next[i]));
 }
 
+// The norm without statistics, y = tanh(alpha x) w + b entry by entry, alpha one stored number. With `d` the sublayer's output
+// joins the stream first: x += d, y from the sum. VEC entries per thread; `rows` gathers.
+template <int VEC>
+__global__ void __launch_bounds__(kThreads)
+tanh_norm_kernel(float* x, const float* __restrict__ d, const float* __restrict__ alpha, const float* __restrict__ w,
+                 const float* __restrict__ b, act_t* y, const int* __restrict__ rows, int width) {
+  bw::pdl_enter();
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+  if (c >= width) return;
+  const int r = blockIdx.x;
+  const size_t from = static_cast<size_t>(rows ? rows[r] : r) * width + c, to = static_cast<size_t>(r) * width + c;
+  const float al = alpha[0];
+  float o[VEC];
+  if constexpr (VEC == 4) {
+    float4 v = *reinterpret_cast<const float4*>(x + from);
+    if (d) {
+      const float4 a = *reinterpret_cast<const float4*>(d + from);
+      v.x = __fadd_rn(v.x, a.x), v.y = __fadd_rn(v.y, a.y), v.z = __fadd_rn(v.z, a.z), v.w = __fadd_rn(v.w, a.w);
+      *reinterpret_cast<float4*>(x + from) = v;
+    }
+    const float4 wv = *reinterpret_cast<const float4*>(w + c), bv = *reinterpret_cast<const float4*>(b + c);
+    o[0] = bw::tanh_norm_one(v.x, al, wv.x, bv.x), o[1] = bw::tanh_norm_one(v.y, al, wv.y, bv.y);
+    o[2] = bw::tanh_norm_one(v.z, al, wv.z, bv.z), o[3] = bw::tanh_norm_one(v.w, al, wv.w, bv.w);
+#if BW_ACT_BF16
+    __nv_bfloat162 p[2] = {__floats2bfloat162_rn(o[0], o[1]), __floats2bfloat162_rn(o[2], o[3])};
+    *reinterpret_cast<uint2*>(y + to) = *reinterpret_cast<const uint2*>(p);
+#else
+    *reinterpret_cast<float4*>(y + to) = make_float4(o[0], o[1], o[2], o[3]);
+#endif
+  } else {
+    float v = x[from];
+    if (d) x[from] = v = __fadd_rn(v, d[from]);
+    y[to] = bw::from_f<act_t>(bw::tanh_norm_one(v, al, w[c], b[c]));
+  }
+}
+
 // x += d, element by element (the residual sum of a block whose parts wrote into d).
 __global__ void add_rows_kernel(float* x, const float* __restrict__ d, size_t count) {
   bw::pdl_enter();
@@ -130,6 +166,27 @@ BW_API int BW_FN(layernorm_residual)(const float* d, const float* w, float* x, i
   }
   bw::launch_pdl(layernorm_residual_kernel, dim3(n), dim3(kThreads), static_cast<size_t>(width) * sizeof(float), stream,
                  d, w, x, width, eps, w_next, eps_next, static_cast<act_t*>(xn));
+  return bw::launch_status();
+}
+
+// y[r] = tanh(alpha x[rows[r]]) w + b into the activation type (rows null: row r). d (no rows then): x += d first.
+BW_API int BW_FN(tanh_norm)(float* x, const float* d, const float* alpha, const float* w, const float* b, void* y,
+                            const int* rows, int n, int width, cudaStream_t stream) {
+  if (n <= 0 || width <= 0) return 0;
+  if (d && rows) {
+    bw::set_error("tanh_norm: a residual sum is formed for every row of the stream, not for gathered ones");
+    return -1;
+  }
+  const bool by_four = width % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(d) | reinterpret_cast<uintptr_t>(w) |
+                                           reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
+  const int want = by_four ? width / 4 : width;
+  const int threads = want >= kThreads ? kThreads : (want + 31) / 32 * 32;
+  const dim3 grid(n, (want + threads - 1) / threads);
+  act_t* out = static_cast<act_t*>(y);
+  if (by_four)
+    bw::launch_pdl(tanh_norm_kernel<4>, grid, dim3(threads), 0, stream, x, d, alpha, w, b, out, rows, width);
+  else
+    bw::launch_pdl(tanh_norm_kernel<1>, grid, dim3(threads), 0, stream, x, d, alpha, w, b, out, rows, width);
   return bw::launch_status();
 }
 

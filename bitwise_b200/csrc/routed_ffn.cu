@@ -4,8 +4,10 @@
 //    sigmoid(z); a correction per expert is added for the choice only; the experts form equal
 //    groups of neighbours, a group counts as the sum of its two largest choice scores, and only
 //    the experts of the best groups can be chosen; the weights are the chosen experts' scores
-//    times a constant. `softmax_top`: the choice is by the logits themselves (plus the correction), and
-//    the weights are the softmax over the chosen logits only.
+//    times a constant. Scoring kSoftmaxTop: the choice is by the logits themselves (plus the correction), and
+//    the weights are the softmax over the chosen logits only. Scoring kSoftmax: the scores are the softmax
+//    over all experts. A group may count as its largest choice score alone, and the weights may be
+//    divided by their sum.
 //  * group_rows: (row, choice) pairs listed expert by expert, with the tiles of the grouped
 //    product that follows.
 //  * grouped_linear: out[i] = x[source(i)] W_g^T for the list entries i of every group g, W
@@ -16,7 +18,8 @@
 //  * gather_rows: the rows of a list made contiguous, for the tcgen05 product over long lists
 //    (bf16_gemm_tc.cu), which fetches tiles of consecutive rows.
 //  * glu_clamped: y = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, +-limit).
-//  * combine: x += d + sum_j weight_j * y[place of (row, j)], the sum in the order of choice.
+//  * combine: x += d + sum_j weight_j * y[place of (row, j)], the sum in the order of choice; d may be
+//    multiplied by the sigmoid of one number per row first (a gated shared expert).
 #include "bw_act.cuh"
 #include "bw_mma.cuh"
 
@@ -27,10 +30,12 @@ namespace {
 // ---------------------------------------------------------------------------------------
 // One warp per row. Shared memory per warp: scores s[E] (a taken expert's is set to -1), choice
 // scores c[E] (-inf for the experts of groups that do not stay), group scores [groups].
+enum { kSigmoid = 0, kSoftmaxTop = 1, kSoftmax = 2 };
+
 __global__ void __launch_bounds__(128)
-route_kernel(const float* __restrict__ z, const float* __restrict__ correction, int n, int experts, int groups,
-             int keep, int top, float weight_scale, int softmax_top, int* __restrict__ chosen,
-             float* __restrict__ weights) {
+route_kernel(const float* __restrict__ z, int z_stride, const float* __restrict__ correction, int n, int experts, int groups,
+             int keep, int top, float weight_scale, int scoring, int group_max, float sum_eps /* >= 0: weights over their sum */,
+             int* __restrict__ chosen, float* __restrict__ weights) {
   bw::pdl_enter();
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -39,11 +44,26 @@ route_kernel(const float* __restrict__ z, const float* __restrict__ correction, 
   float* s = sm + static_cast<size_t>(warp) * (2 * experts + groups);
   float* c = s + experts;
   float* gs = c + experts;
-  const float* zr = z + static_cast<size_t>(r) * experts;
-  for (int e = lane; e < experts; e += 32) {
-    const float v = softmax_top ? zr[e] : __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-zr[e])));
-    s[e] = softmax_top ? 0.0f : v;  // (only its sign is used then: negative once taken)
-    c[e] = correction ? __fadd_rn(v, correction[e]) : v;
+  const float* zr = z + static_cast<size_t>(r) * z_stride;
+  const bool softmax_top = scoring == kSoftmaxTop;
+  if (scoring == kSoftmax) {
+    float m = -INFINITY, sum = 0.0f;
+    for (int e = lane; e < experts; e += 32) m = fmaxf(m, zr[e]);
+    m = bw::warp_max(m);
+    for (int e = lane; e < experts; e += 32) sum = __fadd_rn(sum, expf(__fsub_rn(zr[e], m)));
+    sum = bw::warp_sum(sum);
+    for (int e = lane; e < experts; e += 32) {
+      const float v = __fdiv_rn(expf(__fsub_rn(zr[e], m)), sum);
+      s[e] = v;
+      // (the scores order the experts as the logits do, which keep apart what underflows)
+      c[e] = correction ? __fadd_rn(v, correction[e]) : group_max ? zr[e] : v;
+    }
+  } else {
+    for (int e = lane; e < experts; e += 32) {
+      const float v = softmax_top ? zr[e] : __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-zr[e])));
+      s[e] = softmax_top ? 0.0f : v;  // (only its sign is used then: negative once taken)
+      c[e] = correction ? __fadd_rn(v, correction[e]) : v;
+    }
   }
   __syncwarp();
   const int per = experts / groups;
@@ -55,7 +75,7 @@ route_kernel(const float* __restrict__ z, const float* __restrict__ correction, 
         if (v > a) b = a, a = v;
         else if (v > b) b = v;
       }
-      gs[g] = per > 1 ? __fadd_rn(a, b) : a;
+      gs[g] = per > 1 && !group_max ? __fadd_rn(a, b) : a;
     }
     __syncwarp();
     // the groups that stay are taken out of gs one by one (marked +inf); the rest lose their experts
@@ -93,10 +113,17 @@ route_kernel(const float* __restrict__ z, const float* __restrict__ correction, 
     }
     if (lane == 0) {
       chosen[static_cast<size_t>(r) * top + k] = at;
-      weights[static_cast<size_t>(r) * top + k] = softmax_top ? zr[at] : __fmul_rn(s[at], weight_scale);
+      weights[static_cast<size_t>(r) * top + k] = softmax_top ? zr[at] : sum_eps >= 0.0f ? s[at] : __fmul_rn(s[at], weight_scale);
       s[at] = -1.0f;  // taken
     }
     __syncwarp();
+  }
+  if (!softmax_top && sum_eps >= 0.0f && lane == 0) {
+    float* wr = weights + static_cast<size_t>(r) * top;
+    float sum = 0.0f;
+    for (int k = 0; k < top; ++k) sum = __fadd_rn(sum, wr[k]);
+    sum = __fadd_rn(sum, sum_eps);
+    for (int k = 0; k < top; ++k) wr[k] = __fmul_rn(__fdiv_rn(wr[k], sum), weight_scale);
   }
   if (softmax_top && lane == 0) {
     // the softmax over the chosen logits, in the order of choice (the first is the largest)
@@ -177,7 +204,7 @@ __global__ void __launch_bounds__(256)
 grouped_linear_kernel(const act_t* __restrict__ x, int x_stride, int x_group_cols, const int* __restrict__ order,
                       int order_div, const act_t* __restrict__ w, OutT* out, int o_stride, int o_group_cols,
                       const int* __restrict__ group_off, const int* __restrict__ tile_prefix, int uniform_rows,
-                      int groups, int n, int k) {
+                      int groups, int n, int k, int act) {
   bw::pdl_enter();
   __shared__ float xs[kStep][kTile + 1];
   __shared__ float ws[kStep][kTile + 1];
@@ -259,7 +286,7 @@ grouped_linear_kernel(const act_t* __restrict__ x, int x_stride, int x_group_col
 #pragma unroll
     for (int b = 0; b < 4; ++b) {
       const int j = j0 + tx * 4 + b;
-      if (j < n) orow[j] = bw::from_f<OutT>(acc[a][b]);
+      if (j < n) orow[j] = bw::from_f<OutT>(bw::out_act(acc[a][b], act));
     }
   }
 }
@@ -277,7 +304,7 @@ __global__ void __launch_bounds__(WM * WN * 32)
 grouped_linear_mma_kernel(const act_t* __restrict__ x, int x_stride, int x_group_cols, const int* __restrict__ order,
                           int order_div, const act_t* __restrict__ w, OutT* out, int o_stride, int o_group_cols,
                           const int* __restrict__ group_off, const int* __restrict__ tile_prefix, int uniform_rows,
-                          int groups, int n, int k) {
+                          int groups, int n, int k, int act) {
   bw::pdl_enter();
   constexpr int THREADS = WM * WN * 32;
   constexpr int TM = BM / WM, TN = BN / WN, MI = TM / 16, NI = TN / 8;
@@ -398,8 +425,8 @@ grouped_linear_mma_kernel(const act_t* __restrict__ x, int x_stride, int x_group
 #pragma unroll
       for (int ni = 0; ni < NI; ++ni) {
         const int j = j0 + wn + ni * 8 + 2 * (lane & 3);
-        if (j < n) orow[j] = bw::from_f<OutT>(acc[mi][ni][2 * half]);
-        if (j + 1 < n) orow[j + 1] = bw::from_f<OutT>(acc[mi][ni][2 * half + 1]);
+        if (j < n) orow[j] = bw::from_f<OutT>(bw::out_act(acc[mi][ni][2 * half], act));
+        if (j + 1 < n) orow[j + 1] = bw::from_f<OutT>(bw::out_act(acc[mi][ni][2 * half + 1], act));
       }
     }
 }
@@ -409,7 +436,7 @@ constexpr int kBigTile = 128;
 template <typename OutT, int BM, int BN, int WM, int WN, int STAGES>
 int launch_grouped_mma(dim3 grid, cudaStream_t stream, const act_t* x, int x_stride, int x_group_cols, const int* order,
                        int order_div, const act_t* w, OutT* out, int o_stride, int o_group_cols, const int* group_off,
-                       const int* tile_prefix, int rows, int groups, int n, int k) {
+                       const int* tile_prefix, int rows, int groups, int n, int k, int act) {
   auto kernel = grouped_linear_mma_kernel<OutT, BM, BN, WM, WN, STAGES>;
   constexpr size_t smem = static_cast<size_t>(STAGES) * (BM + BN) * kMmaRow * sizeof(__nv_bfloat16);
   static bool raised = false;
@@ -422,7 +449,7 @@ int launch_grouped_mma(dim3 grid, cudaStream_t stream, const act_t* x, int x_str
     raised = true;
   }
   bw::launch_pdl(kernel, grid, dim3(WM * WN * 32), smem, stream, x, x_stride, x_group_cols, order, order_div, w, out,
-                 o_stride, o_group_cols, group_off, tile_prefix, rows, groups, n, k);
+                 o_stride, o_group_cols, group_off, tile_prefix, rows, groups, n, k, act);
   return bw::launch_status();
 }
 #endif
@@ -482,7 +509,7 @@ __global__ void glu_clamped_kernel(const act_t* __restrict__ gate_up, act_t* __r
 template <bool VEC>
 __global__ void combine_kernel(float* x, const float* __restrict__ d, const float* __restrict__ y,
                                const int* __restrict__ place, const float* __restrict__ weights, int top, int width,
-                               const float* __restrict__ scale) {
+                               const float* __restrict__ scale, const float* __restrict__ d_gate, int gate_stride) {
   bw::pdl_enter();
   constexpr int per = VEC ? 4 : 1;
   const int r = blockIdx.x;
@@ -502,18 +529,22 @@ __global__ void combine_kernel(float* x, const float* __restrict__ d, const floa
     }
   }
   const size_t o = static_cast<size_t>(r) * width + c;
+  const float gate = d_gate ? __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-d_gate[static_cast<size_t>(r) * gate_stride]))) : 1.0f;
 #pragma unroll
   for (int e = 0; e < per; ++e) {
     float v = s[e];
-    if (d) v = __fadd_rn(d[o + e], v);
+    if (d) v = d_gate ? __fmaf_rn(gate, d[o + e], v) : __fadd_rn(d[o + e], v);
     x[o + e] = scale ? __fmaf_rn(scale[c + e], v, x[o + e]) : __fadd_rn(x[o + e], v);
   }
 }
 
 }  // namespace
 
-BW_API int BW_FN(route)(const float* z, const float* correction, int n, int experts, int groups, int keep, int top,
-                        float weight_scale, int softmax_top, int* chosen, float* weights, cudaStream_t stream) {
+// z: rows of z_stride floats (at least `experts`). scoring: 0 sigmoid, 1 the softmax over the chosen, 2 the softmax over all.
+// group_max: a group counts as its largest score. sum_eps >= 0: the weights are divided by their sum plus sum_eps.
+BW_API int BW_FN(route)(const float* z, int z_stride, const float* correction, int n, int experts, int groups, int keep, int top,
+                        float weight_scale, int scoring, int group_max, float sum_eps, int* chosen, float* weights,
+                        cudaStream_t stream) {
   if (n <= 0) return 0;
   if (experts <= 0 || groups <= 0 || experts % groups || keep <= 0 || keep > groups || top <= 0 ||
       top > keep * (experts / groups)) {
@@ -526,8 +557,8 @@ BW_API int BW_FN(route)(const float* z, const float* correction, int n, int expe
     bw::set_error("route: %d experts are beyond the kernel", experts);
     return -1;
   }
-  bw::launch_pdl(route_kernel, dim3((n + warps - 1) / warps), dim3(warps * 32), smem, stream, z, correction, n, experts,
-                 groups, keep, top, weight_scale, softmax_top, chosen, weights);
+  bw::launch_pdl(route_kernel, dim3((n + warps - 1) / warps), dim3(warps * 32), smem, stream, z, z_stride, correction, n, experts,
+                 groups, keep, top, weight_scale, scoring, group_max, sum_eps, chosen, weights);
   return bw::launch_status();
 }
 
@@ -564,7 +595,12 @@ BW_API int BW_FN(group_rows)(const int* chosen, int pairs, int experts, int* gro
 BW_API int BW_FN(grouped_linear)(const act_t* x, int x_stride, int x_group_cols, const int* order, int order_div,
                                  const act_t* w, void* out, int out_is_f32, int o_stride, int o_group_cols,
                                  const int* group_off, const int* tile_prefix, int rows, int groups, int n, int k,
-                                 cudaStream_t stream) {
+                                 int act, cudaStream_t stream) {
+  // act: what an output passes before it is stored (bw::out_act: 0 nothing, 1 the square of relu)
+  if (act != bw::kOutNone && act != bw::kOutRelu2) {
+    bw::set_error("grouped_linear: unknown activation %d", act);
+    return -1;
+  }
   if (rows <= 0 || groups <= 0 || n <= 0) return 0;
   if (k <= 0 || order_div <= 0) {
     bw::set_error("grouped_linear: inner size %d", k);
@@ -591,26 +627,26 @@ BW_API int BW_FN(grouped_linear)(const act_t* x, int x_stride, int x_group_cols,
       if (out_is_f32)
         return launch_grouped_mma<float, 128, 128, 2, 4, 4>(bgrid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                             static_cast<float*>(out), o_stride, o_group_cols, group_off,
-                                                            prefix, rows, groups, n, k);
+                                                            prefix, rows, groups, n, k, act);
       return launch_grouped_mma<act_t, 128, 128, 2, 4, 4>(bgrid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                           static_cast<act_t*>(out), o_stride, o_group_cols, group_off,
-                                                          prefix, rows, groups, n, k);
+                                                          prefix, rows, groups, n, k, act);
     }
     if (out_is_f32)
       return launch_grouped_mma<float, 64, 64, 2, 2, 3>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                         static_cast<float*>(out), o_stride, o_group_cols, group_off,
-                                                        tile_prefix, rows, groups, n, k);
+                                                        tile_prefix, rows, groups, n, k, act);
     return launch_grouped_mma<act_t, 64, 64, 2, 2, 3>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                       static_cast<act_t*>(out), o_stride, o_group_cols, group_off,
-                                                      tile_prefix, rows, groups, n, k);
+                                                      tile_prefix, rows, groups, n, k, act);
   }
 #endif
   if (out_is_f32)
     bw::launch_pdl(grouped_linear_kernel<float>, grid, dim3(256), 0, stream, x, x_stride, x_group_cols, order, order_div,
-                   w, static_cast<float*>(out), o_stride, o_group_cols, group_off, tile_prefix, rows, groups, n, k);
+                   w, static_cast<float*>(out), o_stride, o_group_cols, group_off, tile_prefix, rows, groups, n, k, act);
   else
     bw::launch_pdl(grouped_linear_kernel<act_t>, grid, dim3(256), 0, stream, x, x_stride, x_group_cols, order, order_div,
-                   w, static_cast<act_t*>(out), o_stride, o_group_cols, group_off, tile_prefix, rows, groups, n, k);
+                   w, static_cast<act_t*>(out), o_stride, o_group_cols, group_off, tile_prefix, rows, groups, n, k, act);
   return bw::launch_status();
 }
 
@@ -637,13 +673,14 @@ BW_API int BW_FN(glu_clamped)(const act_t* gate_up, act_t* out, int n, int inter
 }
 
 BW_API int BW_FN(combine)(float* x, const float* d, const float* y, const int* place, const float* weights, int n,
-                          int top, int width, const float* scale, cudaStream_t stream) {
+                          int top, int width, const float* scale, const float* d_gate, int gate_stride, cudaStream_t stream) {
+  // d_gate: d is multiplied by the sigmoid of d_gate[r * gate_stride] first (null: as it is)
   if (n <= 0 || width <= 0) return 0;
   if (width % 4 == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0)
     bw::launch_pdl(combine_kernel<true>, dim3(n, (width / 4 + 127) / 128), dim3(128), 0, stream, x, d, y, place, weights, top,
-                   width, scale);
+                   width, scale, d_gate, gate_stride);
   else
     bw::launch_pdl(combine_kernel<false>, dim3(n, (width + 255) / 256), dim3(256), 0, stream, x, d, y, place, weights, top,
-                   width, scale);
+                   width, scale, d_gate, gate_stride);
   return bw::launch_status();
 }

@@ -9,7 +9,9 @@
 //   conv_state_update  the convolution's inputs of a request's last taps - 1 positions
 //   scored_attention   s = (q . k) * scale; s <- cap * tanh(s / cap); s <- s - slope_h * (i - j);
 //                      window or chunks; softmax with an optional extra one in the denominator; the values
-//                      may be the keys themselves (no value pages)
+//                      may be the keys themselves (no value pages); several maps (attentions with queries and keys
+//                      of their own) may weight the same values
+//   scored_difference  two maps of a head become one output: a1 - lambda a2, a norm over the head, an output gate
 //
 // Everything after the projection is float32 in both precisions; only what is loaded and stored
 // changes type. Keys are walked in tiles of 32 at fixed absolute positions, so what a query gets
@@ -382,7 +384,13 @@ struct ScoreArgs {
   const float* sinks;   // [heads] or null: with `sink`, exp(sinks[h]) joins the denominator instead of exp(0)
   int keep_first;       // with a window: the keys j < keep_first stay visible to every later position
   int chunk;            // > 0: position i sees the keys j <= i with j / chunk == i / chunk (no window then)
+  int maps;             // key heads that share a value head: key head g holds map g % maps of value head g / maps, and
+                        // query head h is map h % maps of result head h / maps
 };
+// The first query head of a block's share of the heads on key head g (the others follow `maps` apart).
+__device__ __forceinline__ int first_head(const ScoreArgs& sa, int g, int rep, int skip) {
+  return (g / sa.maps * rep + skip) * sa.maps + g % sa.maps;
+}
 // The first key that a query at position pq sees (kept first keys apart). It never falls as pq grows.
 __device__ __forceinline__ int first_seen(const ScoreArgs& sa, int pq) {
   if (sa.chunk > 0) return pq / sa.chunk * sa.chunk;
@@ -443,7 +451,7 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
                         const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
                         const int* __restrict__ tile_rows, const int* __restrict__ seq_pos0,
                         const int* __restrict__ seq_row0, act_t* out, int o_stride, int heads, int kv_heads, int hb,
-                        int dim, int vdim, int page, const ScoreArgs sa) {
+                        int dim, int vdim, int page, const ScoreArgs sa, float* partial) {
   bw::pdl_enter();
   extern __shared__ float sm[];
   const int ks = dim + 1;
@@ -452,15 +460,15 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
   const int vs = vcache ? vdim : ks;
   float* qs = keys + kKeys * ks + (vcache ? kKeys * vdim : 0);
   const int t = blockIdx.x, g = blockIdx.y;
-  const int rep = heads / kv_heads;
-  const int h0 = g * rep + blockIdx.z * hb;
+  const int rep = heads / kv_heads, v_heads = kv_heads / sa.maps, gv = g / sa.maps;
+  const int h0 = first_head(sa, g, rep, blockIdx.z * hb);
   const int nh = min(hb, rep - blockIdx.z * hb);
   const int seq = tile_seq[t], row0 = tile_row0[t], rows = tile_rows[t];
   const int nq = rows * nh;
   const int p0 = seq_pos0[seq] + (row0 - seq_row0[seq]);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int qi = warp; qi < nq; qi += kWarps) {
-    const act_t* src = q + static_cast<size_t>(row0 + qi / nh) * q_stride + (h0 + qi % nh) * dim;
+    const act_t* src = q + static_cast<size_t>(row0 + qi / nh) * q_stride + (h0 + qi % nh * sa.maps) * dim;
     for (int d = lane; d < dim; d += 32) qs[qi * dim + d] = bw::to_f(src[d]);
   }
   float m[kQW], l[kQW], acc[kQW][ACC];
@@ -480,11 +488,14 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
     for (int kk = warp; kk < kKeys; kk += kWarps) {
       const int kp = k0 + kk;
       const bool have = kp <= last && (kp >= first || kp < keep);
-      size_t at = 0;
-      if (have) at = (static_cast<size_t>(bt[kp / page]) * kv_heads + g) * page + kp % page;
+      size_t at = 0, vat = 0;
+      if (have) {
+        const size_t blk = bt[kp / page];
+        at = (blk * kv_heads + g) * page + kp % page, vat = (blk * v_heads + gv) * page + kp % page;
+      }
       for (int d = lane; d < dim; d += 32) keys[kk * ks + d] = have ? bw::to_f(kcache[at * dim + d]) : 0.0f;
       if (vcache)
-        for (int d = lane; d < vdim; d += 32) vals[kk * vs + d] = have ? bw::to_f(vcache[at * vdim + d]) : 0.0f;
+        for (int d = lane; d < vdim; d += 32) vals[kk * vs + d] = have ? bw::to_f(vcache[vat * vdim + d]) : 0.0f;
     }
     __syncthreads();
 #pragma unroll
@@ -499,7 +510,7 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
       const float* kv = keys + lane * ks;
       float s = 0.0f;
       for (int d = 0; d < dim; ++d) s = __fmaf_rn(qv[d], kv[d], s);
-      s = modify_score(s, sa, head_bias(sa, h0 + qi % nh, true), pq, kp);
+      s = modify_score(s, sa, head_bias(sa, h0 + qi % nh * sa.maps, true), pq, kp);
       const bool seen = key_seen(sa, pq, lo, kp);
       if (!seen) s = -INFINITY;
       const float mt = bw::warp_max(s);
@@ -526,10 +537,19 @@ scored_attention_kernel(const act_t* __restrict__ q, int q_stride, const act_t* 
   for (int j = 0; j < kQW; ++j) {
     const int qi = warp + kWarps * j;
     if (qi >= nq) continue;
+    const int h = h0 + qi % nh * sa.maps;
+    if (partial) {  // a record for the kernel that joins the maps: maximum, sum, weighted values relative to that maximum
+      float* rec = partial + (static_cast<size_t>(row0 + qi / nh) * heads + h) * (vdim + 2);
+      if (lane == 0) rec[0] = m[j], rec[1] = l[j];
+#pragma unroll
+      for (int i = 0; i < ACC; ++i)
+        if (i * 32 + lane < vdim) rec[2 + i * 32 + lane] = acc[j][i];
+      continue;
+    }
     float den = l[j];
-    if (sa.sink) den = __fadd_rn(den, expf(__fsub_rn(sa.sinks ? sa.sinks[h0 + qi % nh] : 0.0f, m[j])));  // the extra key (score 0 unless given)
+    if (sa.sink) den = __fadd_rn(den, expf(__fsub_rn(sa.sinks ? sa.sinks[h] : 0.0f, m[j])));  // the extra key (score 0 unless given)
     const float inv = __fdiv_rn(1.0f, den);
-    act_t* dst = out + static_cast<size_t>(row0 + qi / nh) * o_stride + (h0 + qi % nh) * vdim;
+    act_t* dst = out + static_cast<size_t>(row0 + qi / nh) * o_stride + h * vdim;
 #pragma unroll
     for (int i = 0; i < ACC; ++i) {
       const int d = i * 32 + lane;
@@ -542,7 +562,7 @@ template <int ACC>
 int launch_scored(dim3 grid, size_t smem, cudaStream_t stream, const act_t* q, int q_stride, const act_t* kcache,
                   const act_t* vcache, const int* block_table, int max_blocks, const int* tile_seq, const int* tile_row0,
                   const int* tile_rows, const int* seq_pos0, const int* seq_row0, act_t* out, int o_stride, int heads,
-                  int kv_heads, int hb, int dim, int vdim, int page, const ScoreArgs& sa) {
+                  int kv_heads, int hb, int dim, int vdim, int page, const ScoreArgs& sa, float* partial) {
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
     cudaError_t e = cudaFuncSetAttribute(scored_attention_kernel<ACC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -555,8 +575,73 @@ int launch_scored(dim3 grid, size_t smem, cudaStream_t stream, const act_t* q, i
   }
   bw::launch_pdl(scored_attention_kernel<ACC>, grid, dim3(kThreads), smem, stream, q, q_stride, kcache, vcache, block_table,
                  max_blocks, tile_seq, tile_row0, tile_rows, seq_pos0, seq_row0, out, o_stride, heads, kv_heads, hb, dim,
-                 vdim, page, sa);
+                 vdim, page, sa, partial);
   return bw::launch_status();
+}
+
+// ---------------------------------------------------------------------------------------
+// Two maps of a result head joined: the spans' records of query heads 2h and 2h + 1 merged in ascending order of the spans, as
+// scored_attention_merge does, then o = a1 - lambda a2, o <- o / sqrt(mean(o^2) + eps) * keep, and the output gate. A warp per
+// row and result head.
+struct DifferenceArgs {
+  const float* partial;  // [n, 2 * heads, spans, vdim + 2]
+  int spans, queries /* n * heads */, heads, vdim;
+  const float* lambda;   // one number
+  float keep, eps;
+  const float* gate;     // row r, head h: gate + r * gate_stride + (h * vdim + d) / gate_group, or null
+  int gate_stride, gate_group;
+  act_t* out;            // [n, heads * vdim]
+};
+
+__device__ __forceinline__ void merge_spans(const float* __restrict__ rec, int spans, int vdim, int lane, float (&acc)[8]) {
+  float m = -INFINITY;
+  for (int s = 0; s < spans; ++s) m = fmaxf(m, rec[static_cast<size_t>(s) * (vdim + 2)]);
+  float l = 0.0f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = 0.0f;
+  for (int s = 0; s < spans; ++s) {
+    const float* r = rec + static_cast<size_t>(s) * (vdim + 2);
+    if (r[0] == -INFINITY) continue;  // a span in which the query saw no key
+    const float f = expf(__fsub_rn(r[0], m));
+    l = __fmaf_rn(r[1], f, l);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int d = i * 32 + lane;
+      if (d < vdim) acc[i] = __fmaf_rn(r[2 + d], f, acc[i]);
+    }
+  }
+  const float inv = __fdiv_rn(1.0f, l);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = __fmul_rn(acc[i], inv);
+}
+
+__global__ void __launch_bounds__(128) scored_difference_kernel(const DifferenceArgs a) {
+  bw::pdl_enter();
+  const int qi = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (qi >= a.queries) return;
+  const size_t each = static_cast<size_t>(a.spans) * (a.vdim + 2);
+  float o[8], o2[8];
+  merge_spans(a.partial + 2 * static_cast<size_t>(qi) * each, a.spans, a.vdim, lane, o);
+  merge_spans(a.partial + (2 * static_cast<size_t>(qi) + 1) * each, a.spans, a.vdim, lane, o2);
+  const float lam = a.lambda[0];
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {  // (entries beyond the head are zero)
+    o[i] = __fmaf_rn(-lam, o2[i], o[i]);
+    ss = __fmaf_rn(o[i], o[i], ss);
+  }
+  const float f = __fmul_rn(bw::rms_scale(bw::warp_sum(ss), a.vdim, a.eps), a.keep);
+  const int r = qi / a.heads, h = qi - r * a.heads;
+  const float* gate = a.gate ? a.gate + static_cast<size_t>(r) * a.gate_stride : nullptr;
+  act_t* dst = a.out + static_cast<size_t>(qi) * a.vdim;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int d = i * 32 + lane;
+    if (d >= a.vdim) continue;
+    float v = __fmul_rn(o[i], f);
+    if (gate) v = __fdiv_rn(v, __fadd_rn(1.0f, expf(-gate[(h * a.vdim + d) / a.gate_group])));
+    dst[d] = bw::from_f<act_t>(v);
+  }
 }
 
 
@@ -592,9 +677,9 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   __nv_bfloat16* vs_all = vcache ? ks_all + 2 * kMmaKeys * kst : ks_all;  // [2][32][vst]; the keys where values are keys
   const int vst = vcache ? vst_own : kst;
   const int t = blockIdx.x, g = blockIdx.y;
-  const int rep = heads / kv_heads;
+  const int rep = heads / kv_heads, v_heads = kv_heads / sa.maps, gv = g / sa.maps;
   const int zh = blockIdx.z / spans, span = blockIdx.z - zh * spans;  // the block's share of heads and of keys
-  const int h0 = g * rep + zh * hb;
+  const int h0 = first_head(sa, g, rep, zh * hb), hstep = sa.maps;
   const int nh = min(hb, rep - zh * hb);
   const int seq = tile_seq[t], row0 = tile_row0[t], rows = tile_rows[t];
   const int nq = rows * nh;
@@ -606,7 +691,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   const bool ok_a = sr_a < nq, ok_b = sr_b < nq;
   const int pq_a = p0 + (ok_a ? sr_a / nh : 0), pq_b = p0 + (ok_b ? sr_b / nh : 0);
   const int lo_a = first_seen(sa, pq_a), lo_b = first_seen(sa, pq_b);
-  const HeadBias slope_a = head_bias(sa, h0 + sr_a % nh, ok_a), slope_b = head_bias(sa, h0 + sr_b % nh, ok_b);
+  const HeadBias slope_a = head_bias(sa, h0 + sr_a % nh * hstep, ok_a), slope_b = head_bias(sa, h0 + sr_b % nh * hstep, ok_b);
   const int keep = sa.window > 0 ? sa.keep_first : 0;
   // the positions that this warp's queries span: tiles outside are skipped by the whole warp
   const int w_first = min(warp * 16, max(nq - 1, 0)) / nh, w_last = min(warp * 16 + 15, max(nq - 1, 0)) / nh;
@@ -634,7 +719,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     if (k_begin > k_end) {
       // none of the block's queries reaches into this span: records that say so, nothing else
       for (int sr = tid; sr < nq; sr += kMmaWarps * 32) {
-        float* rec = partial + ((static_cast<size_t>(row0 + sr / nh) * heads + h0 + sr % nh) * spans + span) * (vdim + 2);
+        float* rec = partial + ((static_cast<size_t>(row0 + sr / nh) * heads + h0 + sr % nh * hstep) * spans + span) * (vdim + 2);
         rec[0] = -INFINITY, rec[1] = 0.0f;
       }
       return;
@@ -644,7 +729,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   for (int c = tid; c < kMmaRows * dparts; c += kMmaWarps * 32) {
     const int sr = c / dparts, part = c - sr * dparts;
     const bool valid = sr < nq;
-    const __nv_bfloat16* src = valid ? q + static_cast<size_t>(row0 + sr / nh) * q_stride + (h0 + sr % nh) * dim + part * 8 : q;
+    const __nv_bfloat16* src = valid ? q + static_cast<size_t>(row0 + sr / nh) * q_stride + (h0 + sr % nh * hstep) * dim + part * 8 : q;
     bw::copy16_async(bw::smem_addr(qs + sr * kst + part * 8), src, valid);
   }
   bw::copies_commit();
@@ -677,7 +762,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
         const __nv_bfloat16* src = vcache;
         if (have) {
           const int blk = page_shift >= 0 ? kp >> page_shift : kp / page, slot = kp - blk * page;
-          src = vcache + ((static_cast<size_t>(bt[blk]) * kv_heads + g) * page + slot) * vdim + part_v * 8;
+          src = vcache + ((static_cast<size_t>(bt[blk]) * v_heads + gv) * page + slot) * vdim + part_v * 8;
         }
         if (part_v < vparts) bw::copy16_async(bw::smem_addr(vd + kk * vst + part_v * 8), src, have);
       }
@@ -800,13 +885,13 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     // the span's record per query: maximum, sum, weighted values relative to that maximum
     const int colp = 2 * (lane & 3);
     if (ok_a) {
-      float* rec = partial + ((static_cast<size_t>(row0 + sr_a / nh) * heads + h0 + sr_a % nh) * spans + span) * (vdim + 2);
+      float* rec = partial + ((static_cast<size_t>(row0 + sr_a / nh) * heads + h0 + sr_a % nh * hstep) * spans + span) * (vdim + 2);
       if ((lane & 3) == 0) rec[0] = m_a, rec[1] = l_a;
 #pragma unroll
       for (int j = 0; j < VT; ++j) rec[2 + j * 8 + colp] = acc[j][0], rec[2 + j * 8 + colp + 1] = acc[j][1];
     }
     if (ok_b) {
-      float* rec = partial + ((static_cast<size_t>(row0 + sr_b / nh) * heads + h0 + sr_b % nh) * spans + span) * (vdim + 2);
+      float* rec = partial + ((static_cast<size_t>(row0 + sr_b / nh) * heads + h0 + sr_b % nh * hstep) * spans + span) * (vdim + 2);
       if ((lane & 3) == 0) rec[0] = m_b, rec[1] = l_b;
 #pragma unroll
       for (int j = 0; j < VT; ++j) rec[2 + j * 8 + colp] = acc[j][2], rec[2 + j * 8 + colp + 1] = acc[j][3];
@@ -814,19 +899,19 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     return;
   }
   if (sa.sink) {  // the extra key (score 0 unless the head has a number of its own)
-    const float sk_a = sa.sinks && ok_a ? sa.sinks[h0 + sr_a % nh] : 0.0f, sk_b = sa.sinks && ok_b ? sa.sinks[h0 + sr_b % nh] : 0.0f;
+    const float sk_a = sa.sinks && ok_a ? sa.sinks[h0 + sr_a % nh * hstep] : 0.0f, sk_b = sa.sinks && ok_b ? sa.sinks[h0 + sr_b % nh * hstep] : 0.0f;
     l_a = __fadd_rn(l_a, expf(__fsub_rn(sk_a, m_a))), l_b = __fadd_rn(l_b, expf(__fsub_rn(sk_b, m_b)));
   }
   const float inv_a = __fdiv_rn(1.0f, l_a), inv_b = __fdiv_rn(1.0f, l_b);
   const int col = 2 * (lane & 3);
   if (ok_a) {
-    __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_a / nh) * o_stride + (h0 + sr_a % nh) * vdim + col;
+    __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_a / nh) * o_stride + (h0 + sr_a % nh * hstep) * vdim + col;
 #pragma unroll
     for (int j = 0; j < VT; ++j)
       *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][0], inv_a), __fmul_rn(acc[j][1], inv_a));
   }
   if (ok_b) {
-    __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_b / nh) * o_stride + (h0 + sr_b % nh) * vdim + col;
+    __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_b / nh) * o_stride + (h0 + sr_b % nh * hstep) * vdim + col;
 #pragma unroll
     for (int j = 0; j < VT; ++j)
       *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][2], inv_b), __fmul_rn(acc[j][3], inv_b));
@@ -909,7 +994,7 @@ BW_API int BW_FN(qkv_prepare)(const float* u, int cols, const float* conv_w, con
                               const int* seq_slot, const int* block_table, int max_blocks, void* kcache, void* vcache,
                               void* q_out, int n, int heads, int kv_heads, int dim, int vdim, int page,
                               const float* bias, const float* vmix_src, const float* vmix_lambda, float* v_keep,
-                              int u_stride, int half_layout, cudaStream_t stream) {
+                              int u_stride, int half_layout, int v_heads, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (u_stride < cols) {
     bw::set_error("qkv_prepare: rows %d floats apart do not hold %d columns", u_stride, cols);
@@ -932,7 +1017,7 @@ BW_API int BW_FN(qkv_prepare)(const float* u, int cols, const float* conv_w, con
   a.pos = pos, a.row_seq = row_seq, a.seq_row0 = seq_row0, a.seq_pos0 = seq_pos0, a.seq_slot = seq_slot;
   a.block_table = block_table, a.max_blocks = max_blocks;
   a.kcache = static_cast<act_t*>(kcache), a.vcache = static_cast<act_t*>(vcache), a.q_out = static_cast<act_t*>(q_out);
-  a.heads = heads, a.kv_heads = kv_heads, a.v_heads = vcache ? kv_heads : 0, a.dim = dim, a.vdim = vdim, a.page = page;
+  a.heads = heads, a.kv_heads = kv_heads, a.v_heads = vcache ? v_heads : 0, a.dim = dim, a.vdim = vdim, a.page = page;
   const int total = heads + kv_heads + a.v_heads;
   // four entries per lane where every head and row starts on 16 bytes (and the taps came transposed)
   const bool by_four = dim % 4 == 0 && vdim % 4 == 0 && cols % 4 == 0 && u_stride % 4 == 0 && (!conv_w || conv_wt) &&
@@ -970,11 +1055,13 @@ BW_API int BW_FN(scored_attention)(const void* q, int q_stride, const void* kcac
                                    const int* tile_rows, int tiles, const int* seq_pos0, const int* seq_row0, void* out,
                                    int o_stride, int heads, int kv_heads, int dim, int vdim, int page, float scale,
                                    float softcap, int sink, const float* slopes, int window, const float* dist_a,
-                                   const float* dist_b, const float* sinks, int keep_first, int chunk,
-                                   cudaStream_t stream) {
+                                   const float* dist_b, const float* sinks, int keep_first, int chunk, int maps,
+                                   float* partial, cudaStream_t stream) {
+  // maps > 1: kv_heads key heads, of which `maps` neighbours share a value head. partial: [n, heads, vdim + 2] records for
+  // scored_difference instead of `out`.
   if (tiles <= 0) return 0;
-  if (kv_heads <= 0 || heads % kv_heads) {
-    bw::set_error("scored_attention: %d heads on %d key/value heads", heads, kv_heads);
+  if (kv_heads <= 0 || heads % kv_heads || maps <= 0 || kv_heads % maps || (maps > 1 && !vcache)) {
+    bw::set_error("scored_attention: %d heads on %d key/value heads, %d maps", heads, kv_heads, maps);
     return -1;
   }
   const int acc = (vdim + 31) / 32;
@@ -993,7 +1080,7 @@ BW_API int BW_FN(scored_attention)(const void* q, int q_stride, const void* kcac
   ScoreArgs sa;
   sa.scale = scale, sa.softcap = softcap, sa.sink = sink, sa.slopes = slopes, sa.window = window;
   sa.dist_a = dist_a, sa.dist_b = dist_a ? dist_b : nullptr, sa.sinks = sinks, sa.keep_first = window > 0 ? keep_first : 0;
-  sa.chunk = chunk;
+  sa.chunk = chunk, sa.maps = maps;
   sa.cap_exp = 0.0f;  // (the tensor-core kernel's)
   const dim3 grid(tiles, kv_heads, (rep + hb - 1) / hb);
 #define BW_SCORED(A)                                                                                                      \
@@ -1001,7 +1088,7 @@ BW_API int BW_FN(scored_attention)(const void* q, int q_stride, const void* kcac
     return launch_scored<A>(grid, smem, stream, static_cast<const act_t*>(q), q_stride, static_cast<const act_t*>(kcache), \
                             static_cast<const act_t*>(vcache), block_table, max_blocks, tile_seq, tile_row0, tile_rows,   \
                             seq_pos0, seq_row0, static_cast<act_t*>(out), o_stride, heads, kv_heads, hb, dim, vdim, page, \
-                            sa);
+                            sa, partial);
   switch (acc) {
     BW_SCORED(1) BW_SCORED(2) BW_SCORED(3) BW_SCORED(4) BW_SCORED(5) BW_SCORED(6) BW_SCORED(7) BW_SCORED(8)
   }
@@ -1030,13 +1117,15 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
                                         int o_stride, int heads, int kv_heads, int dim, int vdim, int page, float scale,
                                         float softcap, int sink, const float* slopes, int window, int n, int spans,
                                         float* partial, const float* dist_a, const float* dist_b, const float* sinks,
-                                        int keep_first, int chunk, cudaStream_t stream) {
+                                        int keep_first, int chunk, int maps, cudaStream_t stream) {
+  // maps > 1 (maps as for scored_attention): the spans' records (one span at least) stay in `partial` for scored_difference.
   // spans > 1 (`partial` holding n * heads * spans * (vdim + 2) floats): every query's keys are spread
   // over blocks of kSpanTiles key tiles each, at fixed absolute positions, and a second kernel joins
   // the spans' records in ascending order.
   if (tiles <= 0) return 0;
-  if (kv_heads <= 0 || heads % kv_heads || !bw_bf16_scored_attention_mma_tile_rows(heads / kv_heads, dim, vdim)) {
-    bw::set_error("scored_attention (tensor cores): %d heads on %d, sizes %d / %d", heads, kv_heads, dim, vdim);
+  if (kv_heads <= 0 || heads % kv_heads || maps <= 0 || kv_heads % maps || (maps > 1 && (!vcache || !partial)) ||
+      !bw_bf16_scored_attention_mma_tile_rows(heads / kv_heads, dim, vdim)) {
+    bw::set_error("scored_attention (tensor cores): %d heads on %d, %d maps, sizes %d / %d", heads, kv_heads, maps, dim, vdim);
     return -1;
   }
   const int rep = heads / kv_heads;
@@ -1046,9 +1135,9 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
   ScoreArgs sa;
   sa.scale = scale, sa.softcap = softcap, sa.sink = sink, sa.slopes = slopes, sa.window = window;
   sa.dist_a = dist_a, sa.dist_b = dist_a ? dist_b : nullptr, sa.sinks = sinks, sa.keep_first = window > 0 ? keep_first : 0;
-  sa.chunk = chunk;
+  sa.chunk = chunk, sa.maps = maps;
   sa.cap_exp = softcap > 0.0f ? 2.0f * scale / softcap * 1.4426950408889634f : 0.0f;
-  const bool split = spans > 1 && partial != nullptr;
+  const bool split = (spans > 1 || maps > 1) && partial != nullptr;
   if (!split) spans = 1;
   const dim3 grid(tiles, kv_heads, (rep + hb - 1) / hb * spans);
   typedef const __nv_bfloat16* in_t;
@@ -1065,7 +1154,7 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
     BW_SCORED_MMA(8) BW_SCORED_MMA(16)
   }
 #undef BW_SCORED_MMA
-  if (rc != 0 || !split) return rc;
+  if (rc != 0 || !split || maps > 1) return rc;
   bw::launch_pdl(scored_attention_merge_kernel, dim3((n * heads + 3) / 4), dim3(128), 0, stream,
                  static_cast<const float*>(partial), static_cast<__nv_bfloat16*>(out), o_stride, n * heads, heads, vdim, spans, sink, sinks);
   return bw::launch_status();
@@ -1083,3 +1172,21 @@ BW_API int bw_bf16_scored_attention_spans(int max_keys, int reach, int tile_rows
   return near < all ? static_cast<int>(near) : all;
 }
 #endif  // BW_ACT_BF16
+
+// Two maps per head become one output (see scored_difference_kernel). partial: [n, 2 * heads, spans, vdim + 2] records of
+// scored_attention; gate: float32 rows of `gate_stride` floats with heads * vdim / gate_group numbers each, or null.
+BW_API int BW_FN(scored_difference)(const float* partial, int spans, const float* lambda, float keep, float eps,
+                                    const float* gate, int gate_stride, int gate_group, void* out, int n, int heads, int vdim,
+                                    cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (spans <= 0 || heads <= 0 || vdim <= 0 || vdim > 256 || gate_group <= 0) {
+    bw::set_error("scored_difference: %d spans, %d heads of %d (up to 256)", spans, heads, vdim);
+    return -1;
+  }
+  DifferenceArgs a;
+  a.partial = partial, a.spans = spans, a.queries = n * heads, a.heads = heads, a.vdim = vdim, a.lambda = lambda;
+  a.keep = keep, a.eps = eps, a.gate = gate, a.gate_stride = gate_stride, a.gate_group = gate_group;
+  a.out = static_cast<act_t*>(out);
+  bw::launch_pdl(scored_difference_kernel, dim3((a.queries + 3) / 4), dim3(128), 0, stream, a);
+  return bw::launch_status();
+}

@@ -1,4 +1,4 @@
-// Mixers whose memory is one matrix per head: three recurrences over the tokens of a sequence on one
+// Mixers whose memory is one matrix per head: four recurrences over the tokens of a sequence on one
 // kernel, what prepares their operands, and what finishes their outputs. Per head the state S is
 // dim x vdim float32 numbers of a request (zero before its first token):
 //
@@ -7,6 +7,7 @@
 //   bonus    o = (S + diag(u) k v^T)^T q, then S <- diag(w) S + k v^T, w = exp(-exp(z + z0))
 //   memory   m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, the normaliser n alike with
 //            k alone, o = S^T q (divided later by max(|n . q|, e^-m) + 1e-6)
+//   space    S <- a S + k (t v)^T, o = S^T q + D v, with two numbers per token and head: the decay a and the step t
 //
 // The columns of S (one per value channel) do not meet inside a token, so a block walks the rows of one
 // sequence of the step for one head and a few columns, from the state that the request's slot holds.
@@ -26,7 +27,7 @@ namespace {
 constexpr int kThreads = 128;
 constexpr int kWarps = kThreads / 32;
 constexpr int kCols = 2;  // columns of a lane
-enum { kDelta = 0, kBonus = 1, kMemory = 2 };
+enum { kDelta = 0, kBonus = 1, kMemory = 2, kSpace = 3 };
 
 // The serving precision takes the hardware's exponential (relative error about 1e-7 times the exponent's size, far
 // below that of the bfloat16 operands of the products before it).
@@ -57,14 +58,14 @@ struct ScanArgs {
   const float* decay;      // delta: g; bonus: z. Row r, head h: decay + r * decay_stride + h * dim
   int decay_stride;
   const float* decay_bias;  // bonus: z0 [heads * dim]
-  const float* bonus;      // bonus: u [heads * dim]
-  const float* s0;         // delta: beta; memory: the forget gate's projection. Row r, head h: s0 + r * s_stride + h
-  const float* s1;         // delta: q . k, one per query head (h / rep); memory: the input gate's projection, one per head
+  const float* bonus;      // bonus: u [heads * dim]; space: D [heads]
+  const float* s0;         // delta: beta; memory: the forget gate's projection; space: a. Row r, head h: s0 + r * s_stride + h
+  const float* s1;         // delta: q . k, one per query head (h / rep); memory: the input gate's projection; space: t; one per head
   int s_stride;
   const float* s0_bias;    // memory: [heads]
   const float* s1_bias;
   float cap;               // memory: gates are cap * tanh(. / cap)
-  float* state;            // [slots, heads, columns, column]: delta, bonus: vdim columns of dim; memory: vdim + 1
+  float* state;            // [slots, heads, columns, column]: delta, bonus, space: vdim columns of dim; memory: vdim + 1
                            // columns of dim + 4 (the last column is n; entry dim of every column is m)
   float* o;                // [n, heads * vdim]
   float* aux;              // memory: [n, heads, 2]: n . q and m
@@ -106,7 +107,7 @@ template <int MODE, int LP, int V>
 struct Shape {
   static constexpr int CB = kThreads / LP * kCols;  // columns of a block
   static constexpr int DP = LP * 4 * V;      // rows held; those from dim on are zero
-  static constexpr int VECS = MODE == kMemory ? 2 : 3;
+  static constexpr int VECS = MODE == kMemory || MODE == kSpace ? 2 : 3;
   static constexpr int SC = VECS * DP + CB;  // where a token's scalars start
   static constexpr int W = SC + 4;           // a staged token: k | q | decay | values | scalars
   static constexpr int G = LP < 8 ? LP : 8;  // tokens whose outputs are summed together
@@ -157,7 +158,7 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
   const int seq = a.tile_seq[t], row0 = a.tile_row0[t], cnt = a.tile_rows[t];
   const int tid = threadIdx.x;
   const int p = tid & (LP - 1), col = tid / LP * kCols;  // this lane's rows and its first column in the block
-  constexpr bool kMem = MODE == kMemory;
+  constexpr bool kMem = MODE == kMemory, kRowScalars = kMem || MODE == kSpace;
   const int cols = kMem ? vdim + 1 : vdim, col_size = kMem ? dim + 4 : dim;
   float* head_state = a.state + (static_cast<size_t>(a.seq_slot[seq]) * a.heads + h) * cols * col_size;
   float* sp = head_state + static_cast<size_t>(c0 + col) * col_size;
@@ -250,7 +251,7 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
       for (int tt = tid; tt < len; tt += kThreads) {
         const size_t r = static_cast<size_t>(row0 + first + tt);
         copy4_async(buf + tt * T::W + T::SC, a.s0 + r * a.s_stride + h);
-        copy4_async(buf + tt * T::W + T::SC + 1, a.s1 + r * a.s_stride + (kMem ? h : kh));
+        copy4_async(buf + tt * T::W + T::SC + 1, a.s1 + r * a.s_stride + (kRowScalars ? h : kh));
       }
     }
     bw::copies_commit();
@@ -258,7 +259,7 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
   auto load = [&](const float* tok) -> Token<V> {
     Token<V> x;
     x.k = load_rows<LP, V>(tok, p), x.q = load_rows<LP, V>(tok + T::DP, p);
-    if (!kMem) x.d = load_rows<LP, V>(tok + 2 * T::DP, p);
+    if (!kRowScalars) x.d = load_rows<LP, V>(tok + 2 * T::DP, p);
 #pragma unroll
     for (int j = 0; j < kCols; ++j) x.v[j] = tok[T::VECS * T::DP + col + j];
     x.s0 = MODE == kBonus ? 0.0f : tok[T::SC], x.s1 = MODE == kBonus ? 0.0f : tok[T::SC + 1];
@@ -301,7 +302,7 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
           }
           o[j] = dot<V>(x.q, seen);
         } else {
-          const float add = __fmul_rn(x.s1, c0 + col + j == vdim ? 1.0f : x.v[j]);  // (the normaliser's column takes ones)
+          const float add = __fmul_rn(x.s1, kMem && c0 + col + j == vdim ? 1.0f : x.v[j]);  // (the normaliser's column takes ones)
 #pragma unroll
           for (int i = 0; i < 4 * V; ++i) S[j].v[i] = __fmaf_rn(x.k.v[i], add, __fmul_rn(x.s0, S[j].v[i]));
           o[j] = dot<V>(x.q, S[j]);
@@ -404,11 +405,14 @@ __global__ void __launch_bounds__(kThreads) state_scan_kernel(const ScanArgs a) 
     }
     __syncthreads();
     const int cc = c0 + tid % T::CB;
+    const float skip = MODE == kSpace ? a.bonus[h] : 0.0f;
     for (int i = tid; i < len * T::CB; i += kThreads) {
       const int ti = i / T::CB;
       const size_t r = static_cast<size_t>(row0 + first + ti);
       if (cc < vdim) {
-        a.o[r * a.heads * vdim + h * vdim + cc] = outs[i];
+        const float o = outs[i];
+        a.o[r * a.heads * vdim + h * vdim + cc] =
+            MODE == kSpace ? __fmaf_rn(skip, buf[ti * T::W + T::VECS * T::DP + tid % T::CB], o) : o;
       } else if (kMem && cc == vdim) {
         float* x = a.aux + (r * a.heads + h) * 2;
         x[0] = outs[i], x[1] = buf[ti * T::W + T::SC + 2];
@@ -638,6 +642,148 @@ __global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const DeltaPrep
   }
 }
 
+// What the state-space recurrence reads, row by row. The columns conv0 .. conv0 + channels - 1 of a projected row pass a causal
+// convolution over time (a bias per channel; inputs before the step's first row of a sequence from the request's state, zeros
+// before position 0) and SiLU; the columns step0 .. step0 + heads - 1 become steps t = ln(1 + e^(z + bias_h)) and decays
+// e^(-rate_h t). With `keep` (steps of one row per sequence) the state is brought up to date here as well.
+struct SpacePrepArgs {
+  const float* u;         // [n, u_stride]
+  int u_stride, conv0, channels, step0, heads;
+  const float* conv_t;    // [taps, channels]
+  const float* conv_b;    // [channels]
+  int taps;
+  float* conv_state;      // [slots, taps - 1, channels] or null
+  int keep;
+  const float* dt_bias;   // [heads]
+  const float* rate;      // [heads]
+  float* out;             // [n, out_stride]: the channels, from out_step on the heads' steps, then their decays
+  int out_stride, out_step;
+  const int* pos;
+  const int* row_seq;
+  const int* seq_row0;
+  const int* seq_slot;
+  int n;
+};
+
+// A thread walks VEC neighbouring channels down ROWS rows; with TAPS > 0 (their number known) the inputs of the rows before
+// stay in registers as long as the sequence goes on, else every tap's input is fetched. The order of a channel's sum is the
+// taps', either way. The blocks behind those of the channels form the steps.
+template <int VEC, int TAPS, int ROWS>
+__global__ void __launch_bounds__(kThreads) space_prepare_kernel(const SpacePrepArgs a, int conv_blocks) {
+  bw::pdl_enter();
+  typedef typename VecOf<VEC>::type vec_t;
+  const int r0 = blockIdx.x * ROWS, end = min(r0 + ROWS, a.n);
+  if (static_cast<int>(blockIdx.y) >= conv_blocks) {
+    const int h = (blockIdx.y - conv_blocks) * kThreads + threadIdx.x;
+    if (h >= a.heads) return;
+    const float bias = a.dt_bias[h], rate = a.rate[h];
+    for (int r = r0; r < end; ++r) {
+      float* to = a.out + static_cast<size_t>(r) * a.out_stride + a.out_step + h;
+      const float t = softplus_f(__fadd_rn(a.u[static_cast<size_t>(r) * a.u_stride + a.step0 + h], bias));
+      to[0] = t, to[a.heads] = expf(-__fmul_rn(rate, t));
+    }
+    return;
+  }
+  const int c = (blockIdx.y * kThreads + threadIdx.x) * VEC;
+  if (c >= a.channels) return;
+  const vec_t bias = *reinterpret_cast<const vec_t*>(a.conv_b + c);
+  constexpr int KEPT = TAPS > 0 ? TAPS : 1;
+  vec_t x[KEPT], w[KEPT];  // the inputs that a row's taps see, the row's own last
+#pragma unroll
+  for (int t = 0; t < TAPS; ++t) w[t] = *reinterpret_cast<const vec_t*>(a.conv_t + static_cast<size_t>(t) * a.channels + c);
+  const float* u = a.u + a.conv0 + c;
+  int seq_before = -1;
+  for (int r = r0; r < end; ++r) {
+    const int p = a.pos[r], seq = a.row_seq[r], row0 = a.seq_row0[seq];
+    float* st = a.conv_state ? a.conv_state + static_cast<size_t>(a.seq_slot[seq]) * (a.taps - 1) * a.channels + c : nullptr;
+    auto input = [&](int back) -> vec_t {  // the input `back` rows before this one
+      if (p - back < 0) return vec_t{};
+      return *reinterpret_cast<const vec_t*>(r - back >= row0 ? u + static_cast<size_t>(r - back) * a.u_stride
+                                                              : st + static_cast<size_t>(a.taps - 1 - (row0 - (r - back))) * a.channels);
+    };
+    vec_t sum = bias;
+    float* sf = reinterpret_cast<float*>(&sum);
+    auto add = [&](const vec_t& wt, const vec_t& xt) {
+      const float* xf = reinterpret_cast<const float*>(&xt);
+      const float* wf = reinterpret_cast<const float*>(&wt);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sf[e] = __fmaf_rn(wf[e], xf[e], sf[e]);
+    };
+    if (TAPS > 0) {
+      if (seq == seq_before) {
+#pragma unroll
+        for (int t = 0; t < TAPS - 1; ++t) x[t] = x[t + 1];
+      } else {
+#pragma unroll
+        for (int t = 0; t < TAPS - 1; ++t) x[t] = input(TAPS - 1 - t);
+      }
+      x[KEPT - 1] = input(0);
+#pragma unroll
+      for (int t = 0; t < TAPS; ++t) add(w[t], x[t]);
+      if (a.keep && st) {  // the sequence's only row: the inputs move up by one
+#pragma unroll
+        for (int t = 1; t < TAPS; ++t) *reinterpret_cast<vec_t*>(st + static_cast<size_t>(t - 1) * a.channels) = x[t];
+      }
+      seq_before = seq;
+    } else {
+      for (int t = 0; t < a.taps; ++t) {
+        const vec_t xt = input(a.taps - 1 - t);
+        add(*reinterpret_cast<const vec_t*>(a.conv_t + static_cast<size_t>(t) * a.channels + c), xt);
+        if (a.keep && st && t >= 1) *reinterpret_cast<vec_t*>(st + static_cast<size_t>(t - 1) * a.channels) = xt;
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sf[e] = __fmul_rn(sf[e], sigmoid_f(sf[e]));
+    *reinterpret_cast<vec_t*>(a.out + static_cast<size_t>(r) * a.out_stride + c) = sum;
+  }
+}
+
+// What follows the state-space recurrence: y = o * g sigmoid(g), then every one of the row's `groups` equal parts divided by
+// sqrt(mean(y^2) + eps) of its own, times w. A block per row and part.
+template <int VEC>
+__global__ void __launch_bounds__(256)
+gated_group_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int gate_stride, const float* __restrict__ w,
+                        float eps, act_t* out, int width, int size) {
+  bw::pdl_enter();
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[32];
+  typedef typename VecOf<VEC>::type vec_t;
+  const int first = blockIdx.y * size;
+  const float* src = o + static_cast<size_t>(blockIdx.x) * width + first;
+  const float* g = gate + static_cast<size_t>(blockIdx.x) * gate_stride + first;
+  act_t* dst = out + static_cast<size_t>(blockIdx.x) * width + first;
+  float ss = 0.0f;
+  for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {
+    vec_t v = *reinterpret_cast<const vec_t*>(src + i);
+    const vec_t z = *reinterpret_cast<const vec_t*>(g + i);
+    float* vf = reinterpret_cast<float*>(&v);
+    const float* zf = reinterpret_cast<const float*>(&z);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      vf[e] = __fmul_rn(vf[e], __fmul_rn(zf[e], sigmoid_f(zf[e])));
+      ss = __fmaf_rn(vf[e], vf[e], ss);
+    }
+    *reinterpret_cast<vec_t*>(row + i) = v;
+  }
+  const float inv = bw::rms_scale(bw::block_sum(ss, red), size, eps);
+  for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {  // (each thread reads back only what it wrote)
+    float y[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y[e] = bw::rms_apply(row[i + e], inv, w[first + i + e]);
+    if constexpr (VEC == 4) {
+#if BW_ACT_BF16
+      uint2 packed;
+      packed.x = bw::pack_bf16(y[0], y[1]), packed.y = bw::pack_bf16(y[2], y[3]);
+      *reinterpret_cast<uint2*>(dst + i) = packed;
+#else
+      *reinterpret_cast<float4*>(dst + i) = make_float4(y[0], y[1], y[2], y[3]);
+#endif
+    } else {
+      dst[i] = bw::from_f<act_t>(y[0]);
+    }
+  }
+}
+
 // Token shift: mix_s = x + (x' - x) mu_s for `mixes` vectors mu, x' the row before of the same sequence (from the
 // state for the step's first row, zero for a sequence's first token). out: [mixes, n, width], as the products read them.
 // With `keep` (steps of one row per sequence) the state becomes the row.
@@ -746,7 +892,8 @@ bool on16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 }  // namespace
 
 // mode 0: the delta rule (decay = g, s0 = beta, s1 = q . k per query head); 1: the bonus form (decay = z with decay_bias, bonus = u); 2: the matrix memory
-// (s0, s1 = the projections of the forget and the input gate with their biases, cap; aux [n, heads, 2]). q and k
+// (s0, s1 = the projections of the forget and the input gate with their biases, cap; aux [n, heads, 2]); 3: the state-space form (s0 = the
+// decays, s1 = the steps, bonus = D [heads]). q and k
 // rows hold heads / rep heads. o: [n, heads * vdim]. tiles: one per sequence (sequence, first row, rows).
 BW_API int BW_FN(state_scan)(int mode, const float* q, int q_stride, const float* k, int k_stride, const float* v,
                              int v_stride, int rep, const float* decay, int decay_stride, const float* decay_bias,
@@ -773,6 +920,7 @@ BW_API int BW_FN(state_scan)(int mode, const float* q, int q_stride, const float
     case kDelta: return launch_mode<kDelta>(a, tiles, longest, stream);
     case kBonus: return launch_mode<kBonus>(a, tiles, longest, stream);
     case kMemory: return launch_mode<kMemory>(a, tiles, longest, stream);
+    case kSpace: return launch_mode<kSpace>(a, tiles, longest, stream);
   }
   bw::set_error("state_scan: unknown mode %d", mode);
   return -1;
@@ -813,6 +961,75 @@ BW_API int BW_FN(delta_prepare)(const float* u, int u_stride, int beta_col, cons
     bw::launch_pdl(delta_prepare_kernel<4>, grid, dim3(kThreads), 0, stream, a);
   else
     bw::launch_pdl(delta_prepare_kernel<1>, grid, dim3(kThreads), 0, stream, a);
+  return bw::launch_status();
+}
+
+// u's columns: conv0 .. conv0 + channels - 1 into the convolution, step0 .. step0 + heads - 1 the steps' projections. out
+// [n, out_stride]: the channels, from out_step (>= channels) on the heads' steps and their decays.
+BW_API int BW_FN(space_prepare)(const float* u, int u_stride, int conv0, int channels, int step0, int heads, const float* conv_t,
+                                const float* conv_b, int taps, float* conv_state, int keep, const float* dt_bias,
+                                const float* rate, float* out, int out_stride, int out_step, const int* pos, const int* row_seq,
+                                const int* seq_row0, const int* seq_slot, int n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (taps <= 0 || channels <= 0 || heads <= 0 || (taps > 1 && !conv_state)) {
+    bw::set_error("space_prepare: %d channels, %d heads, %d taps (more than one needs the requests' state)", channels, heads, taps);
+    return -1;
+  }
+  SpacePrepArgs a;
+  a.u = u, a.u_stride = u_stride, a.conv0 = conv0, a.channels = channels, a.step0 = step0, a.heads = heads;
+  a.conv_t = conv_t, a.conv_b = conv_b, a.taps = taps, a.conv_state = taps > 1 ? conv_state : nullptr, a.keep = keep;
+  a.dt_bias = dt_bias, a.rate = rate, a.out = out, a.out_stride = out_stride, a.out_step = out_step;
+  a.pos = pos, a.row_seq = row_seq, a.seq_row0 = seq_row0, a.seq_slot = seq_slot, a.n = n;
+  const bool by_four = channels % 4 == 0 && u_stride % 4 == 0 && out_stride % 4 == 0 && conv0 % 4 == 0 && on16(u) && on16(conv_t) &&
+                       on16(conv_b) && on16(conv_state) && on16(out);
+  const int vec = by_four ? 4 : 1;
+  const int conv_blocks = (channels / vec + kThreads - 1) / kThreads;
+  const unsigned blocks = conv_blocks + (heads + kThreads - 1) / kThreads;
+#define BW_SPACE(T, R)                                                                                                      \
+  do {                                                                                                                      \
+    if (by_four) bw::launch_pdl(space_prepare_kernel<4, T, R>, dim3((n + R - 1) / R, blocks), dim3(kThreads), 0, stream, a, conv_blocks); \
+    else bw::launch_pdl(space_prepare_kernel<1, T, R>, dim3((n + R - 1) / R, blocks), dim3(kThreads), 0, stream, a, conv_blocks); \
+  } while (0)
+  // (a step of few rows spreads them over the machine)
+  if (n <= 64) {
+    switch (taps) {
+      case 1: BW_SPACE(1, 1); break;
+      case 2: BW_SPACE(2, 1); break;
+      case 3: BW_SPACE(3, 1); break;
+      case 4: BW_SPACE(4, 1); break;
+      default: BW_SPACE(0, 1);
+    }
+  } else {
+    switch (taps) {
+      case 1: BW_SPACE(1, 4); break;
+      case 2: BW_SPACE(2, 4); break;
+      case 3: BW_SPACE(3, 4); break;
+      case 4: BW_SPACE(4, 4); break;
+      default: BW_SPACE(0, 1);
+    }
+  }
+#undef BW_SPACE
+  return bw::launch_status();
+}
+
+// o: [n, width], gate: float32 rows of gate_stride floats, w: [width], out: [n, width] in the activation type.
+BW_API int BW_FN(gated_group_norm)(const float* o, const float* gate, int gate_stride, const float* w, float eps, void* out, int n,
+                                   int width, int groups, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (groups <= 0 || width <= 0 || width % groups || width / groups > 48 * 1024 / 4 || groups > 65535) {
+    bw::set_error("gated_group_norm: %d columns in %d groups (of at most 12288)", width, groups);
+    return -1;
+  }
+  const int size = width / groups;
+  const bool by_four = size % 4 == 0 && gate_stride % 4 == 0 && on16(o) && on16(gate) && on16(out);
+  const int want = by_four ? size / 4 : size;
+  const int threads = want >= 256 ? 256 : (want + 31) / 32 * 32;
+  const size_t smem = static_cast<size_t>(size) * sizeof(float);
+  act_t* dst = static_cast<act_t*>(out);
+  if (by_four)
+    bw::launch_pdl(gated_group_norm_kernel<4>, dim3(n, groups), dim3(threads), smem, stream, o, gate, gate_stride, w, eps, dst, width, size);
+  else
+    bw::launch_pdl(gated_group_norm_kernel<1>, dim3(n, groups), dim3(threads), smem, stream, o, gate, gate_stride, w, eps, dst, width, size);
   return bw::launch_status();
 }
 

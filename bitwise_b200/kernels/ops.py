@@ -679,6 +679,30 @@ class KernelOps:
         self._pcall("layernorm_residual", _p(d), _p(weight), _p(x), _c_int(n), _c_int(width), _c_float(eps),
                     _p(next_weight), _c_float(next_eps), _p(next_out), self._stream())
 
+    def tanh_norm(self, x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor,
+                  rows: Optional[torch.Tensor] = None, d: Optional[torch.Tensor] = None) -> None:
+        """out[r] = tanh(alpha * x[rows[r]]) * weight + bias (row r without ``rows``), x the float32 stream, out
+        act_dtype, alpha one float32 number.  ``d`` (float32, no ``rows``): x += d first."""
+        n, width = out.shape
+        _need(x, torch.float32, "tanh_norm x", 2)
+        _need(out, self.act_dtype, "tanh_norm out", 2)
+        for t_, count, what in ((alpha, 1, "alpha"), (weight, width, "weight"), (bias, width, "bias")):
+            _need(t_, torch.float32, "tanh_norm " + what)
+            if t_.numel() != count:
+                raise KernelError(f"tanh_norm: {what} does not hold {count} numbers")
+        if x.shape[1] != width or (rows is None and x.shape[0] < n):
+            raise KernelError("tanh_norm: shapes differ")
+        if rows is not None:
+            _need(rows, torch.int32, "tanh_norm rows", 1)
+            if rows.shape[0] < n:
+                raise KernelError("tanh_norm: fewer row indices than outputs")
+        if d is not None:
+            _need(d, torch.float32, "tanh_norm d", 2)
+            if rows is not None or d.shape != x.shape or x.shape != out.shape:
+                raise KernelError("tanh_norm: a residual sum wants every row of the stream")
+        self._pcall("tanh_norm", _p(x), _p(d), _p(alpha), _p(weight), _p(bias), _p(out), _p(rows), _c_int(n), _c_int(width),
+                    self._stream())
+
     def add_rows(self, x: torch.Tensor, d: torch.Tensor) -> None:
         """x += d (float32, same shape)."""
         _need(x, torch.float32, "add_rows x")
@@ -840,24 +864,34 @@ class KernelOps:
                     _p(batch.seq_row0), _p(out), _c_int(out.shape[1]), _c_int(heads), _c_int(rank), _c_int(rot_dim),
                     _c_int(page), _c_int(window), _c_float(scale), _p(sinks), self._stream())
 
+    ROUTE_SCORES = ("sigmoid", "softmax_top", "softmax")
+
     def route(self, logits: torch.Tensor, correction: Optional[torch.Tensor], groups: int, keep: int, top: int,
-              weight_scale: float, chosen: torch.Tensor, weights: torch.Tensor, softmax_top: bool = False) -> None:
+              weight_scale: float, chosen: torch.Tensor, weights: torch.Tensor, softmax_top: bool = False,
+              scoring: Optional[str] = None, group_max: bool = False, sum_eps: Optional[float] = None) -> None:
         """Per row of ``logits`` (float32 [n, experts]): scores sigmoid(z); the ``top`` experts with
         the largest score + correction among the experts of the ``keep`` best of ``groups`` equal
         groups of neighbours (a group counts as the sum of its two largest corrected scores);
         chosen int32 [n, top], weights float32 [n, top] = score * weight_scale.  ``softmax_top``: the choice
         is by the logits themselves (plus the correction) and the weights are the softmax over the chosen
-        logits only, times weight_scale."""
+        logits only, times weight_scale.  ``scoring`` names the kind instead (of ROUTE_SCORES); "softmax": the scores
+        are the softmax over all experts.  ``group_max``: a group counts as its largest choice score alone.
+        ``sum_eps``: the weights are the chosen scores divided by (their sum + sum_eps), times weight_scale.  The
+        rows of ``logits`` may be columns of wider rows."""
         n, experts = logits.shape
-        _need(logits, torch.float32, "route logits", 2)
+        scoring = scoring or ("softmax_top" if softmax_top else "sigmoid")
+        if scoring not in self.ROUTE_SCORES or (sum_eps is not None and (scoring == "softmax_top" or sum_eps < 0)):
+            raise KernelError(f"route: scores {scoring!r}, weights over their sum + {sum_eps!r}")
+        _need_rows(logits, torch.float32, "route logits")
         _need(chosen, torch.int32, "route chosen", 2)
         _need(weights, torch.float32, "route weights", 2)
         if correction is not None:
             _need(correction, torch.float32, "route correction", 1)
         if tuple(chosen.shape) != (n, top) or tuple(weights.shape) != (n, top):
             raise KernelError("route: outputs are not [rows, top]")
-        self._pcall("route", _p(logits), _p(correction), _c_int(n), _c_int(experts), _c_int(groups), _c_int(keep),
-                    _c_int(top), _c_float(weight_scale), _c_int(int(bool(softmax_top))), _p(chosen), _p(weights),
+        self._pcall("route", _p(logits), _c_int(logits.stride(0)), _p(correction), _c_int(n), _c_int(experts), _c_int(groups),
+                    _c_int(keep), _c_int(top), _c_float(weight_scale), _c_int(self.ROUTE_SCORES.index(scoring)),
+                    _c_int(int(bool(group_max))), _c_float(-1.0 if sum_eps is None else sum_eps), _p(chosen), _p(weights),
                     self._stream())
 
     def group_rows(self, chosen: torch.Tensor, experts: int, group_off: torch.Tensor, tile_prefix: torch.Tensor,
@@ -895,14 +929,18 @@ class KernelOps:
 
     def grouped_linear(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows: int, x_group_cols: int = 0,
                        o_group_cols: int = 0, lists=None, order_div: int = 1, gather: bool = True,
-                       sorted_x: Optional[torch.Tensor] = None) -> None:
+                       sorted_x: Optional[torch.Tensor] = None, activation: Optional[str] = None) -> None:
         """One product per group with w [groups, n, k].  Without ``lists`` every group g takes rows
         0 .. rows-1: out[r, g * o_group_cols + j] = sum_i x[r, g * x_group_cols + i] w[g, j, i].  With
         ``lists`` = (group_off, tile_prefix, order) from ``group_rows`` entry i of group g reads row
         order[i] // order_div of x (row i when ``gather`` is False) and writes row i of out; ``rows``
         is then the length of the list.  ``sorted_x``: scratch [rows, k] for the gathered rows, used
-        where ``grouped_takes_tiles`` says so."""
+        where ``grouped_takes_tiles`` says so.  ``activation`` "relu2" (out act_dtype): the square of relu of
+        every output, in the product's epilogue."""
         groups, n, k = w.shape
+        if activation not in (None, "relu2") or (activation and out.dtype != self.act_dtype):
+            raise KernelError(f"grouped_linear: activation {activation!r} on {out.dtype} outputs")
+        act = self.OUT_ACTIVATIONS.index(activation)
         _need(x, self.act_dtype, "grouped_linear x", 2)
         _need(w, self.act_dtype, "grouped_linear w", 3)
         if out.dtype not in (torch.float32, self.act_dtype):
@@ -926,14 +964,14 @@ class KernelOps:
                     self.gather_rows(x, order, order_div, sorted_x, rows)
                     src = sorted_x
                 if self.lib.bw_bf16_linear_tc_grouped_usable(_p(src), _p(w), _p(out), _c_int(n), _c_int(k)):
-                    self._call("bw_bf16_linear_tc_grouped", _p(src), _p(w), _p(out), _c_int(int(out.dtype == torch.float32)),
+                    self._call("bw_bf16_linear_tc_grouped", _p(src), _p(w), _p(out), _c_int(1 if out.dtype == torch.float32 else 2 * act),
                                _c_int(rows), _c_int(n), _c_int(k), _p(group_off), _p(tile_prefix[1]), _c_int(groups),
                                self._stream())
                     return
                 x, order, order_div = src, None, 1
         self._pcall("grouped_linear", _p(x), _c_int(x.shape[1]), _c_int(x_group_cols), _p(order), _c_int(order_div),
                     _p(w), _p(out), _c_int(int(out.dtype == torch.float32)), _c_int(out.shape[1]), _c_int(o_group_cols),
-                    _p(group_off), _p(tile_prefix), _c_int(rows), _c_int(groups), _c_int(n), _c_int(k), self._stream())
+                    _p(group_off), _p(tile_prefix), _c_int(rows), _c_int(groups), _c_int(n), _c_int(k), _c_int(act), self._stream())
 
     def glu_clamped(self, gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float) -> None:
         """out = g' * sigmoid(alpha * g') * (u' + 1) for rows laid out [gate | up], with
@@ -947,9 +985,11 @@ class KernelOps:
                     self._stream())
 
     def combine(self, x: torch.Tensor, d: Optional[torch.Tensor], y: torch.Tensor, place: torch.Tensor,
-                weights: torch.Tensor, top: int, scale: Optional[torch.Tensor] = None) -> None:
+                weights: torch.Tensor, top: int, scale: Optional[torch.Tensor] = None,
+                d_gate: Optional[torch.Tensor] = None) -> None:
         """x[r] += d[r] + sum_j weights[r, j] * y[place[r * top + j]] (float32; d may be None); with ``scale``
-        [width] what is added is multiplied by it column by column first."""
+        [width] what is added is multiplied by it column by column first.  ``d_gate`` (float32 [n, 1], may be a
+        column of wider rows): d[r] is multiplied by sigmoid(d_gate[r]) first."""
         n, width = x.shape
         _need(x, torch.float32, "combine x", 2)
         _need(y, torch.float32, "combine y", 2)
@@ -963,8 +1003,12 @@ class KernelOps:
             _need(scale, torch.float32, "combine scale", 1)
             if scale.shape[0] != width:
                 raise KernelError("combine: one factor per column is needed")
+        if d_gate is not None:
+            _need_rows(d_gate, torch.float32, "combine d_gate")
+            if d is None or tuple(d_gate.shape) != (n, 1):
+                raise KernelError("combine: one gate number per row of d is needed")
         self._pcall("combine", _p(x), _p(d), _p(y), _p(place), _p(weights), _c_int(n), _c_int(top), _c_int(width),
-                    _p(scale), self._stream())
+                    _p(scale), _p(d_gate), _c_int(d_gate.stride(0) if d_gate is not None else 0), self._stream())
 
     # -- element-wise steps of gated designs (their library is loaded at first use) ---------------------
     def _gated_lib(self):
@@ -1111,7 +1155,7 @@ class KernelOps:
                     write_kv_heads: int, dim: int, vdim: int, conv_wt: Optional[torch.Tensor] = None,
                     bias: Optional[torch.Tensor] = None, vmix_src: Optional[torch.Tensor] = None,
                     vmix_lambda: Optional[torch.Tensor] = None, v_keep: Optional[torch.Tensor] = None,
-                    half_layout: bool = False) -> None:
+                    half_layout: bool = False, v_heads: Optional[int] = None) -> None:
         """From the projected rows ``u`` (float32 [n, cols]: ``heads`` query heads of ``dim``, then, when
         ``write_kv_heads`` > 0, that many key heads of ``dim`` and, with ``vcache``, value heads of
         ``vdim``): the convolution over time with ``conv_w`` [cols, taps] (inputs before the step's
@@ -1123,8 +1167,10 @@ class KernelOps:
         channels at a time.  ``bias`` [cols] is added to every projected row first.  ``vmix_src`` (float32 [n,
         kv_heads * vdim]) and ``vmix_lambda`` (one float32): the values become (1 - lambda) v + lambda vmix_src
         before they are stored; ``v_keep`` (same shape) receives the values as stored, in float32.  ``half_layout``:
-        the rotation's pair i is made of entries i and i + pairs of a head instead of 2i and 2i + 1."""
+        the rotation's pair i is made of entries i and i + pairs of a head instead of 2i and 2i + 1.  ``v_heads``: the
+        number of value heads where several key heads share one."""
         n, cols = u.shape
+        v_heads = write_kv_heads if v_heads is None or not write_kv_heads else v_heads
         _need_rows(u, torch.float32, "qkv_prepare u")
         _need(q_out, self.act_dtype, "qkv_prepare q_out", 2)
         _need(block_table, torch.int32, "qkv_prepare block_table", 2)
@@ -1145,14 +1191,14 @@ class KernelOps:
                 if w_.shape[0] != dim:
                     raise KernelError("qkv_prepare: a norm weight is not of the head's size")
         pairs = self._check_tables(cos, sin, dim, "qkv_prepare")
-        want = heads * dim + write_kv_heads * dim + (write_kv_heads * vdim if vcache is not None else 0)
+        want = heads * dim + write_kv_heads * dim + (v_heads * vdim if vcache is not None else 0)
         if cols != want or tuple(q_out.shape) != (n, heads * dim):
             raise KernelError(f"qkv_prepare: rows of {cols} columns do not hold {want}")
         if write_kv_heads and (tuple(kcache.shape[1:]) != (write_kv_heads, kcache.shape[2], dim)):
             raise KernelError("qkv_prepare: key cache is not [pages, kv_heads, page, dim]")
         if vcache is not None:
             _need(vcache, self.act_dtype, "qkv_prepare vcache", 4)
-            if write_kv_heads and tuple(vcache.shape[1:]) != (write_kv_heads, kcache.shape[2], vdim):
+            if write_kv_heads and tuple(vcache.shape[1:]) != (v_heads, kcache.shape[2], vdim):
                 raise KernelError("qkv_prepare: value cache is not [pages, kv_heads, page, vdim]")
         if bias is not None:
             _need(bias, torch.float32, "qkv_prepare bias", 1)
@@ -1161,7 +1207,7 @@ class KernelOps:
         for t_, what in ((vmix_src, "vmix_src"), (v_keep, "v_keep")):
             if t_ is not None:
                 _need(t_, torch.float32, "qkv_prepare " + what, 2)
-                if vcache is None or not write_kv_heads or tuple(t_.shape) != (n, write_kv_heads * vdim):
+                if vcache is None or not write_kv_heads or tuple(t_.shape) != (n, v_heads * vdim):
                     raise KernelError(f"qkv_prepare: {what} is not [rows, kv_heads * vdim] of values that are stored")
         if (vmix_src is None) != (vmix_lambda is None):
             raise KernelError("qkv_prepare: mixing values needs both the other values and the factor")
@@ -1176,7 +1222,7 @@ class KernelOps:
                     _p(batch.seq_pos0), _p(batch.seq_slot), _p(block_table), _c_int(block_table.shape[1]), _p(kcache),
                     _p(vcache if write_kv_heads else None), _p(q_out), _c_int(n), _c_int(heads), _c_int(write_kv_heads),
                     _c_int(dim), _c_int(vdim), _c_int(kcache.shape[2]), _p(bias), _p(vmix_src), _p(vmix_lambda), _p(v_keep),
-                    _c_int(u.stride(0)), _c_int(int(half_layout)), self._stream())
+                    _c_int(u.stride(0)), _c_int(int(half_layout)), _c_int(v_heads), self._stream())
 
     def conv_state_update(self, u: torch.Tensor, state: torch.Tensor, batch, taps: int, seq_tiles) -> None:
         """state[slot of s][i] = the projected row of position end_s - (taps - 1) + i for every sequence s
@@ -1194,7 +1240,8 @@ class KernelOps:
                          block_table: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
                          scale: float, softcap: float, sink: bool, slopes: Optional[torch.Tensor], window: int,
                          batch, dist_a: Optional[torch.Tensor] = None, dist_b: Optional[torch.Tensor] = None,
-                         sinks: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0) -> None:
+                         sinks: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0,
+                         difference: Optional[tuple] = None) -> None:
         """out[r, h] = sum_j p_j v_j over the cached positions j <= pos[r] of row r's sequence (from pos -
         window + 1 on when window > 0) with s_j = (q[r, h] . k_j) * scale, then s_j <- softcap * tanh(s_j /
         softcap) when softcap > 0, then s_j <- s_j - slopes[h] * (pos[r] - j) when slopes are given, and
@@ -1202,8 +1249,24 @@ class KernelOps:
         ``dist_a``, ``dist_b`` [heads]: s_j <- s_j - dist_a[h] * ln(1 + dist_b[h] * (pos[r] - j)) as well.  ``sinks``
         [heads]: with ``sink``, exp(sinks[h]) joins the denominator instead of 1.  ``keep_first``: with a window,
         the keys j < keep_first are seen too.  ``chunk`` > 0 (and no window): only the keys of the row's own chunk of
-        that many positions are seen, j // chunk == pos[r] // chunk."""
+        that many positions are seen, j // chunk == pos[r] // chunk.
+
+        ``difference`` = (lambda, keep, eps, gate, gate_group): two maps per head.  ``heads`` and ``kv_heads`` count the
+        maps (query head 2h + m and key head 2g + m hold map m of heads h and g), the values have kv_heads / 2 heads,
+        and with a1, a2 the two maps' outputs out[r, h] = o / sqrt(mean(o^2) + eps) * keep * sigmoid(gate), o = a1 -
+        lambda a2 (lambda one float32 number; gate float32 rows with one number per ``gate_group`` entries of out, or
+        None); out is [n, heads / 2 * vdim].  No sink then."""
         n = q.shape[0]
+        maps = 1 if difference is None else 2
+        if maps == 2:
+            lam, keep, norm_eps, gate, gate_group = difference
+            _need(lam, torch.float32, "scored_attention lambda")
+            if heads % 2 or kv_heads % 2 or sink or vcache is None or lam.numel() != 1 or vcache.shape[1] != kv_heads // 2:
+                raise KernelError("scored_attention: two maps want an even number of heads, values of their own and no sink")
+            if gate is not None:
+                _need_rows(gate, torch.float32, "scored_attention gate")
+                if gate_group <= 0 or tuple(gate.shape) != (n, heads // 2 * vdim // gate_group):
+                    raise KernelError("scored_attention: the gate's numbers do not fit the heads")
         _need(q, self.act_dtype, "scored_attention q", 2)
         _need(out, self.act_dtype, "scored_attention out", 2)
         _need(kcache, self.act_dtype, "scored_attention kcache", 4)
@@ -1216,7 +1279,7 @@ class KernelOps:
             _need(slopes, torch.float32, "scored_attention slopes", 1)
             if slopes.shape[0] != heads:
                 raise KernelError("scored_attention: one slope per head is needed")
-        if q.shape[1] != heads * dim or tuple(out.shape) != (n, heads * vdim) or kcache.shape[1] != kv_heads or \
+        if q.shape[1] != heads * dim or tuple(out.shape) != (n, heads // maps * vdim) or kcache.shape[1] != kv_heads or \
                 kcache.shape[3] != dim:
             raise KernelError("scored_attention: shapes do not fit the heads")
         if (dist_a is None) != (dist_b is None):
@@ -1228,7 +1291,7 @@ class KernelOps:
                     raise KernelError(f"scored_attention: {what} is not one number per head")
         if chunk and window:
             raise KernelError("scored_attention: chunks or a window, not both")
-        tail = (_p(dist_a), _p(dist_b), _p(sinks), _c_int(int(keep_first)), _c_int(int(chunk or 0)))
+        tail = (_p(dist_a), _p(dist_b), _p(sinks), _c_int(int(keep_first)), _c_int(int(chunk or 0)), _c_int(maps))
         tc_rows = self._scored_mma_rows(heads // kv_heads, dim, vdim)
         if tc_rows and (not hasattr(batch, "tile_sets") or tc_rows in batch.tile_sets):
             # The serving precision's tensor-core kernel.  Contexts beyond 256 keys are walked in spans
@@ -1242,21 +1305,33 @@ class KernelOps:
                 reach = int(chunk or (0 if keep_first else window) or 0)
                 spans = int(self._mixers_lib().bw_bf16_scored_attention_spans(_c_int(batch.max_keys), _c_int(reach),
                                                                               _c_int(tc_rows)))
-                scratch, launches = self._latent_scratch(n * heads * spans * (vdim + 2), q.device), 2
+                launches = 2
+            if launches == 2 or maps == 2:
+                scratch = self._latent_scratch(n * heads * spans * (vdim + 2), q.device)
             self._mcall("scored_attention_mma", _p(q), _c_int(q.shape[1]), _p(kcache), _p(vcache), _p(block_table),
                         _c_int(block_table.shape[1]), _p(t_seq), _p(t_row0), _p(t_rows), _c_int(t_count), _p(batch.seq_pos0),
                         _p(batch.seq_row0), _p(out), _c_int(out.shape[1]), _c_int(heads), _c_int(kv_heads), _c_int(dim),
                         _c_int(vdim), _c_int(kcache.shape[2]), _c_float(scale), _c_float(softcap), _c_int(int(bool(sink))),
                         _p(slopes), _c_int(window), _c_int(n), _c_int(spans), _p(scratch), *tail, self._stream(),
-                        launches=launches)
+                        launches=1 if maps == 2 else launches)
+            if maps == 2:
+                self._join_maps(scratch, spans, lam, keep, norm_eps, gate, gate_group, out, heads // 2, vdim)
             return
         fn = getattr(self._mixers_lib(), f"bw_{self.kind}_scored_attention_tile_rows")
         t_seq, t_row0, t_rows, t_count = batch.query_tiles(int(fn(_c_int(heads // kv_heads))))
+        scratch = self._latent_scratch(n * heads * (vdim + 2), q.device) if maps == 2 else None
         self._mcall("scored_attention", _p(q), _c_int(q.shape[1]), _p(kcache), _p(vcache), _p(block_table),
                     _c_int(block_table.shape[1]), _p(t_seq), _p(t_row0), _p(t_rows), _c_int(t_count), _p(batch.seq_pos0),
                     _p(batch.seq_row0), _p(out), _c_int(out.shape[1]), _c_int(heads), _c_int(kv_heads), _c_int(dim),
                     _c_int(vdim), _c_int(kcache.shape[2]), _c_float(scale), _c_float(softcap), _c_int(int(bool(sink))),
-                    _p(slopes), _c_int(window), *tail, self._stream())
+                    _p(slopes), _c_int(window), *tail, _p(scratch), self._stream())
+        if maps == 2:
+            self._join_maps(scratch, 1, lam, keep, norm_eps, gate, gate_group, out, heads // 2, vdim)
+
+    def _join_maps(self, records, spans: int, lam, keep: float, eps: float, gate, gate_group: int, out, heads: int, vdim: int) -> None:
+        self._mcall("scored_difference", _p(records), _c_int(spans), _p(lam), _c_float(keep), _c_float(eps), _p(gate),
+                    _c_int(gate.stride(0) if gate is not None else 0), _c_int(gate_group if gate is not None else 1), _p(out),
+                    _c_int(out.shape[0]), _c_int(heads), _c_int(vdim), self._stream())
 
     def gla_scan(self, u: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, tau: float, state: torch.Tensor,
                  norm_w: torch.Tensor, eps: float, out: torch.Tensor, heads: int, dim: int, vdim: int, q_scale: float,
@@ -1288,7 +1363,7 @@ class KernelOps:
                     _c_float(q_scale), self._stream(), launches=2)
 
     # -- recurrences over a matrix of state per head (their library is loaded at first use) ---------------
-    SCAN_MODES = ("delta", "bonus", "memory")
+    SCAN_MODES = ("delta", "bonus", "memory", "space")
 
     def _scan_lib(self):
         lib = getattr(self, "_scanlib", None)
@@ -1329,7 +1404,8 @@ class KernelOps:
                    decay_bias: Optional[torch.Tensor] = None, bonus: Optional[torch.Tensor] = None,
                    beta: Optional[torch.Tensor] = None, forget: Optional[torch.Tensor] = None,
                    qk: Optional[torch.Tensor] = None, inp: Optional[torch.Tensor] = None, forget_bias: Optional[torch.Tensor] = None,
-                   inp_bias: Optional[torch.Tensor] = None, cap: float = 0.0, aux: Optional[torch.Tensor] = None) -> None:
+                   inp_bias: Optional[torch.Tensor] = None, cap: float = 0.0, aux: Optional[torch.Tensor] = None,
+                   step: Optional[torch.Tensor] = None, skip: Optional[torch.Tensor] = None) -> None:
         """One recurrence over the rows of every sequence of the step (``seq_tiles``: one tile per sequence), from and
         into ``state`` [slots, *scan_state_shape] (zero at a request's first position); the outputs before their norm
         into ``o`` [n, heads * vdim].  q, k [n, heads' * dim] (heads a multiple of heads'; head h reads head h // (heads
@@ -1341,7 +1417,8 @@ class KernelOps:
           = z0 and ``bonus`` = u [heads * dim];
         * "memory": m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, n alike, o = S^T q; i = cap tanh((inp +
           inp_bias) / cap), f = ln sigmoid(cap tanh((forget + forget_bias) / cap)); ``inp``, ``forget`` [n, heads]; ``aux`` [n,
-          heads, 2] receives n . q and m'."""
+          heads, 2] receives n . q and m';
+        * "space": S <- a S + k (t v)^T, o = S^T q + D v; ``decay`` = a and ``step`` = t [n, heads], ``skip`` = D [heads]."""
         n = q.shape[0]
         if mode not in self.SCAN_MODES:
             raise KernelError(f"state_scan: mode {mode!r}")
@@ -1364,6 +1441,11 @@ class KernelOps:
                 raise KernelError("state_scan: the rows of beta and of q . k must lie equally far apart")
         elif mode == "bonus":
             vectors += [(decay_bias, heads * dim, "decay_bias"), (bonus, heads * dim, "bonus")]
+        elif mode == "space":
+            rows += [(decay, heads, "decay"), (step, heads, "step")]
+            vectors.append((skip, heads, "skip"))
+            if decay is not None and step is not None and decay.stride(0) != step.stride(0):
+                raise KernelError("state_scan: the rows of decays and of steps must lie equally far apart")
         else:
             rows += [(forget, heads, "forget"), (inp, heads, "inp")]
             vectors += [(forget_bias, heads, "forget_bias"), (inp_bias, heads, "inp_bias")]
@@ -1389,8 +1471,9 @@ class KernelOps:
             if t_.numel() != count:
                 raise KernelError(f"state_scan: {what} does not hold {count} numbers")
         t_seq, t_row0, t_rows, t_count = seq_tiles
-        s0 = beta if mode == "delta" else forget if mode == "memory" else None
-        s1 = inp if mode == "memory" else qk if mode == "delta" else None
+        s0, s1 = {"delta": (beta, qk), "memory": (forget, inp), "space": (decay, step)}.get(mode, (None, None))
+        if mode == "space":
+            decay, bonus = None, skip
         self._sccall("state_scan", _c_int(self.SCAN_MODES.index(mode)), _p(q), _c_int(q.stride(0)), _p(k), _c_int(k.stride(0)),
                      _p(v), _c_int(v.stride(0)), _c_int(heads // (q.shape[1] // dim)), _p(decay),
                      _c_int(decay.stride(0) if decay is not None else 0), _p(decay_bias), _p(bonus), _p(s0), _p(s1),
@@ -1450,6 +1533,48 @@ class KernelOps:
                      _c_int(int(keep)), _p(z), _c_int(z.stride(0)), _p(dt_bias), _p(a_log), _p(out), _c_int(out.stride(0)),
                      _p(batch.pos), _p(batch.row_seq), _p(batch.seq_row0), _p(batch.seq_slot), _c_int(n), _c_int(heads),
                      _c_int(kv_heads), _c_int(dim), _c_int(vdim), _c_float(q_scale), self._stream())
+
+    def space_prepare(self, u: torch.Tensor, conv0: int, step0: int, conv_t: torch.Tensor, conv_b: torch.Tensor,
+                      conv_state: Optional[torch.Tensor], dt_bias: torch.Tensor, rate: torch.Tensor, out: torch.Tensor,
+                      out_step: int, batch, keep: bool = False) -> None:
+        """What the state-space recurrence reads.  The columns of ``u`` (float32 rows) from ``conv0`` on, one per channel,
+        pass the convolution over time with ``conv_t`` [taps, channels] and ``conv_b`` [channels] (earlier inputs from
+        ``conv_state`` [slots, taps - 1, channels], zeros before position 0) and SiLU; the columns from ``step0`` on, one per
+        head, become t = ln(1 + e^(z + dt_bias)) and e^(-rate t).  ``out`` (float32 rows) receives the channels, and from
+        ``out_step`` on the heads' t and their decays.  ``keep``: every sequence of the step has one row, and its state is
+        brought up to date here."""
+        n = u.shape[0]
+        _need_rows(u, torch.float32, "space_prepare u")
+        _need_rows(out, torch.float32, "space_prepare out")
+        for t_, dims, what in ((conv_t, 2, "conv_t"), (conv_b, 1, "conv_b"), (dt_bias, 1, "dt_bias"), (rate, 1, "rate")):
+            _need(t_, torch.float32, "space_prepare " + what, dims)
+        taps, channels = conv_t.shape
+        heads = rate.shape[0]
+        if conv_b.shape[0] != channels or dt_bias.shape[0] != heads or u.shape[1] < max(conv0 + channels, step0 + heads) or \
+                out.shape[0] != n or out_step < channels or out.shape[1] < out_step + 2 * heads:
+            raise KernelError("space_prepare: shapes do not fit the channels and heads")
+        if conv_state is not None:
+            _need(conv_state, torch.float32, "space_prepare conv_state", 3)
+            if tuple(conv_state.shape[1:]) != (taps - 1, channels):
+                raise KernelError("space_prepare: the state is not [slots, taps - 1, channels]")
+        self._sccall("space_prepare", _p(u), _c_int(u.stride(0)), _c_int(conv0), _c_int(channels), _c_int(step0), _c_int(heads),
+                     _p(conv_t), _p(conv_b), _c_int(taps), _p(conv_state), _c_int(int(keep)), _p(dt_bias), _p(rate), _p(out),
+                     _c_int(out.stride(0)), _c_int(out_step), _p(batch.pos), _p(batch.row_seq), _p(batch.seq_row0),
+                     _p(batch.seq_slot), _c_int(n), self._stream())
+
+    def gated_group_norm(self, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                         groups: int) -> None:
+        """y = o * silu(gate), then each of the row's ``groups`` equal parts divided by sqrt(mean(y^2) + eps) of its own, times
+        ``weight`` [width].  o float32 [n, width], gate float32 rows (may be columns of wider rows), out act_dtype."""
+        n, width = o.shape
+        _need(o, torch.float32, "gated_group_norm o", 2)
+        _need(weight, torch.float32, "gated_group_norm weight", 1)
+        _need_rows(gate, torch.float32, "gated_group_norm gate")
+        _need(out, self.act_dtype, "gated_group_norm out", 2)
+        if gate.shape != o.shape or out.shape != o.shape or weight.shape[0] != width or groups <= 0 or width % groups:
+            raise KernelError(f"gated_group_norm: {width} columns in {groups} groups, shapes differ")
+        self._sccall("gated_group_norm", _p(o), _p(gate), _c_int(gate.stride(0)), _p(weight), _c_float(eps), _p(out), _c_int(n),
+                     _c_int(width), _c_int(groups), self._stream())
 
     def shift_mix(self, x: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, out: torch.Tensor, batch, keep: bool = False) -> None:
         """out[s, r] = x[r] + (x'[r] - x[r]) * mu[s], x' the row before of the same sequence: from the step, from ``last``

@@ -9,8 +9,9 @@ from .mlp import DenseFFN, SwiGLU
 from .latent_attention import LatentAttention
 from .linear_recurrence import GatedLinearAttention
 from .paired import PairedMixer
-from .state_recurrence import ChannelDelta, MatrixMemory, ShiftedRecurrence
-from .norm import LayerNorm, RMSNorm
-from .rope import HalfRotaryEncoding, LinearScaling, RampScaling, RotaryEncoding, inverse_frequencies
+from .state_recurrence import ChannelDelta, MatrixMemory, ShiftedRecurrence, StateSpace
+from .norm import LayerNorm, RMSNorm, TanhNorm
+from .rope import (HalfRotaryEncoding, LinearScaling, PairRotaryEncoding, RampScaling, RotaryEncoding, WavelengthScaling,
+                   inverse_frequencies)
 from .routed_ffn import ClampedGLU, RoutedFFN
 from .scored_attention import SEQUENCE_TILE, ScoredAttention, distance_slopes

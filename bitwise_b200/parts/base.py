@@ -30,13 +30,15 @@ class PagedKVNeed:
     ``v_dim``: the size of a value where it differs from a key's (None: ``head_dim``); 0 keeps no
     values at all (a mixer whose values are its keys).  ``keep_first``: with a window, the first
     ``keep_first`` positions of a request stay in the cache as well.  ``chunk`` (instead of a window): positions
-    see the positions of their own chunk of ``chunk`` positions only, counted from a request's first."""
+    see the positions of their own chunk of ``chunk`` positions only, counted from a request's first.
+    ``v_heads``: the number of value heads where it differs from the keys' (several key heads that share one)."""
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_dim: Optional[int] = None
     keep_first: int = 0
     chunk: Optional[int] = None
+    v_heads: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -65,7 +67,7 @@ class SlotStateNeed:
 class PagedKVView:
     """The cache of one layer run, as a mixer sees it during a step."""
     k: torch.Tensor            # [pages, kv_heads, page, head_dim]
-    v: Optional[torch.Tensor]  # [pages, kv_heads, page, v_dim]; None where no values are kept
+    v: Optional[torch.Tensor]  # [pages, kv_heads or v_heads, page, v_dim]; None where no values are kept
     block_table: torch.Tensor  # int32 [step sequences, max blocks] of the layer's group
     page_size: int
     writable: bool = True      # False: the run reads another run's cache and stores nothing

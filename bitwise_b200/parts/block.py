@@ -17,6 +17,7 @@ from .base import FeedForward, Mixer, Norm, Part, SlotStateNeed, StepContext
 
 
 class PreNormBlock(Part):
+    """``feed_forward`` None: the layer is its mixer alone (and has no second norm)."""
     graph_safe = True  # kernels only: a step through this part can be captured
 
     def __init__(self, width: int, mixer: Mixer, feed_forward: FeedForward, mixer_norm: Norm, ffn_norm: Norm,
@@ -27,10 +28,11 @@ class PreNormBlock(Part):
         self.names = names  # keys: mixer_norm, mixer, ffn_norm, feed_forward
 
     def _children(self, prefix: str):
-        return [(self.mixer_norm, f"{prefix}.{self.names['mixer_norm']}"),
+        kids = [(self.mixer_norm, f"{prefix}.{self.names['mixer_norm']}"),
                 (self.mixer, f"{prefix}.{self.names['mixer']}"),
                 (self.ffn_norm, f"{prefix}.{self.names['ffn_norm']}"),
                 (self.feed_forward, f"{prefix}.{self.names['feed_forward']}")]
+        return [(p, n) for p, n in kids if p is not None]
 
     def param_specs(self, prefix: str) -> List[ParamSpec]:
         return [s for part, p in self._children(prefix) for s in part.param_specs(p)]
@@ -57,6 +59,8 @@ class PreNormBlock(Part):
         xn = ctx.workspace.rows("normed", ctx.n, self.width, ctx.act_dtype)
         self.mixer_norm.forward(ctx, x, xn)
         self.mixer.forward(ctx, xn, x, cache)
+        if self.feed_forward is None:
+            return
         self.ffn_norm.forward(ctx, x, xn)
         self.feed_forward.forward(ctx, xn, x)
 
@@ -67,10 +71,6 @@ class ParallelBlock(PreNormBlock):
     float32 buffer, the feed-forward adds to it, and the sum goes into the stream; a feed-forward
     that has ``forward_sum`` does the last two in its own last kernel.  ``feed_forward`` None: the
     layer is its mixer alone."""
-
-    def _children(self, prefix: str):
-        kids = super()._children(prefix)
-        return [(p, n) for p, n in kids if p is not None]
 
     def forward(self, ctx: StepContext, x: torch.Tensor, cache) -> None:
         xn = ctx.workspace.rows("normed", ctx.n, self.width, ctx.act_dtype)

@@ -5,7 +5,8 @@ eps) * w with var the mean of the squared deviations.  The statistics are always
 checkpoints, nothing where the tensor carries the norm's own name).  A norm may hold its weight
 around zero (``offset`` 1: the factor is 1 + w) and carry a constant ``gain`` (a model's output
 scale applied with its last norm); both are folded into the 32-bit weight once, when it is loaded:
-the kernels multiply by ``(offset + w) * gain``."""
+the kernels multiply by ``(offset + w) * gain``.  :class:`TanhNorm` computes no statistics: y = tanh(alpha x) w +
+b with a stored number alpha."""
 from __future__ import annotations
 
 from typing import Dict, List, Optional
@@ -93,5 +94,31 @@ class LayerNorm(RMSNorm):
         ctx.ops.layernorm_residual(d, self.weight, self.eps, x, next_weight=nxt.weight, next_eps=nxt.eps, next_out=out)
 
 
+class TanhNorm(Norm):
+    """tanh(alpha * x) * w + b entry by entry: a number ``alpha`` and the vectors w and b, stored as ``<name>.alpha``,
+    ``<name>`` and ``<name>.b``.  Being entry by entry, it can follow a residual sum in that sum's own kernel."""
+    graph_safe = True  # kernels only
+
+    def __init__(self, width: int, suffix: str = ""):
+        self.width, self.suffix = width, suffix
+        self.alpha = self.weight = self.bias = None
+
+    def param_specs(self, prefix: str) -> List[ParamSpec]:
+        return [ParamSpec(prefix + self.suffix, (self.width,), KEEP32, init="ones"),
+                ParamSpec(f"{prefix}.b", (self.width,), KEEP32, init="zeros"),
+                ParamSpec(f"{prefix}.alpha", (), KEEP32, init="ones")]
+
+    def load_params(self, state: Dict[str, torch.Tensor], prefix: str) -> None:
+        self.weight, self.bias = state[prefix + self.suffix], state[f"{prefix}.b"]
+        self.alpha = state[f"{prefix}.alpha"].reshape(1).contiguous()
+
+    def param_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in (self.alpha, self.weight, self.bias))
+
+    def forward(self, ctx: StepContext, x, out, rows=None) -> None:
+        ctx.ops.tanh_norm(x, self.alpha, self.weight, self.bias, out, rows)
+
+
 register_norm("rmsnorm", RMSNorm)
 register_norm("layernorm", LayerNorm)
+register_norm("tanhnorm", TanhNorm)

@@ -156,10 +156,41 @@ class LinearScaling:
         return np.array([base ** (-2.0 * i / dims) / self.factor for i in range(dims // 2)], dtype=np.float64)
 
 
+class WavelengthScaling:
+    """A rescaling by wavelength ``l = 2 pi / f``: frequencies with ``l < original / high`` stay, those with ``l > original
+    / low`` are divided by ``factor``, between the two ``(1 - s) f / factor + s f`` with ``s = (original / l - low) / (high -
+    low)``.  (The rule of ``inverse_frequencies``, in 64-bit throughout.)"""
+
+    def __init__(self, factor: float, low: float, high: float, original: float):
+        if not (factor > 0 and 0 < low <= high and original > 0):
+            raise ValueError("a rescaling by wavelength needs a positive factor and original, and 0 < low <= high")
+        self.factor, self.low, self.high, self.original = float(factor), float(low), float(high), float(original)
+
+    def key(self):
+        return ("wavelength", self.factor, self.low, self.high, self.original)
+
+    def gain(self) -> float:
+        return 1.0
+
+    def frequencies(self, dims: int, base: float) -> np.ndarray:
+        out = np.empty(dims // 2, dtype=np.float64)
+        for i in range(dims // 2):
+            f = base ** (-2.0 * i / dims)
+            turns = self.original * f / (2.0 * math.pi)  # original / l
+            if turns > self.high:
+                out[i] = f
+            elif turns < self.low or self.low == self.high:
+                out[i] = f / self.factor
+            else:
+                s = (turns - self.low) / (self.high - self.low)
+                out[i] = (1.0 - s) * f / self.factor + s * f
+        return out
+
+
 class HalfRotaryEncoding(RotaryEncoding):
     """Tables for a rotation whose pair i is made of entries i and i + dims / 2 of the turned part (the
     kernels are told the layout; the tables are [positions, dims / 2] either way), with an optional
-    :class:`RampScaling` or :class:`LinearScaling`.  Frequencies and angles are formed in 64-bit and rounded once, to the 32-bit
+    :class:`RampScaling`, :class:`LinearScaling` or :class:`WavelengthScaling`.  Frequencies and angles are formed in 64-bit and rounded once, to the 32-bit
     tables that the kernels read; the tables carry the scaling's gain."""
     layout = "half"
 
@@ -195,5 +226,11 @@ class HalfRotaryEncoding(RotaryEncoding):
         self._device_tables = {}
 
 
+class PairRotaryEncoding(HalfRotaryEncoding):
+    """The same tables for pairs of neighbours: pair i is made of entries 2i and 2i + 1."""
+    layout = "pairs"
+
+
 register_position_encoding("rotary", RotaryEncoding)
+register_position_encoding("rotary_pairs", PairRotaryEncoding)
 register_position_encoding("rotary_half", HalfRotaryEncoding)

@@ -27,6 +27,11 @@ On the scores ``s = (q . k) * scale``:
 * ``sink``: one is added to the softmax's denominator (a key of score 0 that has no value);
   ``sink="learned"``: ``exp(sink_h)`` with a learned number per head instead.
 
+``difference``: a head runs two softmaxes, its maps, with a query and a key of ``dim`` entries for either and one value for
+both (the rows of a head's two maps follow each other in the projections).  With ``lambda = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + difference`` (four
+learned vectors of ``dim``, one lambda for the layer) the head's output is ``o = a1 - lambda a2``, then ``o / sqrt(mean(o^2)
++ eps) * (1 - difference)``.  The convolution, norms and rotation run on each map of a head by itself.
+
 ``gate`` ("entry" or "head"): the heads' outputs are multiplied by the sigmoid of a projection of the
 mixer's input, per entry or per head, before the output projection (:class:`OutputGate`).
 
@@ -60,7 +65,7 @@ class ScoredAttention(Mixer):
     stacks_input = True  # ``w_in`` is one product of the mixer's input, and ``forward`` takes its result ready-made
 
     NAMES = {"q": "q", "k": "k", "v": "v", "out": "o", "conv": ".conv", "norm": ".norm", "bias": ".b", "vmix": "vmix",
-             "dist_a": "r1", "dist_b": "r2", "sink": "sink", "gate": "g"}
+             "dist_a": "r1", "dist_b": "r2", "sink": "sink", "gate": "g", "maps": ("lq1", "lk1", "lq2", "lk2")}
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float = 1e-6,
                  conv_taps: int = 0, qk_norm: bool = False, position: Optional[PositionEncoding] = None, rot_dims: int = 0,
@@ -68,7 +73,9 @@ class ScoredAttention(Mixer):
                  window: Optional[int] = None, values_are_keys: bool = False, shares_cache: bool = False,
                  names: Optional[Dict[str, str]] = None, bias: bool = False, distance_log: bool = False,
                  keep_first: int = 0, value_mix: Optional[str] = None, gate: Optional[str] = None,
-                 chunk: Optional[int] = None):
+                 chunk: Optional[int] = None, difference: Optional[float] = None):
+        if difference is not None and (values_are_keys or sink or slopes is not None or distance_log or value_mix):
+            raise NotImplementedError("two maps per head with values that are keys, a sink, a distance term or mixed values")
         if chunk is not None and (window is not None or chunk <= 0):
             raise ValueError("chunks have a positive size and stand instead of a window")
         if heads % kv_heads:
@@ -96,18 +103,20 @@ class ScoredAttention(Mixer):
         self.slopes_host = [float(s) for s in slopes] if slopes is not None else None
         self.values_are_keys, self.shares_cache = values_are_keys, shares_cache
         self.names = dict(self.NAMES, **(names or {}))
-        self.q_cols = heads * dim
-        self.k_cols = 0 if shares_cache else kv_heads * dim
+        self.difference = float(difference) if difference is not None else None
+        self.maps = 1 if difference is None else 2
+        self.q_cols = heads * self.maps * dim
+        self.k_cols = 0 if shares_cache else kv_heads * self.maps * dim
         self.v_cols = 0 if shares_cache or values_are_keys else kv_heads * vdim
         self.cols = self.q_cols + self.k_cols + self.v_cols
         self.w_in = self.w_o = self.conv_w = self.conv_wt = self.q_norm = self.k_norm = self.slopes = None
-        self.b_in = self.dist_a = self.dist_b = self.sinks = self.vmix = None
+        self.b_in = self.dist_a = self.dist_b = self.sinks = self.vmix = self.lam = None
         self.gate = OutputGate(width, heads, vdim, gate, self.names["gate"]) if gate else None
 
     # -- what the cache keeps --------------------------------------------------------------
     def cache_need(self):
-        return PagedKVNeed(self.kv_heads, self.dim, self.window, v_dim=0 if self.values_are_keys else self.vdim,
-                           keep_first=self.keep_first, chunk=self.chunk)
+        return PagedKVNeed(self.kv_heads * self.maps, self.dim, self.window, v_dim=0 if self.values_are_keys else self.vdim,
+                           keep_first=self.keep_first, chunk=self.chunk, v_heads=self.kv_heads if self.maps > 1 else None)
 
     def state_need(self):
         """The convolution's inputs of the last ``taps - 1`` positions, for every channel it runs on."""
@@ -151,6 +160,8 @@ class ScoredAttention(Mixer):
                       ParamSpec(f"{prefix}.{n['dist_b']}", (self.heads,), KEEP32, init="positive")]
         if self.learned_sink:
             specs.append(ParamSpec(f"{prefix}.{n['sink']}", (self.heads,), KEEP32))
+        if self.difference is not None:
+            specs += [ParamSpec(f"{prefix}.{name}", (self.dim,), KEEP32) for name in n["maps"]]
         if self.gate is not None:
             specs += self.gate.param_specs(prefix)
         specs.append(ParamSpec(f"{prefix}.{n['out']}", (self.width, self.heads * self.vdim), MATRIX))
@@ -184,13 +195,17 @@ class ScoredAttention(Mixer):
             self.dist_a, self.dist_b = state[f"{prefix}.{n['dist_a']}"], state[f"{prefix}.{n['dist_b']}"]
         if self.learned_sink:
             self.sinks = state[f"{prefix}.{n['sink']}"]
+        if self.difference is not None:
+            q1, k1, q2, k2 = (state[f"{prefix}.{name}"].double() for name in n["maps"])
+            lam = torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum()) + self.difference
+            self.lam = lam.float().reshape(1).contiguous()
         if self.slopes_host is not None:
             self.slopes = torch.tensor(self.slopes_host, dtype=torch.float32, device=self.w_o.device)
 
     def param_bytes(self) -> int:
         ts = (self.w_in, self.w_o, self.conv_w, None if self.unit_norm else self.q_norm,
               None if self.unit_norm else self.k_norm, self.b_in, self.vmix, self.dist_a, self.dist_b,
-              self.sinks)  # (the transposed taps are a copy)
+              self.sinks, self.lam)  # (the transposed taps are a copy)
         return sum(t.numel() * t.element_size() for t in ts if t is not None)  # (the gate's rows are part of w_in)
 
     # -- one step --------------------------------------------------------------------------
@@ -228,17 +243,22 @@ class ScoredAttention(Mixer):
                 extra["v_keep"] = first
             else:
                 extra["vmix_src"], extra["vmix_lambda"] = first, self.vmix
+        if self.maps > 1:
+            extra["v_heads"] = self.kv_heads
+        heads, kv_heads = self.heads * self.maps, self.kv_heads * self.maps
         ops.qkv_prepare(u, self.conv_w, state.state if state is not None else None, self.q_norm, self.k_norm, self.eps,
-                        cos, sin, ctx, cache.block_table, cache.k, cache.v, q, self.heads,
-                        self.kv_heads if writes else 0, self.dim, self.vdim, conv_wt=self.conv_wt, **extra)
+                        cos, sin, ctx, cache.block_table, cache.k, cache.v, q, heads,
+                        kv_heads if writes else 0, self.dim, self.vdim, conv_wt=self.conv_wt, **extra)
         if state is not None:
             ops.conv_state_update(u, state.state, ctx, self.taps, ctx.query_tiles(SEQUENCE_TILE))
         mixed = ws.rows("scored_mixed", n, self.heads * self.vdim, ctx.act_dtype)
-        ops.scored_attention(q, cache.k, cache.v, cache.block_table, mixed, self.heads, self.kv_heads, self.dim, self.vdim,
+        options = {"chunk": self.chunk} if self.chunk else {}
+        if self.difference is not None:  # the kernel that joins the maps applies the gate as well
+            options["difference"] = (self.lam, 1.0 - self.difference, self.eps, gate_logits, self.gate.group if self.gate else 1)
+        ops.scored_attention(q, cache.k, cache.v, cache.block_table, mixed, heads, kv_heads, self.dim, self.vdim,
                              self.scale, self.softcap or 0.0, self.sink, self.slopes, self.window or 0, ctx,
-                             dist_a=self.dist_a, dist_b=self.dist_b, sinks=self.sinks, keep_first=self.keep_first,
-                             **({"chunk": self.chunk} if self.chunk else {}))
-        if self.gate is not None:
+                             dist_a=self.dist_a, dist_b=self.dist_b, sinks=self.sinks, keep_first=self.keep_first, **options)
+        if self.gate is not None and self.difference is None:
             self.gate.apply(ctx, xn, mixed, gate_logits)
         ops.linear(mixed, self.w_o, x, residual=x if accumulate else None)
 

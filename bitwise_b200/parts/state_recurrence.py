@@ -5,9 +5,12 @@
   k))^T``, ``o = S^T q``.
 * :class:`ShiftedRecurrence`: every projection reads its own mix of the current and the previous row; ``o = (S +
   diag(u) k v^T)^T r``, then ``S <- diag(w) S + k v^T`` with a decay w from the input and a bonus u.
+* :class:`StateSpace`: x, B and C pass a short causal convolution over time and SiLU; per head ``S <- e^(-rate t) S + t B
+  x^T``, ``y = S^T C + D x`` with a step t from the input.
 * :class:`MatrixMemory`: exponential input and forget gates under a running maximum, a normaliser beside S.
 
-In all of them a head's output is divided by its root mean square, times a weight and a gate, and projected by W_o.
+In all of them but the state space a head's output is divided by its root mean square, times a weight and a gate, and
+projected by W_o; the state space's is gated first and normed in equal parts of the row.
 
 The state is float32 and lives in a state slot of the request, as do a convolution's last inputs and the
 previous row.  The projections may run in the activation type; the convolution, decays, gates of the recurrence,
@@ -292,6 +295,84 @@ class MatrixMemory(_StateMixer):
         ops.linear(gated, self.w_o, x, residual=x if accumulate else None)
 
 
+class StateSpace(_StateMixer):
+    """Per head h with vdim values and a state of ``state`` numbers each: ``t = ln(1 + e^(dt + dt_bias_h))``, ``S <- e^(-e^(A_log_h)
+    t) S + t B x^T``, ``y = S^T C + D_h x``.  B and C belong to ``groups`` groups of heads.  One projection gives [z | x | B | C |
+    dt]; x, B and C pass a causal convolution over time with a bias, and SiLU.  The row y is multiplied by ``silu(z)``, each of
+    its ``norm_groups`` equal parts divided by its own root mean square, times a weight, and projected by W_o."""
+
+    NAMES = {"in": "in", "out": "o", "conv": "conv", "conv_bias": "conv.b", "step_bias": "dt_bias", "decay_log": "A_log", "skip": "D",
+             "norm": "norm"}
+
+    def __init__(self, width: int, heads: int, vdim: int, state: int, groups: int, conv_taps: int, norm_groups: int = 1,
+                 eps: float = 1e-6, names: Optional[Dict[str, str]] = None):
+        _check("state space", heads=heads, vdim=vdim, state=state, groups=groups, conv_taps=conv_taps, norm_groups=norm_groups)
+        if heads % groups:
+            raise ValueError(f"{heads} heads are not a multiple of {groups} groups")
+        if heads * vdim % norm_groups:
+            raise ValueError(f"{heads * vdim} entries do not form {norm_groups} equal parts")
+        self.width, self.heads, self.vdim, self.state, self.groups = width, heads, vdim, state, groups
+        self.taps, self.norm_groups, self.eps = conv_taps, norm_groups, float(eps)
+        self.names = dict(self.NAMES, **(names or {}))
+        self.inner = heads * vdim
+        self.channels = self.inner + 2 * groups * state
+        self.step0 = self.inner + self.channels             # where the steps' columns of the projection begin
+        self.w_in = self.conv_t = self.conv_b = self.step_bias = self.rate = self.skip = self.norm = self.w_o = None
+
+    def cache_need(self):
+        """A head's value columns one after the other."""
+        return SlotStateNeed((self.heads, self.vdim, self.state), torch.float32)
+
+    def state_need(self):
+        """The convolution's inputs of the last ``taps - 1`` positions."""
+        return SlotStateNeed((self.taps - 1, self.channels), torch.float32) if self.taps > 1 else None
+
+    def param_specs(self, prefix: str) -> List[ParamSpec]:
+        n = self.names
+        return [ParamSpec(f"{prefix}.{n['in']}", (self.step0 + self.heads, self.width), MATRIX),
+                ParamSpec(f"{prefix}.{n['conv']}", (self.channels, self.taps), KEEP32),
+                ParamSpec(f"{prefix}.{n['conv_bias']}", (self.channels,), KEEP32),
+                ParamSpec(f"{prefix}.{n['step_bias']}", (self.heads,), KEEP32),
+                ParamSpec(f"{prefix}.{n['decay_log']}", (self.heads,), KEEP32),
+                ParamSpec(f"{prefix}.{n['skip']}", (self.heads,), KEEP32, init="ones"),
+                ParamSpec(f"{prefix}.{n['norm']}", (self.inner,), KEEP32, init="ones"),
+                ParamSpec(f"{prefix}.{n['out']}", (self.width, self.inner), MATRIX)]
+
+    def load_params(self, state: Dict[str, torch.Tensor], prefix: str) -> None:
+        t = {k: state[f"{prefix}.{v}"] for k, v in self.names.items()}
+        self.w_in = stacked_rows([t["in"]])
+        self.conv_t, self.conv_b = t["conv"].t().contiguous(), t["conv_bias"]
+        self.step_bias, self.skip, self.norm, self.w_o = t["step_bias"], t["skip"], t["norm"], t["out"]
+        self.rate = torch.exp(t["decay_log"].double()).float()
+
+    def _tensors(self):
+        return (self.w_in, self.conv_t, self.conv_b, self.step_bias, self.rate, self.skip, self.norm, self.w_o)
+
+    def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, cache: SlotStateView,
+                accumulate: bool = True) -> None:
+        """``accumulate`` False: the output is written to ``x`` instead of added to it."""
+        ops, ws, n, H, ch = ctx.ops, ctx.workspace, ctx.n, self.heads, self.channels
+        tiles = ctx.query_tiles(SEQUENCE_TILE)
+        conv_state = cache.beside.state if self.taps > 1 else None
+        u = ws.rows("space_in32", n, self.w_in.shape[0], torch.float32)
+        ops.linear(xn, self.w_in, u)
+        step = _padded(ch)
+        ready = ws.rows("space_ready32", n, _padded(step + 2 * H), torch.float32)
+        keep = one_row_each(ctx)
+        ops.space_prepare(u, self.inner, self.step0, self.conv_t, self.conv_b, conv_state, self.step_bias, self.rate, ready, step, ctx,
+                          keep=keep)
+        if conv_state is not None and not keep:
+            ops.conv_state_update(u[:, self.inner:self.step0], conv_state, ctx, self.taps, tiles)
+        o = ws.rows("scan_out32", n, self.inner, torch.float32)
+        b, c = self.inner, self.inner + self.groups * self.state
+        ops.state_scan("space", ready[:, c:ch], ready[:, b:c], ready[:, :b], cache.state, o, ctx, tiles, H, self.state, self.vdim,
+                       step=ready[:, step:step + H], decay=ready[:, step + H:step + 2 * H], skip=self.skip)
+        gated = ws.rows("scan_gated", n, self.inner, ctx.act_dtype)
+        ops.gated_group_norm(o, u[:, :self.inner], self.norm, self.eps, gated, self.norm_groups)
+        ops.linear(gated, self.w_o, x, residual=x if accumulate else None)
+
+
 register_mixer("channel_delta", ChannelDelta)
+register_mixer("state_space", StateSpace)
 register_mixer("shifted_recurrence", ShiftedRecurrence)
 register_mixer("matrix_memory", MatrixMemory)

@@ -36,7 +36,7 @@ class CpuOps:
 
     def qkv_prepare(self, u, conv_w, conv_state, q_norm, k_norm, eps, cos, sin, ctx, block_table, kcache, vcache, q_out,
                     heads, write_kv_heads, dim, vdim, conv_wt=None, bias=None, vmix_src=None, vmix_lambda=None, v_keep=None,
-                    half_layout=False):
+                    half_layout=False, v_heads=None):
         n, cols = u.shape
         page = kcache.shape[2]
         if bias is not None:
@@ -78,7 +78,7 @@ class CpuOps:
             return
         g = write_kv_heads
         k = finish(y[:, heads * dim:(heads + g) * dim], dim, k_norm)
-        v = y[:, (heads + g) * dim:].reshape(n, g, vdim) if vcache is not None else None
+        v = y[:, (heads + g) * dim:].reshape(n, v_heads or g, vdim) if vcache is not None else None
         if vmix_src is not None:
             lam = float(vmix_lambda[0])
             v = (1.0 - lam) * v + lam * vmix_src.reshape(n, g, vdim)
@@ -106,8 +106,22 @@ class CpuOps:
                     state[slot, j] = old[pos - pos0 + taps - 1]
 
     def scored_attention(self, q, kcache, vcache, block_table, out, heads, kv_heads, dim, vdim, scale, softcap, sink,
-                         slopes, window, ctx, dist_a=None, dist_b=None, sinks=None, keep_first=0, chunk=0):
+                         slopes, window, ctx, dist_a=None, dist_b=None, sinks=None, keep_first=0, chunk=0, difference=None):
         n = q.shape[0]
+        if difference is not None:
+            lam, keep, eps, gate, gate_group = difference
+            maps = []
+            for m in range(2):
+                o = torch.zeros(n, heads // 2 * vdim)
+                self.scored_attention(q.reshape(n, heads, dim)[:, m::2].reshape(n, -1), kcache[:, m::2], vcache, block_table, o, heads // 2,
+                                      kv_heads // 2, dim, vdim, scale, softcap, sink, slopes, window, ctx, keep_first=keep_first, chunk=chunk)
+                maps.append(o.view(n, heads // 2, vdim))
+            o = maps[0] - float(lam) * maps[1]
+            o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * keep).reshape(n, -1)
+            if gate is not None:
+                o = o * torch.sigmoid(gate).repeat_interleave(gate_group, 1)
+            out.copy_(o.to(out.dtype))
+            return
         page = kcache.shape[2]
         grp = heads // kv_heads
         for r in range(n):
@@ -192,7 +206,20 @@ class CpuOps:
         u = gate_up[:, inter:].float().clamp(-limit, limit)
         out.copy_((g * torch.sigmoid(alpha * g) * (u + 1.0)).to(out.dtype))
 
-    def route(self, logits, correction, groups, keep, top, weight_scale, chosen, weights, softmax_top=False):
+    def route(self, logits, correction, groups, keep, top, weight_scale, chosen, weights, softmax_top=False, scoring=None,
+              group_max=False, sum_eps=None):
+        if scoring == "softmax":
+            if correction is not None or not group_max:
+                raise NotImplementedError("the stand-in keeps groups by their largest score")
+            s = torch.softmax(logits, -1)
+            n, experts = s.shape
+            best = torch.sort(s.view(n, groups, -1).max(-1).values, dim=-1, descending=True, stable=True).indices[:, :keep]
+            allowed = torch.zeros(n, groups).scatter_(1, best, 1.0).repeat_interleave(experts // groups, 1) > 0
+            order = torch.sort(s.masked_fill(~allowed, -1.0), dim=-1, descending=True, stable=True).indices[:, :top]
+            w = torch.gather(s, 1, order)
+            chosen.copy_(order.to(torch.int32))
+            weights.copy_((w if sum_eps is None else w / (w.sum(-1, keepdim=True) + sum_eps)) * weight_scale)
+            return
         if groups != 1 or not softmax_top:
             raise NotImplementedError("the stand-in routes by the largest logits only")
         z = logits if correction is None else logits + correction
@@ -207,7 +234,7 @@ class CpuOps:
         place.reshape(-1)[:pairs] = torch.arange(pairs, dtype=torch.int32)
 
     def grouped_linear(self, x, w, out, rows, x_group_cols=0, o_group_cols=0, lists=None, order_div=1, gather=True,
-                       sorted_x=None):
+                       sorted_x=None, activation=None):
         if lists is None:
             # one product per group over the same rows: group g reads the columns g * x_group_cols .. + k of x
             # and writes the columns g * o_group_cols .. + n of out (w: [groups, n, k])
@@ -219,13 +246,13 @@ class CpuOps:
         order = lists[2].reshape(-1)
         for i in range(rows):
             src = x[int(order[i]) // order_div] if gather else x[i]
-            out[i] = (w[int(self._entry_expert[i])].float() @ src.float()).to(out.dtype)
+            out[i] = self._activated(w[int(self._entry_expert[i])].float() @ src.float(), activation).to(out.dtype)
 
-    def combine(self, x, d, y, place, weights, top, scale=None):
+    def combine(self, x, d, y, place, weights, top, scale=None, d_gate=None):
         n = x.shape[0]
         add = (weights[:, :, None] * y[place.reshape(-1).long()[:n * top]].view(n, top, -1)).sum(1)
         if d is not None:
-            add = add + d
+            add = add + (d if d_gate is None else d * torch.sigmoid(d_gate))
         x += add if scale is None else scale * add
 
     def gla_scan(self, u, z, bias, tau, state, norm_w, eps, out, heads, dim, vdim, q_scale, ctx, tiles, scratch=None):
@@ -311,8 +338,39 @@ class CpuOps:
         soft = torch.nn.functional.softplus(z + dt_bias).view(n, heads, dim)
         z.copy_(torch.exp(-torch.exp(a_log).view(1, -1, 1) * soft).reshape(n, -1))
 
+    def space_prepare(self, u, conv0, step0, conv_t, conv_b, conv_state, dt_bias, rate, out, out_step, ctx, keep=False):
+        n, (taps, channels), heads = u.shape[0], conv_t.shape, rate.shape[0]
+        x = u[:, conv0:conv0 + channels]
+        for r in range(n):
+            s = int(ctx.row_seq[r])
+            row0, slot, pos = int(ctx.seq_row0[s]), int(ctx.seq_slot[s]), int(ctx.pos[r])
+            inputs = torch.zeros(taps, channels)
+            for j in range(taps):
+                back = taps - 1 - j
+                if pos - back >= 0:
+                    inputs[j] = x[r - back] if r - back >= row0 else conv_state[slot, taps - 1 - (row0 - (r - back))]
+            y = conv_b + (conv_t * inputs).sum(0)
+            out[r, :channels] = y * torch.sigmoid(y)
+            if keep and conv_state is not None:
+                conv_state[slot] = inputs[1:]
+        t = torch.nn.functional.softplus(u[:, step0:step0 + heads] + dt_bias)
+        out[:, out_step:out_step + heads] = t
+        out[:, out_step + heads:out_step + 2 * heads] = torch.exp(-rate * t)
+
+    def gated_group_norm(self, o, gate, weight, eps, out, groups):
+        n, width = o.shape
+        y = (o * gate * torch.sigmoid(gate)).view(n, groups, -1)
+        y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+        out.copy_((y.reshape(n, width) * weight).to(out.dtype))
+
+    def tanh_norm(self, x, alpha, weight, bias, out, rows=None, d=None):
+        if d is not None:
+            x += d
+        src = x if rows is None else x[rows.long()]
+        out.copy_((torch.tanh(alpha * src) * weight + bias).to(out.dtype))
+
     def state_scan(self, mode, q, k, v, state, o, ctx, tiles, heads, dim, vdim, decay=None, decay_bias=None, bonus=None,
-                   beta=None, qk=None, forget=None, inp=None, forget_bias=None, inp_bias=None, cap=0.0, aux=None):
+                   beta=None, qk=None, forget=None, inp=None, forget_bias=None, inp_bias=None, cap=0.0, aux=None, step=None, skip=None):
         n = q.shape[0]
         rep = heads // (q.shape[1] // dim)
         qh = q.reshape(n, -1, dim).repeat_interleave(rep, 1)
@@ -333,6 +391,9 @@ class CpuOps:
                     S.add_(w[:, :, None] * kh[r][:, None, :])
                     out = torch.einsum("hvd,hd->hv", S, qh[r])
                     assert torch.allclose((q.reshape(n, -1, dim)[r] * k.reshape(n, -1, dim)[r]).sum(-1), qk[r], atol=1e-5)
+                elif mode == "space":
+                    S.mul_(decay[r][:, None, None]).add_(step[r][:, None, None] * kv)
+                    out = torch.einsum("hvd,hd->hv", S, qh[r]) + skip[:, None] * vh[r]
                 elif mode == "bonus":
                     out = torch.einsum("hvd,hd->hv", S + bonus.view(heads, 1, dim) * kv, qh[r])
                     w = torch.exp(-torch.exp(decay[r] + decay_bias)).view(heads, 1, dim)
