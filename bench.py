@@ -1304,6 +1304,227 @@ def compare_zuzupel(args, pk):
     return line
 
 
+# ---- the Sazisun design beside Favudra at equal size (--compare sazisun) ------------------------
+SAZISUN_SIZES = {
+    # width, layers; attention: heads on kv_heads, dim per map, vdim; state space: heads x vdim, state, groups, taps, norm_groups;
+    # experts in groups of which keep stay, top, ff of an expert, of the shared one, of the dense layer; vocab
+    "small": dict(width=1024, layers=4, heads=8, kv_heads=2, dim=64, vdim=128, rot_dims=64, s_heads=32, s_vdim=64, state=128, s_groups=8,
+                  taps=4, norm_groups=8, experts=16, groups=4, keep=2, top=2, ff=704, shared_ff=1408, dense_ff=2816, vocab=32768),
+    "medium": dict(width=2048, layers=4, heads=16, kv_heads=4, dim=64, vdim=128, rot_dims=64, s_heads=64, s_vdim=64, state=128, s_groups=8,
+                   taps=4, norm_groups=8, experts=64, groups=8, keep=4, top=6, ff=1408, shared_ff=2816, dense_ff=5632, vocab=32768),
+}
+
+
+def sazisun_config(z):
+    """Layers in the order state space, attention, state space, attention on the second layer's keys and values, and so on; the
+    first layer with a dense feed-forward, the others with experts."""
+    from bitwise_b200.config import (ExpertsConfig, FeedForwardConfig, SazisunConfig, SazisunLayerConfig, StateSpaceConfig,
+                                     TwoMapAttentionConfig, WavelengthScalingConfig)
+    layers = []
+    for i in range(z["layers"]):
+        if i % 2 == 0:
+            m = StateSpaceConfig(z["s_heads"], z["s_vdim"], z["state"], z["s_groups"], z["taps"], z["norm_groups"])
+        else:
+            m = TwoMapAttentionConfig(z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dim"] ** -0.5, 0.6, 50.0, 5e5, z["rot_dims"],
+                                      WavelengthScalingConfig(8.0, 1.0, 4.0, 8192), kv_from=1 if i % 4 == 3 else None)
+        f = FeedForwardConfig(z["dense_ff"]) if i == 0 else ExpertsConfig(z["ff"], z["experts"], z["top"], 2.5, z["groups"], z["keep"],
+                                                                           z["shared_ff"])
+        layers.append(SazisunLayerConfig(m, f))
+    return SazisunConfig(vocab=z["vocab"], width=z["width"], eps=1e-5, layers=tuple(layers))
+
+
+def sazisun_twin(z):
+    """Favudra with the same width, layers and vocabulary: gated linear attention with the state's heads and sizes where Sazisun
+    has a state space, capped attention with as many heads as Sazisun has maps (the fourth layer on the second's keys and values)
+    where it has two-map attention, and feed-forwards of the dense layer's size."""
+    from bitwise_b200.config import FavudraConfig, FavudraLayerConfig, FavudraMixerConfig
+    layers = []
+    for i in range(z["layers"]):
+        if i % 2 == 0:
+            m = FavudraMixerConfig("gla", z["s_heads"], z["state"], z["s_vdim"], tau=16.0, decay_rank=64)
+        else:
+            m = FavudraMixerConfig("attention", 2 * z["heads"], z["dim"], z["vdim"], kv_heads=2 * z["kv_heads"], scale=z["dim"] ** -0.5,
+                                   conv=z["taps"], rot_base=5e5, rot_dims=z["rot_dims"], softcap=50.0, kv_from=1 if i % 4 == 3 else None)
+        layers.append(FavudraLayerConfig(m, z["dense_ff"]))
+    return FavudraConfig(vocab=z["vocab"], width=z["width"], eps=1e-5, embedding_scale=z["width"] ** 0.5, logit_scale=0.25,
+                         layers=tuple(layers))
+
+
+def sazisun_kernel_table(z, pk, page=16):
+    """Every kernel that the design added or changed, alone at the size's shapes, beside the like kernel of an
+    earlier design: milliseconds and the fraction of its roofline (measured copy bandwidth, bf16 peak, or the CUDA cores'
+    float32 rate for the walk along a prompt)."""
+    import torch
+    from bitwise_b200.kernels.ops import get_ops
+    from bitwise_b200.parts.rope import PairRotaryEncoding, WavelengthScaling
+    from bitwise_b200.parts.scored_attention import SEQUENCE_TILE
+    ops = get_ops("bfloat16")
+    dev, bf = "cuda:0", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    width, taps = z["width"], z["taps"]
+    out = {}
+    fp32 = pk.get("fp32_tflops", 74.0)
+
+    def frac_flops(flops, ms, peak=None):
+        return round(flops / (ms / 1e3) / 1e12 / (peak or pk["bf16_tflops"]), 4)
+
+    def frac_bytes(nbytes, ms):
+        return round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4)
+
+    def put(name, ms, frac, twin_ms, twin_frac, bound, twin):
+        out[name] = {"ms": round(ms, 4), "frac": frac, "twin_ms": round(twin_ms, 4), "twin_frac": twin_frac, "bound": bound,
+                     "twin": twin, "gap_ratio": round(twin_frac / frac, 2) if frac else None}
+
+    rnd = lambda *s: torch.randn(*s, device=dev)
+    ones = lambda *s: torch.ones(*s, device=dev)
+    time_it = lambda fn: timed_device(fn, flush=flush)
+    cos, sin = PairRotaryEncoding(z["rot_dims"], 5e5, WavelengthScaling(8.0, 1.0, 4.0, 8192), positions=2048).rotary_tables(dev)
+    H, G, dim, vdim = z["heads"], z["kv_heads"], z["dim"], z["vdim"]
+    for label, seqs in (("prefill_2048", [(0, 2048)]), ("decode_b8_ctx2048", [(2047, 1)] * 8)):
+        keys = max(p0 + c for p0, c in seqs)
+        blocks = (keys + page - 1) // page
+        nseq = len(seqs)
+        table = torch.arange(nseq * blocks, dtype=torch.int32, device=dev).reshape(nseq, blocks)
+        b = KernelBatch(seqs, sorted(set(ops.scored_attention_tile_heights(H // G, dim, vdim)) | {SEQUENCE_TILE}), dev)
+        b.seq_slot = torch.arange(nseq, dtype=torch.int32, device=dev)
+        n = b.n
+        prefill = n > nseq
+        tiles = b.query_tiles(SEQUENCE_TILE)
+        # two maps and their difference, norm and gate, beside capped attention with as many heads (a value head per key head)
+        kc, vc = rnd(nseq * blocks + 1, 2 * G, page, dim).to(bf), rnd(nseq * blocks + 1, G, page, vdim).to(bf)
+        vc2 = rnd(nseq * blocks + 1, 2 * G, page, vdim).to(bf)
+        q, o1, o2 = rnd(n, 2 * H * dim).to(bf), torch.empty(n, H * vdim, dtype=bf, device=dev), torch.empty(n, 2 * H * vdim, dtype=bf, device=dev)
+        lam, gate = torch.full((1,), 0.6, device=dev), rnd(n, H * vdim)
+        attend = lambda vv, oo, **k: ops.scored_attention(q, kc, vv, table, oo, 2 * H, 2 * G, dim, vdim, dim ** -0.5, 50.0, False, None, 0, b, **k)
+        ms = time_it(lambda: attend(vc, o1, difference=(lam, 0.4, 1e-5, gate, 1)))
+        tms = time_it(lambda: attend(vc2, o2))
+        pairs = sum(sum(p + 1 for p in range(p0, p0 + c)) for p0, c in seqs)
+        if prefill:
+            fl = 2.0 * 2 * H * (dim + vdim) * pairs
+            put(f"two_map_attention_{label}", ms, frac_flops(fl, ms), tms, frac_flops(fl, tms), "bf16 peak", "capped attention, as many heads")
+        else:
+            put(f"two_map_attention_{label}", ms, frac_bytes(pairs * G * (2 * dim + vdim) * 2, ms), tms,
+                frac_bytes(pairs * 2 * G * (dim + vdim) * 2, tms), "copy bandwidth", "capped attention, as many heads")
+        # rotation and store beside convolution, rotation, store
+        cols = 2 * (H + G) * dim + G * vdim
+        tcols = 2 * (H + G) * dim + 2 * G * vdim
+        wide, tu, cw = rnd(n, cols + H * vdim), rnd(n, tcols), rnd(tcols, taps)
+        cwt, st = cw.t().contiguous(), torch.zeros(nseq + 1, taps - 1, tcols, device=dev)
+        ms = time_it(lambda: ops.qkv_prepare(wide[:, :cols], None, None, None, None, 1e-5, cos, sin, b, table, kc, vc, q, 2 * H, 2 * G, dim,
+                                             vdim, v_heads=G))
+        tms = time_it(lambda: (ops.qkv_prepare(tu, cw, st, None, None, 1e-5, cos, sin, b, table, kc, vc2, q, 2 * H, 2 * G, dim, vdim, conv_wt=cwt),
+                               ops.conv_state_update(tu, st, b, taps, tiles)))
+        put(f"rotate_store_{label}", ms, frac_bytes(n * cols * 6, ms), tms, frac_bytes(n * tcols * 6, tms), "copy bandwidth",
+            "convolution, rotation, store")
+        del kc, vc, vc2
+        # the state-space walk and what finishes it beside the bonus form's at the same heads and sizes
+        SH, sv, N, SG = z["s_heads"], z["s_vdim"], z["state"], z["s_groups"]
+        inner, gn = SH * sv, SG * N
+        ch = inner + 2 * gn
+        u, ready = rnd(n, 2 * inner + 2 * gn + SH + (-SH) % 8), torch.rand(n, ch + 2 * SH, device=dev)
+        ct, cb, db, rate = rnd(taps, ch), rnd(ch), rnd(SH), ones(SH)
+        cst = torch.zeros(nseq + 1, taps - 1, ch, device=dev)
+        state, o32 = torch.zeros(nseq + 1, SH, sv, N, device=dev), torch.empty(n, inner, device=dev)
+        og, skip, w = torch.empty(n, inner, dtype=bf, device=dev), ones(SH), ones(inner)
+        scan = lambda: ops.state_scan("space", ready[:, inner + gn:ch], ready[:, inner:inner + gn], ready[:, :inner], state, o32, b, tiles, SH,
+                                      N, sv, step=ready[:, ch:ch + SH], decay=ready[:, ch + SH:], skip=skip)
+        finish = lambda: ops.gated_group_norm(o32, u[:, :inner], w, 1e-5, og, z["norm_groups"])
+        ms, ms_alone = time_it(lambda: (scan(), finish())), time_it(scan)
+        bq, bk, bv, bz, bg = rnd(n, SH * N), rnd(n, SH * N), rnd(n, inner), rnd(n, SH * N), rnd(n, inner)
+        b0, bu = rnd(SH * N), rnd(SH * N)
+        bscan = lambda: ops.state_scan("bonus", bq, bk, bv, state, o32, b, tiles, SH, N, sv, decay=bz, decay_bias=b0, bonus=bu)
+        tms = time_it(lambda: (bscan(), ops.scan_finish(o32, w, bg, 1e-5, og, SH, sv)))
+        per = n * SH * N * sv
+        if prefill:
+            put(f"space_scan_{label}", ms, frac_flops(4.0 * per, ms, fp32), tms, frac_flops(4.0 * per, tms, fp32), "float32 on the CUDA cores",
+                "the bonus form's walk")
+        else:
+            put(f"space_scan_{label}", ms, frac_bytes(8 * per, ms), tms, frac_bytes(8 * per, tms), "copy bandwidth", "the bonus form's walk")
+        out[f"space_scan_{label}"]["scan_alone_ms"] = round(ms_alone, 4)
+        ms, tms = time_it(finish), time_it(lambda: ops.scan_finish(o32, w, bg, 1e-5, og, SH, sv))
+        put(f"gated_group_norm_{label}", ms, frac_bytes(n * inner * 10, ms), tms, frac_bytes(n * inner * 10, tms), "copy bandwidth",
+            "norm per head and gate")
+        # what the state space reads beside what the delta rule reads (its channels and decays)
+        keep = not prefill
+        ms = time_it(lambda: (ops.space_prepare(u, inner, inner + ch, ct, cb, cst, db, rate, ready, ch, b, keep=keep),
+                              None if keep else ops.conv_state_update(u[:, inner:inner + ch], cst, b, taps, tiles)))
+        du, dz, dr = rnd(n, ch + SH), rnd(n, SH * N), torch.empty(n, ch + SH + SG, device=dev)
+        dst, dbb, al = torch.zeros(nseq + 1, taps - 1, ch, device=dev), rnd(SH * N), rnd(SH)
+        tms = time_it(lambda: (ops.delta_prepare(du, ch, ct, dst, dz, dbb, al, dr, b, SH, SG, N, sv, N ** -0.5, keep=keep),
+                               None if keep else ops.conv_state_update(du[:, :ch], dst, b, taps, tiles)))
+        put(f"space_prepare_{label}", ms, frac_bytes(n * ch * 8, ms), tms, frac_bytes(n * (ch + SH * N) * 8, tms), "copy bandwidth",
+            "what the delta rule reads")
+        del u, ready, bq, bk, bv, bz, bg, state, du, dz
+        # the norm without statistics beside the root-mean-square norm
+        x, ww, xn = rnd(n, width), ones(width), torch.empty(n, width, dtype=bf, device=dev)
+        al1, bb = ones(1), rnd(width)
+        ms, tms = time_it(lambda: ops.tanh_norm(x, al1, ww, bb, xn)), time_it(lambda: ops.rmsnorm(x, ww, 1e-5, xn))
+        put(f"tanh_norm_{label}", ms, frac_bytes(n * width * 6, ms), tms, frac_bytes(n * width * 6, tms), "copy bandwidth", "norm")
+        # routing beside sigmoid scores; the experts' products beside gated experts; the combination
+        E, top, ff = z["experts"], z["top"], z["ff"]
+        lg = rnd(n, E + 1 + (-E - 1) % 8)
+        chosen, wts = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+        lists = torch.empty(3, E + 1, dtype=torch.int32, device=dev)
+        order, place = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, dtype=torch.int32, device=dev)
+        group = lambda: ops.group_rows(chosen, E, lists[0], lists[1:3], order, place)
+        ms = time_it(lambda: (ops.route(lg[:, :E], None, z["groups"], z["keep"], top, 2.5, chosen, wts, scoring="softmax", group_max=True,
+                                        sum_eps=1e-20), group()))
+        lg2, corr = lg[:, :E].contiguous(), torch.zeros(E, device=dev)
+        tms = time_it(lambda: (ops.route(lg2, corr, z["groups"], z["keep"], top, 2.5, chosen, wts), group()))
+        put(f"route_{label}", ms, frac_bytes(n * E * 4, ms), tms, frac_bytes(n * E * 4, tms), "launch", "sigmoid scores")
+        ops.route(lg[:, :E], None, z["groups"], z["keep"], top, 2.5, chosen, wts, scoring="softmax", group_max=True, sum_eps=1e-20)
+        group()
+        grouped = (lists[0], lists[1:3], order)
+        pr = n * top
+        xb, w1, w1g = rnd(n, width).to(bf), (rnd(E, ff, width) * 0.02).to(bf), (rnd(E, 2 * ff, width) * 0.02).to(bf)
+        w2 = (rnd(E, width, ff) * 0.02).to(bf)
+        h1, gu, y = torch.empty(pr, ff, dtype=bf, device=dev), torch.empty(pr, 2 * ff, dtype=bf, device=dev), torch.empty(pr, width, device=dev)
+        xs = torch.empty(pr, width, dtype=bf, device=dev)
+        used = len(set(chosen.flatten().tolist()))
+        ms = time_it(lambda: ops.grouped_linear(xb, w1, h1, pr, lists=grouped, order_div=top, sorted_x=xs, activation="relu2"))
+        tms = time_it(lambda: (ops.grouped_linear(xb, w1g, gu, pr, lists=grouped, order_div=top, sorted_x=xs), ops.glu_clamped(gu, h1, 7.0, 1.7)))
+        if prefill:
+            put(f"experts_up_relu2_{label}", ms, frac_flops(2.0 * pr * ff * width, ms), tms, frac_flops(4.0 * pr * ff * width, tms), "bf16 peak",
+                "gated experts' gate/up and activation")
+        else:
+            put(f"experts_up_relu2_{label}", ms, frac_bytes(2.0 * used * ff * width, ms), tms, frac_bytes(4.0 * used * ff * width, tms),
+                "copy bandwidth", "gated experts' gate/up and activation")
+        out[f"experts_up_relu2_{label}"]["experts_used"] = used
+        ops.grouped_linear(h1, w2, y, pr, lists=grouped, gather=False)
+        d = rnd(n, width)
+        ms = time_it(lambda: ops.combine(x, d, y, place, wts, top, d_gate=lg[:, E:E + 1]))
+        tms = time_it(lambda: ops.combine(x, d, y, place, wts, top))
+        by = n * width * 4 * (3 + top)
+        put(f"combine_gated_{label}", ms, frac_bytes(by, ms), tms, frac_bytes(by, tms), "copy bandwidth", "combination without a gate")
+        del w1, w1g, w2
+        torch.cuda.empty_cache()
+    return out
+
+
+def compare_sazisun(args, pk):
+    import torch
+    from bitwise_b200 import Model
+    z = SAZISUN_SIZES[args.size]
+    line = {"metric": f"Sazisun beside Favudra at equal size ({args.size}): prefill of 2,048 tokens and decode at batch "
+                      f"{args.batch}, {args.ctx or 2048:,}-token contexts", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16",
+            "data": "synthetic: random N(0,0.02) weights, prompt ids uniform over the vocabulary", "size": z,
+            "peaks": "of " + pk["source"], "l2": "whole models: weights and cache exceed L2; kernels alone: L2 flushed "
+            "before every repetition"}
+    ctx = args.ctx or 2048
+    for name, cfg in (("sazisun", sazisun_config(z)), ("favudra_twin", sazisun_twin(z))):
+        model = Model.random(cfg, seed=0, dtype="bfloat16", device="cuda:0", fast=True)
+        with ClockSampler() as clocks:
+            ms, launches = run_decode(model, args.batch, ctx, args.steps, max(3, args.warmup), args.page)
+        pms = run_prefill(model, 2048, reps=5, warmup=3, page=args.page)
+        line[name] = {"decode_tok_s": round(args.batch / (ms / 1e3), 1), "decode_ms_per_step": round(ms, 4),
+                      "prefill_tok_s": round(2048 / (pms / 1e3), 1), "prefill_ms": round(pms, 3),
+                      "weight_bytes": model.weight_bytes, "gpu_launches": launches, "clocks": clocks.summary()}
+        del model
+        torch.cuda.empty_cache()
+    line["kernels"] = sazisun_kernel_table(z, pk, args.page)
+    return line
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1322,10 +1543,10 @@ def main():
     ap.add_argument("--page", type=int, default=16)
     ap.add_argument("--skip-points", action="store_true", help="only the headline decode (for profiling runs)")
     ap.add_argument("--skip-prefill", action="store_true")
-    ap.add_argument("--compare", default="", choices=["", "nuderax", "favudra", "sebavik", "kezuvik", "zuzupel"],
+    ap.add_argument("--compare", default="", choices=["", "nuderax", "favudra", "sebavik", "kezuvik", "zuzupel", "sazisun"],
                     help="instead of the headline: this design beside its closest earlier architecture at equal size")
     ap.add_argument("--size", default="small", choices=sorted(set(NUDERAX_SIZES) | set(FAVUDRA_SIZES) | set(SEBAVIK_SIZES) | set(KEZUVIK_SIZES) |
-                                                                set(ZUZUPEL_SIZES)),
+                                                                set(ZUZUPEL_SIZES) | set(SAZISUN_SIZES)),
                     help="layer sizes for --compare")
     args = ap.parse_args()
 
@@ -1351,6 +1572,9 @@ def main():
         return 0
     if args.compare == "zuzupel":
         print(json.dumps(compare_zuzupel(args, pk)))
+        return 0
+    if args.compare == "sazisun":
+        print(json.dumps(compare_sazisun(args, pk)))
         return 0
     if args.compare == "sebavik":
         print(json.dumps(compare_sebavik(args, pk)))
