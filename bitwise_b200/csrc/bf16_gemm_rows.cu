@@ -100,10 +100,18 @@ struct RopeCache {
   int heads, kv_heads, hd, page, write_kv;
 };
 
+// EPI 2: the norm without statistics of the row just summed, formed by the thread that summed the entry.
+struct TanhNormOut {
+  const float* alpha;  // one number
+  const float* w;      // [N]
+  const float* b;      // [N]
+  __nv_bfloat16* out;  // [m][N], or null: no norm
+};
+
 template <int EPI, bool ROWS16, int NT>
 __global__ void __launch_bounds__(NT * kWarps * 32)
 linear_rows_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w, void* Y,
-                   const float* residual, int M, int N, int K, int tiles, RopeCache rc, int* failure, int act) {
+                   const float* residual, int M, int N, int K, int tiles, RopeCache rc, int* failure, int act, TanhNormOut tn) {
   static_assert(EPI != 3 || NT == 2, "a rotation needs both halves of a head in the tile");
   constexpr int R = ROWS16 ? 16 : 8;
   constexpr int kItemBytes = kGroupBytes;  // what a warp fetches per (tile, chunk): its group's 8 rows
@@ -189,14 +197,17 @@ linear_rows_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
   int flip = 0;       // which half of the chunk sums this tile uses
   for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x, flip ^= 1) {
     // the residual of this thread's outputs is asked for now and used after the arithmetic
-    float res[kMine];
+    float res[kMine], nw[kMine], nb[kMine];
 #pragma unroll
     for (int e = 0; e < kMine; ++e) {
-      res[e] = 0.0f;
-      if (EPI == 2 && residual) {
+      res[e] = 0.0f, nw[e] = 0.0f, nb[e] = 0.0f;
+      if (EPI == 2) {
         const int o = tid + e * kThreads;
         const int r = o / (NT * 8), n = tile * (NT * 8) + o % (NT * 8);
-        if (o < kOutputs && r < M && n < N) res[e] = residual[static_cast<size_t>(r) * N + n];
+        if (o < kOutputs && r < M && n < N) {
+          if (residual) res[e] = residual[static_cast<size_t>(r) * N + n];
+          if (tn.out) nw[e] = tn.w[n], nb[e] = tn.b[n];
+        }
       }
     }
     float* sums = part + flip * num_chunks * kOutputs;
@@ -319,6 +330,7 @@ linear_rows_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
         if (EPI == 2) {
           if (residual) v = res[e] + v;
           static_cast<float*>(Y)[at] = v;
+          if (tn.out) tn.out[at] = __float2bfloat16_rn(bw::tanh_norm_one(v, tn.alpha[0], nw[e], nb[e]));
         } else {
           static_cast<__nv_bfloat16*>(Y)[at] = __float2bfloat16_rn(EPI == 0 ? bw::out_act(v, act) : v);
         }
@@ -403,7 +415,8 @@ bool rows_shape(int m, int n, int k, bool swiglu, RowsShape* s) {
 
 template <int EPI, bool ROWS16, int NT>
 int launch_rows(const __nv_bfloat16* x, const __nv_bfloat16* w, void* y, const float* residual, int m, int n, int k,
-                const RowsShape& s, cudaStream_t stream, const RopeCache& rc = RopeCache{}, int act = 0) {
+                const RowsShape& s, cudaStream_t stream, const RopeCache& rc = RopeCache{}, int act = 0,
+                const TanhNormOut& tn = TanhNormOut{}) {
   auto kernel = linear_rows_kernel<EPI, ROWS16, NT>;
   static bool configured = false;
   if (!configured) {
@@ -422,19 +435,19 @@ int launch_rows(const __nv_bfloat16* x, const __nv_bfloat16* w, void* y, const f
   int* word = bw::failure_word();
   if (!word) return -1;
   bw::launch_pdl(kernel, dim3(s.grid), dim3(NT * kWarps * 32), s.smem, stream, map_x, map_w, y, residual, m, n, k, s.tiles, rc,
-                 word, act);
+                 word, act, tn);
   return bw::launch_status();
 }
 
 template <int EPI>
 int launch_rows_epi(const __nv_bfloat16* x, const __nv_bfloat16* w, void* y, const float* residual, int m, int n, int k,
-                    const RowsShape& s, cudaStream_t stream, int act = 0) {
+                    const RowsShape& s, cudaStream_t stream, int act = 0, const TanhNormOut& tn = TanhNormOut{}) {
   if (s.nt == 2)
-    return s.rows16 ? launch_rows<EPI, true, 2>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act)
-                    : launch_rows<EPI, false, 2>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act);
+    return s.rows16 ? launch_rows<EPI, true, 2>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act, tn)
+                    : launch_rows<EPI, false, 2>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act, tn);
   if (EPI == 1) return -1;  // SwiGLU tiles always hold two groups
-  return s.rows16 ? launch_rows<EPI == 1 ? 0 : EPI, true, 1>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act)
-                  : launch_rows<EPI == 1 ? 0 : EPI, false, 1>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act);
+  return s.rows16 ? launch_rows<EPI == 1 ? 0 : EPI, true, 1>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act, tn)
+                  : launch_rows<EPI == 1 ? 0 : EPI, false, 1>(x, w, y, residual, m, n, k, s, stream, RopeCache{}, act, tn);
 }
 
 }  // namespace
@@ -471,6 +484,19 @@ BW_API int bw_bf16_linear_rows(const __nv_bfloat16* x, const __nv_bfloat16* w, v
   if (y_kind == 1) return launch_rows_epi<1>(x, w, y, nullptr, m, n, k, s, stream, act);
   if (y_kind == 2) return launch_rows_epi<2>(x, w, y, residual, m, n, k, s, stream);
   return launch_rows_epi<0>(x, w, y, nullptr, m, n, k, s, stream, act);
+}
+
+// y = (residual +) product in float32 and xn = tanh(alpha y) nw + nb in bfloat16, for shapes of this path.
+BW_API int bw_bf16_linear_rows_tanh(const __nv_bfloat16* x, const __nv_bfloat16* w, float* y, const float* residual, int m, int n,
+                                    int k, const float* alpha, const float* nw, const float* nb, __nv_bfloat16* xn,
+                                    cudaStream_t stream) {
+  if (m <= 0 || n <= 0) return 0;
+  RowsShape s;
+  if (!bw_bf16_linear_rows_usable(x, w, m, n, k, 0) || !rows_shape(m, n, k, false, &s)) {
+    bw::set_error("linear with a norm (few rows): shape [%d x %d] x [%d x %d] is not for this path", m, k, n, k);
+    return -1;
+  }
+  return launch_rows_epi<2>(x, w, y, residual, m, n, k, s, stream, 0, TanhNormOut{alpha, nw, nb, xn});
 }
 
 // Whether the fused q/k/v projection of a step can rotate and store its outputs itself

@@ -30,17 +30,29 @@ namespace {
 // ---------------------------------------------------------------------------------------
 // One warp per row. Shared memory per warp: scores s[E] (a taken expert's is set to -1), choice
 // scores c[E] (-inf for the experts of groups that do not stay), group scores [groups].
+constexpr int kTile = 64;  // list entries of a tile of the grouped product
 enum { kSigmoid = 0, kSoftmaxTop = 1, kSoftmax = 2 };
 
-__global__ void __launch_bounds__(128)
-route_kernel(const float* __restrict__ z, int z_stride, const float* __restrict__ correction, int n, int experts, int groups,
-             int keep, int top, float weight_scale, int scoring, int group_max, float sum_eps /* >= 0: weights over their sum */,
-             int* __restrict__ chosen, float* __restrict__ weights) {
-  bw::pdl_enter();
-  extern __shared__ float sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int r = blockIdx.x * (blockDim.x >> 5) + warp;
-  if (r >= n) return;
+struct RouteArgs {
+  const float* z;
+  int z_stride;
+  const float* correction;
+  int n, experts, groups, keep, top;
+  float weight_scale;
+  int scoring, group_max;
+  float sum_eps;  // >= 0: weights over their sum
+  int* chosen;
+  float* weights;
+};
+
+__device__ __forceinline__ void route_row(const RouteArgs& a, int r, int warp, int lane, float* sm) {
+  const float* __restrict__ z = a.z;
+  const float* __restrict__ correction = a.correction;
+  const int z_stride = a.z_stride, experts = a.experts, groups = a.groups, keep = a.keep, top = a.top;
+  const int scoring = a.scoring, group_max = a.group_max;
+  const float weight_scale = a.weight_scale, sum_eps = a.sum_eps;
+  int* __restrict__ chosen = a.chosen;
+  float* __restrict__ weights = a.weights;
   float* s = sm + static_cast<size_t>(warp) * (2 * experts + groups);
   float* c = s + experts;
   float* gs = c + experts;
@@ -140,6 +152,64 @@ route_kernel(const float* __restrict__ z, int z_stride, const float* __restrict_
   }
 }
 
+__global__ void __launch_bounds__(128) route_kernel(const RouteArgs a) {
+  bw::pdl_enter();
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5;
+  const int r = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (r < a.n) route_row(a, r, warp, threadIdx.x & 31, sm);
+}
+
+// Steps of few rows: one block routes a row per warp and lists the pairs as group_rows does (the same lists). Shared memory:
+// the rows' scores as for route_kernel, then int [experts + 1].
+constexpr int kRouteRows = 16;
+
+__global__ void __launch_bounds__(kRouteRows * 32)
+route_group_kernel(const RouteArgs a, int tile_rows, int* __restrict__ group_off, int* __restrict__ tile_prefix,
+                   int* __restrict__ order, int* __restrict__ place) {
+  bw::pdl_enter();
+  extern __shared__ float sm[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, experts = a.experts;
+  int* off = reinterpret_cast<int*>(sm + static_cast<size_t>(blockDim.x >> 5) * (2 * experts + a.groups));
+  for (int e = tid; e <= experts; e += blockDim.x) off[e] = 0;
+  if (warp < a.n) route_row(a, warp, warp, lane, sm);
+  __syncthreads();
+  const int pairs = a.n * a.top;
+  int* chosen = reinterpret_cast<int*>(sm);  // the scores are done with: the choices take their place
+  for (int p = tid; p < pairs; p += blockDim.x) {
+    const int e = __ldcg(a.chosen + p);  // (this block's own writes, behind the barrier)
+    chosen[p] = e;
+    atomicAdd(&off[e], 1);
+  }
+  __syncthreads();
+  if (warp == 0) {
+    int rows = 0, tiles = 0, big = 0;  // of the experts before this group of 32
+    for (int e0 = 0; e0 < experts; e0 += 32) {
+      const int e = e0 + lane;
+      const int c = e < experts ? off[e] : 0;
+      int sr = c, st = (c + tile_rows - 1) / tile_rows, sb = (c + 2 * tile_rows - 1) / (2 * tile_rows);
+      const int own_t = st, own_b = sb;
+      for (int d = 1; d < 32; d <<= 1) {
+        const int vr = __shfl_up_sync(0xffffffffu, sr, d), vt = __shfl_up_sync(0xffffffffu, st, d), vb = __shfl_up_sync(0xffffffffu, sb, d);
+        if (lane >= d) sr += vr, st += vt, sb += vb;
+      }
+      if (e < experts) {
+        off[e] = rows + sr - c;
+        group_off[e] = rows + sr - c, tile_prefix[e] = tiles + st - own_t, tile_prefix[experts + 1 + e] = big + sb - own_b;
+      }
+      rows += __shfl_sync(0xffffffffu, sr, 31), tiles += __shfl_sync(0xffffffffu, st, 31), big += __shfl_sync(0xffffffffu, sb, 31);
+    }
+    if (lane == 0) group_off[experts] = rows, tile_prefix[experts] = tiles, tile_prefix[2 * experts + 1] = big;
+  }
+  __syncthreads();
+  for (int p = tid; p < pairs; p += blockDim.x) {
+    const int e = chosen[p];
+    int i = off[e];
+    for (int q = 0; q < p; ++q) i += chosen[q] == e;
+    order[i] = p, place[p] = i;
+  }
+}
+
 // ---------------------------------------------------------------------------------------
 // pairs = n * top entries of `chosen`. Every block counts the experts' pairs for itself (shared-memory
 // atomics; the counts do not depend on their order); the placing is shared between the blocks. Outputs: group_off[E + 1] (where each
@@ -197,7 +267,7 @@ group_rows_kernel(const int* __restrict__ chosen, int pairs, int experts, int ti
 // ---------------------------------------------------------------------------------------
 // The grouped product: tiles of 64 list entries x 64 outputs, k in steps of 16, 256 threads with
 // 4 x 4 outputs each.
-constexpr int kTile = 64, kStep = 16;
+constexpr int kStep = 16;
 
 template <typename OutT>
 __global__ void __launch_bounds__(256)
@@ -509,7 +579,8 @@ __global__ void glu_clamped_kernel(const act_t* __restrict__ gate_up, act_t* __r
 template <bool VEC>
 __global__ void combine_kernel(float* x, const float* __restrict__ d, const float* __restrict__ y,
                                const int* __restrict__ place, const float* __restrict__ weights, int top, int width,
-                               const float* __restrict__ scale, const float* __restrict__ d_gate, int gate_stride) {
+                               const float* __restrict__ scale, const float* __restrict__ d_gate, int gate_stride,
+                               const float* __restrict__ alpha, const float* __restrict__ nw, const float* __restrict__ nb, act_t* xn) {
   bw::pdl_enter();
   constexpr int per = VEC ? 4 : 1;
   const int r = blockIdx.x;
@@ -534,7 +605,9 @@ __global__ void combine_kernel(float* x, const float* __restrict__ d, const floa
   for (int e = 0; e < per; ++e) {
     float v = s[e];
     if (d) v = d_gate ? __fmaf_rn(gate, d[o + e], v) : __fadd_rn(d[o + e], v);
-    x[o + e] = scale ? __fmaf_rn(scale[c + e], v, x[o + e]) : __fadd_rn(x[o + e], v);
+    v = scale ? __fmaf_rn(scale[c + e], v, x[o + e]) : __fadd_rn(x[o + e], v);
+    x[o + e] = v;
+    if (xn) xn[o + e] = bw::from_f<act_t>(bw::tanh_norm_one(v, alpha[0], nw[c + e], nb[c + e]));
   }
 }
 
@@ -557,8 +630,29 @@ BW_API int BW_FN(route)(const float* z, int z_stride, const float* correction, i
     bw::set_error("route: %d experts are beyond the kernel", experts);
     return -1;
   }
-  bw::launch_pdl(route_kernel, dim3((n + warps - 1) / warps), dim3(warps * 32), smem, stream, z, z_stride, correction, n, experts,
-                 groups, keep, top, weight_scale, scoring, group_max, sum_eps, chosen, weights);
+  const RouteArgs a{z, z_stride, correction, n, experts, groups, keep, top, weight_scale, scoring, group_max, sum_eps, chosen, weights};
+  bw::launch_pdl(route_kernel, dim3((n + warps - 1) / warps), dim3(warps * 32), smem, stream, a);
+  return bw::launch_status();
+}
+
+// Whether a step of n rows takes route and group_rows in one kernel (route_group).
+BW_API int BW_FN(route_group_usable)(int n, int experts, int groups) {
+  return n > 0 && n <= kRouteRows && static_cast<size_t>(n) * (2 * experts + groups) * 4 + (experts + 1) * 4 <= 48 * 1024;
+}
+
+// route, then group_rows of what it chose, in one kernel (the same choices, weights and lists).
+BW_API int BW_FN(route_group)(const float* z, int z_stride, const float* correction, int n, int experts, int groups, int keep,
+                              int top, float weight_scale, int scoring, int group_max, float sum_eps, int* chosen, float* weights,
+                              int* group_off, int* tile_prefix, int* order, int* place, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (experts <= 0 || groups <= 0 || experts % groups || keep <= 0 || keep > groups || top <= 0 ||
+      top > keep * (experts / groups) || !BW_FN(route_group_usable)(n, experts, groups)) {
+    bw::set_error("route_group: %d rows, %d experts in %d groups of which %d stay, %d choices", n, experts, groups, keep, top);
+    return -1;
+  }
+  const RouteArgs a{z, z_stride, correction, n, experts, groups, keep, top, weight_scale, scoring, group_max, sum_eps, chosen, weights};
+  const size_t smem = static_cast<size_t>(n) * (2 * experts + groups) * sizeof(float) + (experts + 1) * sizeof(int);
+  bw::launch_pdl(route_group_kernel, dim3(1), dim3(n * 32), smem, stream, a, kTile, group_off, tile_prefix, order, place);
   return bw::launch_status();
 }
 
@@ -633,10 +727,10 @@ BW_API int BW_FN(grouped_linear)(const act_t* x, int x_stride, int x_group_cols,
                                                           prefix, rows, groups, n, k, act);
     }
     if (out_is_f32)
-      return launch_grouped_mma<float, 64, 64, 2, 2, 3>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
+      return launch_grouped_mma<float, 64, 64, 2, 2, 6>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                         static_cast<float*>(out), o_stride, o_group_cols, group_off,
                                                         tile_prefix, rows, groups, n, k, act);
-    return launch_grouped_mma<act_t, 64, 64, 2, 2, 3>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
+    return launch_grouped_mma<act_t, 64, 64, 2, 2, 6>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                       static_cast<act_t*>(out), o_stride, o_group_cols, group_off,
                                                       tile_prefix, rows, groups, n, k, act);
   }
@@ -673,14 +767,16 @@ BW_API int BW_FN(glu_clamped)(const act_t* gate_up, act_t* out, int n, int inter
 }
 
 BW_API int BW_FN(combine)(float* x, const float* d, const float* y, const int* place, const float* weights, int n,
-                          int top, int width, const float* scale, const float* d_gate, int gate_stride, cudaStream_t stream) {
+                          int top, int width, const float* scale, const float* d_gate, int gate_stride, const float* alpha,
+                          const float* nw, const float* nb, void* xn, cudaStream_t stream) {
+  // xn: the norm without statistics, tanh(alpha x) nw + nb, of the summed rows as well (null: none)
   // d_gate: d is multiplied by the sigmoid of d_gate[r * gate_stride] first (null: as it is)
   if (n <= 0 || width <= 0) return 0;
   if (width % 4 == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0)
     bw::launch_pdl(combine_kernel<true>, dim3(n, (width / 4 + 127) / 128), dim3(128), 0, stream, x, d, y, place, weights, top,
-                   width, scale, d_gate, gate_stride);
+                   width, scale, d_gate, gate_stride, alpha, nw, nb, static_cast<act_t*>(xn));
   else
     bw::launch_pdl(combine_kernel<false>, dim3(n, (width + 255) / 256), dim3(256), 0, stream, x, d, y, place, weights, top,
-                   width, scale, d_gate, gate_stride);
+                   width, scale, d_gate, gate_stride, alpha, nw, nb, static_cast<act_t*>(xn));
   return bw::launch_status();
 }

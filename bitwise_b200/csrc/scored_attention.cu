@@ -581,8 +581,8 @@ int launch_scored(dim3 grid, size_t smem, cudaStream_t stream, const act_t* q, i
 
 // ---------------------------------------------------------------------------------------
 // Two maps of a result head joined: the spans' records of query heads 2h and 2h + 1 merged in ascending order of the spans, as
-// scored_attention_merge does, then o = a1 - lambda a2, o <- o / sqrt(mean(o^2) + eps) * keep, and the output gate. A warp per
-// row and result head.
+// scored_attention_merge does, then o = a1 - lambda a2, o <- o / sqrt(mean(o^2) + eps) * keep, and the output gate. Two
+// warps per row and result head, one for each map.
 struct DifferenceArgs {
   const float* partial;  // [n, 2 * heads, spans, vdim + 2]
   int spans, queries /* n * heads */, heads, vdim;
@@ -593,41 +593,73 @@ struct DifferenceArgs {
   act_t* out;            // [n, heads * vdim]
 };
 
-__device__ __forceinline__ void merge_spans(const float* __restrict__ rec, int spans, int vdim, int lane, float (&acc)[8]) {
-  float m = -INFINITY;
-  for (int s = 0; s < spans; ++s) m = fmaxf(m, rec[static_cast<size_t>(s) * (vdim + 2)]);
-  float l = 0.0f;
+// The records of one query joined in ascending order of the spans by a warp: m and l of the sum, and the weighted values, lane l's
+// entries l, l + 32, ... of them. A lane looks at one span's maximum and sum, and the values of four spans are asked for together;
+// spans in which the query saw no key hold nothing but their -infinity.
+__device__ __forceinline__ void merge_spans(const float* __restrict__ rec, int spans, int vdim, int lane, float& m, float& l, float (&acc)[8]) {
+  const int stride = vdim + 2;
+  m = -INFINITY;
+  for (int s0 = 0; s0 < spans; s0 += 32)
+    if (s0 + lane < spans) m = fmaxf(m, rec[static_cast<size_t>(s0 + lane) * stride]);
+  m = bw::warp_max(m);
+  l = 0.0f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) acc[i] = 0.0f;
-  for (int s = 0; s < spans; ++s) {
-    const float* r = rec + static_cast<size_t>(s) * (vdim + 2);
-    if (r[0] == -INFINITY) continue;  // a span in which the query saw no key
-    const float f = expf(__fsub_rn(r[0], m));
-    l = __fmaf_rn(r[1], f, l);
+  for (int s0 = 0; s0 < spans; s0 += 32) {
+    const float* r = rec + static_cast<size_t>(s0) * stride;
+    const bool have = s0 + lane < spans;
+    const float ms = have ? r[static_cast<size_t>(lane) * stride] : -INFINITY;
+    const float ls = have ? r[static_cast<size_t>(lane) * stride + 1] : 0.0f;
+    const float fs = ms == -INFINITY ? 0.0f : expf(__fsub_rn(ms, m));
+    unsigned live = __ballot_sync(0xffffffffu, ms != -INFINITY);
+    while (live) {
+      constexpr int kBatch = 4;
+      float v[kBatch][8], f[kBatch], lp[kBatch];
+      bool take[kBatch];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int d = i * 32 + lane;
-      if (d < vdim) acc[i] = __fmaf_rn(r[2 + d], f, acc[i]);
+      for (int b = 0; b < kBatch; ++b) {
+        take[b] = live != 0;
+        const int at = take[b] ? __ffs(live) - 1 : 0;
+        live &= live - 1;
+        f[b] = __shfl_sync(0xffffffffu, fs, at), lp[b] = __shfl_sync(0xffffffffu, ls, at);
+        const float* src = r + static_cast<size_t>(at) * stride + 2 + lane;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[b][i] = take[b] && i * 32 + lane < vdim ? src[i * 32] : 0.0f;
+      }
+#pragma unroll
+      for (int b = 0; b < kBatch; ++b) {
+        if (!take[b]) break;
+        l = __fmaf_rn(lp[b], f[b], l);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) acc[i] = __fmaf_rn(v[b][i], f[b], acc[i]);
+      }
     }
   }
-  const float inv = __fdiv_rn(1.0f, l);
-#pragma unroll
-  for (int i = 0; i < 8; ++i) acc[i] = __fmul_rn(acc[i], inv);
 }
 
 __global__ void __launch_bounds__(128) scored_difference_kernel(const DifferenceArgs a) {
   bw::pdl_enter();
-  const int qi = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (qi >= a.queries) return;
-  const size_t each = static_cast<size_t>(a.spans) * (a.vdim + 2);
-  float o[8], o2[8];
-  merge_spans(a.partial + 2 * static_cast<size_t>(qi) * each, a.spans, a.vdim, lane, o);
-  merge_spans(a.partial + (2 * static_cast<size_t>(qi) + 1) * each, a.spans, a.vdim, lane, o2);
+  __shared__ float second[2][256];  // the second map's outputs of the block's two result heads
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, map = warp & 1;
+  const int qi = blockIdx.x * 2 + (warp >> 1);
+  const bool have = qi < a.queries;
+  float o[8], m, l;
+  if (have) {
+    merge_spans(a.partial + (2 * static_cast<size_t>(qi) + map) * a.spans * (a.vdim + 2), a.spans, a.vdim, lane, m, l, o);
+    const float inv = __fdiv_rn(1.0f, l);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      o[i] = __fmul_rn(o[i], inv);
+      if (map) second[warp >> 1][i * 32 + lane] = o[i];
+    }
+  }
+  __syncthreads();
+  if (!have || map) return;
   const float lam = a.lambda[0];
   float ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) {  // (entries beyond the head are zero)
-    o[i] = __fmaf_rn(-lam, o2[i], o[i]);
+    o[i] = __fmaf_rn(-lam, second[warp >> 1][i * 32 + lane], o[i]);
     ss = __fmaf_rn(o[i], o[i], ss);
   }
   const float f = __fmul_rn(bw::rms_scale(bw::warp_sum(ss), a.vdim, a.eps), a.keep);
@@ -643,7 +675,6 @@ __global__ void __launch_bounds__(128) scored_difference_kernel(const Difference
     dst[d] = bw::from_f<act_t>(v);
   }
 }
-
 
 #if BW_ACT_BF16
 // ---------------------------------------------------------------------------------------
@@ -686,18 +717,22 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   const int p0 = seq_pos0[seq] + (row0 - seq_row0[seq]);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dparts = dim >> 3, vparts = vdim >> 3;
+  // A block of at most 16 queries (a decode step's) gives them to all its warps: each forms all scores and weights, and every
+  // fourth part of 16 value columns is its own. Else a warp has 16 queries of the block. The sums are the same either way.
+  const bool narrow = nq <= 16;
+  const int wr = narrow ? 0 : warp * 16;
   // this thread's two queries: stacked rows sa_ and sb_ of the block
-  const int sr_a = warp * 16 + (lane >> 2), sr_b = sr_a + 8;
+  const int sr_a = wr + (lane >> 2), sr_b = sr_a + 8;
   const bool ok_a = sr_a < nq, ok_b = sr_b < nq;
   const int pq_a = p0 + (ok_a ? sr_a / nh : 0), pq_b = p0 + (ok_b ? sr_b / nh : 0);
   const int lo_a = first_seen(sa, pq_a), lo_b = first_seen(sa, pq_b);
   const HeadBias slope_a = head_bias(sa, h0 + sr_a % nh * hstep, ok_a), slope_b = head_bias(sa, h0 + sr_b % nh * hstep, ok_b);
   const int keep = sa.window > 0 ? sa.keep_first : 0;
   // the positions that this warp's queries span: tiles outside are skipped by the whole warp
-  const int w_first = min(warp * 16, max(nq - 1, 0)) / nh, w_last = min(warp * 16 + 15, max(nq - 1, 0)) / nh;
+  const int w_first = min(wr, max(nq - 1, 0)) / nh, w_last = min(wr + 15, max(nq - 1, 0)) / nh;
   const int w_lo = first_seen(sa, p0 + w_first), w_hi = p0 + w_last;
-  const bool warp_has_rows = warp * 16 < nq;
-  const bool warp_full = warp * 16 + 15 < nq;  // all 16 stacked rows of the warp are queries
+  const bool warp_has_rows = wr < nq;
+  const bool warp_full = wr + 15 < nq;  // all 16 stacked rows of the warp are queries
   const int w_seen_to = p0 + w_first;           // keys up to here are seen by every query of the warp ...
   const int w_seen_from = first_seen(sa, p0 + w_last);  // ... from here on
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
@@ -790,7 +825,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     for (int j = 0; j < 4; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.0f;
     for (int kk = 0; kk < dim; kk += 16) {
       uint32_t a[4], b[4];
-      bw::ldsm4(a, bw::smem_addr(qs + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kst + kk + (lane >> 4) * 8));
+      bw::ldsm4(a, bw::smem_addr(qs + (wr + (lane & 7) + ((lane >> 3) & 1) * 8) * kst + kk + (lane >> 4) * 8));
 #pragma unroll
       for (int jp = 0; jp < 2; ++jp) {  // 16 keys at a time
         bw::ldsm4(b, bw::smem_addr(ks + (jp * 16 + (lane >> 4) * 8 + (lane & 7)) * kst + kk + ((lane >> 3) & 1) * 8));
@@ -867,6 +902,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
       }
 #pragma unroll
       for (int jp = 0; jp < VD16; ++jp) {  // 16 value columns at a time
+        if (narrow && (jp & 3) != warp) continue;
         uint32_t b[4];
         bw::ldsm4_trans(b, bw::smem_addr(vs + (kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * vst + jp * 16 + (lane >> 4) * 8));
         bw::mma16816(acc[2 * jp], hi, b[0], b[1]);
@@ -886,15 +922,17 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     const int colp = 2 * (lane & 3);
     if (ok_a) {
       float* rec = partial + ((static_cast<size_t>(row0 + sr_a / nh) * heads + h0 + sr_a % nh * hstep) * spans + span) * (vdim + 2);
-      if ((lane & 3) == 0) rec[0] = m_a, rec[1] = l_a;
+      if ((lane & 3) == 0 && (warp == 0 || !narrow)) rec[0] = m_a, rec[1] = l_a;
 #pragma unroll
-      for (int j = 0; j < VT; ++j) rec[2 + j * 8 + colp] = acc[j][0], rec[2 + j * 8 + colp + 1] = acc[j][1];
+      for (int j = 0; j < VT; ++j)
+        if (!narrow || ((j >> 1) & 3) == warp) rec[2 + j * 8 + colp] = acc[j][0], rec[2 + j * 8 + colp + 1] = acc[j][1];
     }
     if (ok_b) {
       float* rec = partial + ((static_cast<size_t>(row0 + sr_b / nh) * heads + h0 + sr_b % nh * hstep) * spans + span) * (vdim + 2);
-      if ((lane & 3) == 0) rec[0] = m_b, rec[1] = l_b;
+      if ((lane & 3) == 0 && (warp == 0 || !narrow)) rec[0] = m_b, rec[1] = l_b;
 #pragma unroll
-      for (int j = 0; j < VT; ++j) rec[2 + j * 8 + colp] = acc[j][2], rec[2 + j * 8 + colp + 1] = acc[j][3];
+      for (int j = 0; j < VT; ++j)
+        if (!narrow || ((j >> 1) & 3) == warp) rec[2 + j * 8 + colp] = acc[j][2], rec[2 + j * 8 + colp + 1] = acc[j][3];
     }
     return;
   }
@@ -908,13 +946,15 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_a / nh) * o_stride + (h0 + sr_a % nh * hstep) * vdim + col;
 #pragma unroll
     for (int j = 0; j < VT; ++j)
-      *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][0], inv_a), __fmul_rn(acc[j][1], inv_a));
+      if (!narrow || ((j >> 1) & 3) == warp)
+        *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][0], inv_a), __fmul_rn(acc[j][1], inv_a));
   }
   if (ok_b) {
     __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_b / nh) * o_stride + (h0 + sr_b % nh * hstep) * vdim + col;
 #pragma unroll
     for (int j = 0; j < VT; ++j)
-      *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][2], inv_b), __fmul_rn(acc[j][3], inv_b));
+      if (!narrow || ((j >> 1) & 3) == warp)
+        *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][2], inv_b), __fmul_rn(acc[j][3], inv_b));
   }
 }
 
@@ -925,24 +965,8 @@ scored_attention_merge_kernel(const float* __restrict__ partial, __nv_bfloat16* 
   bw::pdl_enter();
   const int qi = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (qi >= queries) return;
-  const float* rec = partial + static_cast<size_t>(qi) * spans * (vdim + 2);
-  float m = -INFINITY;
-  for (int s = 0; s < spans; ++s) m = fmaxf(m, rec[static_cast<size_t>(s) * (vdim + 2)]);
-  float l = 0.0f;
-  float acc[8];
-#pragma unroll
-  for (int i = 0; i < 8; ++i) acc[i] = 0.0f;
-  for (int s = 0; s < spans; ++s) {
-    const float* r = rec + static_cast<size_t>(s) * (vdim + 2);
-    if (r[0] == -INFINITY) continue;  // a span in which the query saw no key
-    const float f = expf(__fsub_rn(r[0], m));
-    l = __fmaf_rn(r[1], f, l);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int d = i * 32 + lane;
-      if (d < vdim) acc[i] = __fmaf_rn(r[2 + d], f, acc[i]);
-    }
-  }
+  float m, l, acc[8];
+  merge_spans(partial + static_cast<size_t>(qi) * spans * (vdim + 2), spans, vdim, lane, m, l, acc);
   if (sink) l = __fadd_rn(l, expf(__fsub_rn(sinks ? sinks[qi % heads] : 0.0f, m)));
   const float inv = __fdiv_rn(1.0f, l);
   __nv_bfloat16* dst = out + static_cast<size_t>(qi / heads) * o_stride + (qi % heads) * vdim;
@@ -1187,6 +1211,6 @@ BW_API int BW_FN(scored_difference)(const float* partial, int spans, const float
   a.partial = partial, a.spans = spans, a.queries = n * heads, a.heads = heads, a.vdim = vdim, a.lambda = lambda;
   a.keep = keep, a.eps = eps, a.gate = gate, a.gate_stride = gate_stride, a.gate_group = gate_group;
   a.out = static_cast<act_t*>(out);
-  bw::launch_pdl(scored_difference_kernel, dim3((a.queries + 3) / 4), dim3(128), 0, stream, a);
+  bw::launch_pdl(scored_difference_kernel, dim3((a.queries + 1) / 2), dim3(128), 0, stream, a);
   return bw::launch_status();
 }

@@ -186,11 +186,22 @@ class KernelOps:
                    _c_float(eps), self._stream())
 
     def linear(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
-               residual: Optional[torch.Tensor] = None, legacy: bool = False, activation: Optional[str] = None) -> None:
+               residual: Optional[torch.Tensor] = None, legacy: bool = False, activation: Optional[str] = None,
+               then: Optional[tuple] = None) -> None:
         """out = x @ w.T (+ residual).  x [M,K] and w [N,K] in act_dtype; out act_dtype or
         float32; with a float32 residual the sum is formed in 32-bit (out float32, may alias).
         ``activation`` (of OUT_ACTIVATIONS; out act_dtype, no residual): out = act(x @ w.T), applied to the
-        32-bit sums in the product's epilogue on the serving precision."""
+        32-bit sums in the product's epilogue on the serving precision.  ``then`` = (alpha, weight, bias, rows): the norm
+        without statistics of the finished float32 rows into ``rows`` (act_dtype), as ``tanh_norm`` gives it; in the
+        product's own kernel for steps of few rows on the serving precision."""
+        if then is not None:
+            _need(out, torch.float32, "linear out", 2)
+            if self._linear_then(x, w, out, residual, then):
+                return
+            self.linear(x, w, out, residual, legacy, activation)
+            alpha, weight, bias, rows = then
+            self.tanh_norm(out, alpha, weight, bias, rows)
+            return
         act = 0
         if activation is not None:
             if activation not in self.OUT_ACTIVATIONS or residual is not None or out.dtype != self.act_dtype:
@@ -224,6 +235,27 @@ class KernelOps:
                        _p(residual), _c_int(m), _c_int(n), _c_int(k), _p(partials), _p(counters),
                        _c_int(int(legacy)), self._stream(),
                        launches=1 if legacy else self._linear_kernels(m, n, k, False, partials is not None))
+
+    def _linear_then(self, x, w, out, residual, then) -> bool:
+        """``linear`` with the norm that follows in one kernel; False where the shape takes another path."""
+        (m, k), n = x.shape, w.shape[0]
+        if self.kind != "bf16" or m > 16 or not self.lib.bw_bf16_linear_rows_usable(_p(x), _p(w), _c_int(m), _c_int(n), _c_int(k), _c_int(0)):
+            return False
+        alpha, weight, bias, rows = then
+        _need(x, self.act_dtype, "linear x", 2)
+        _need(w, self.act_dtype, "linear w", 2)
+        _need(rows, self.act_dtype, "linear norm rows", 2)
+        for t_, count in ((alpha, 1), (weight, n), (bias, n)):
+            _need(t_, torch.float32, "linear norm")
+            if t_.numel() != count:
+                raise KernelError("linear: the norm's numbers do not fit the product's columns")
+        if residual is not None:
+            _need(residual, torch.float32, "linear residual", 2)
+        if w.shape[1] != k or tuple(out.shape) != (m, n) or rows.shape != out.shape or (residual is not None and residual.shape != out.shape):
+            raise KernelError(f"linear: shapes x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)} norm{tuple(rows.shape)}")
+        self._call("bw_bf16_linear_rows_tanh", _p(x), _p(w), _p(out), _p(residual), _c_int(m), _c_int(n), _c_int(k), _p(alpha), _p(weight),
+                   _p(bias), _p(rows), self._stream())
+        return True
 
     def fuses_swiglu(self, width: int, intermediate: int, activation: str = "silu") -> bool:
         """Whether ``linear_swiglu`` can take a feed-forward of these sizes and this activation (then its
@@ -868,7 +900,7 @@ class KernelOps:
 
     def route(self, logits: torch.Tensor, correction: Optional[torch.Tensor], groups: int, keep: int, top: int,
               weight_scale: float, chosen: torch.Tensor, weights: torch.Tensor, softmax_top: bool = False,
-              scoring: Optional[str] = None, group_max: bool = False, sum_eps: Optional[float] = None) -> None:
+              scoring: Optional[str] = None, group_max: bool = False, sum_eps: Optional[float] = None, lists=None) -> None:
         """Per row of ``logits`` (float32 [n, experts]): scores sigmoid(z); the ``top`` experts with
         the largest score + correction among the experts of the ``keep`` best of ``groups`` equal
         groups of neighbours (a group counts as the sum of its two largest corrected scores);
@@ -877,7 +909,8 @@ class KernelOps:
         logits only, times weight_scale.  ``scoring`` names the kind instead (of ROUTE_SCORES); "softmax": the scores
         are the softmax over all experts.  ``group_max``: a group counts as its largest choice score alone.
         ``sum_eps``: the weights are the chosen scores divided by (their sum + sum_eps), times weight_scale.  The
-        rows of ``logits`` may be columns of wider rows."""
+        rows of ``logits`` may be columns of wider rows.  ``lists`` = (group_off, tile_prefix, order, place): what
+        ``group_rows`` makes of the choices, in the same kernel for steps of few rows."""
         n, experts = logits.shape
         scoring = scoring or ("softmax_top" if softmax_top else "sigmoid")
         if scoring not in self.ROUTE_SCORES or (sum_eps is not None and (scoring == "softmax_top" or sum_eps < 0)):
@@ -889,10 +922,26 @@ class KernelOps:
             _need(correction, torch.float32, "route correction", 1)
         if tuple(chosen.shape) != (n, top) or tuple(weights.shape) != (n, top):
             raise KernelError("route: outputs are not [rows, top]")
-        self._pcall("route", _p(logits), _c_int(logits.stride(0)), _p(correction), _c_int(n), _c_int(experts), _c_int(groups),
-                    _c_int(keep), _c_int(top), _c_float(weight_scale), _c_int(self.ROUTE_SCORES.index(scoring)),
-                    _c_int(int(bool(group_max))), _c_float(-1.0 if sum_eps is None else sum_eps), _p(chosen), _p(weights),
-                    self._stream())
+        args = (_p(logits), _c_int(logits.stride(0)), _p(correction), _c_int(n), _c_int(experts), _c_int(groups), _c_int(keep), _c_int(top),
+                _c_float(weight_scale), _c_int(self.ROUTE_SCORES.index(scoring)), _c_int(int(bool(group_max))),
+                _c_float(-1.0 if sum_eps is None else sum_eps), _p(chosen), _p(weights))
+        if lists is None:
+            self._pcall("route", *args, self._stream())
+            return
+        if not getattr(self._parts_lib(), f"bw_{self.kind}_route_group_usable")(_c_int(n), _c_int(experts), _c_int(groups)):
+            self._pcall("route", *args, self._stream())
+            self.group_rows(chosen, experts, *lists)
+            return
+        self._check_lists(chosen.numel(), experts, *lists)
+        self._pcall("route_group", *args, *(_p(t_) for t_ in lists), self._stream())
+
+    @staticmethod
+    def _check_lists(pairs: int, experts: int, group_off, tile_prefix, order, place) -> None:
+        for t_, what in ((group_off, "group_off"), (tile_prefix, "tile_prefix"), (order, "order"), (place, "place")):
+            _need(t_, torch.int32, "group_rows " + what)
+        if group_off.numel() < experts + 1 or tile_prefix.numel() < 2 * (experts + 1) or order.numel() < pairs or \
+                place.numel() < pairs:
+            raise KernelError("group_rows: an output is too small")
 
     def group_rows(self, chosen: torch.Tensor, experts: int, group_off: torch.Tensor, tile_prefix: torch.Tensor,
                    order: torch.Tensor, place: torch.Tensor) -> None:
@@ -901,12 +950,8 @@ class KernelOps:
         two tile heights), order [pairs]
         (pair index = row * top + choice), place [pairs] (where a pair stands in ``order``)."""
         pairs = chosen.numel()
-        for t_, what in ((chosen, "chosen"), (group_off, "group_off"), (tile_prefix, "tile_prefix"), (order, "order"),
-                         (place, "place")):
-            _need(t_, torch.int32, "group_rows " + what)
-        if group_off.numel() < experts + 1 or tile_prefix.numel() < 2 * (experts + 1) or order.numel() < pairs or \
-                place.numel() < pairs:
-            raise KernelError("group_rows: an output is too small")
+        _need(chosen, torch.int32, "group_rows chosen")
+        self._check_lists(pairs, experts, group_off, tile_prefix, order, place)
         self._pcall("group_rows", _p(chosen), _c_int(pairs), _c_int(experts), _p(group_off), _p(tile_prefix), _p(order),
                     _p(place), self._stream())
 
@@ -986,10 +1031,11 @@ class KernelOps:
 
     def combine(self, x: torch.Tensor, d: Optional[torch.Tensor], y: torch.Tensor, place: torch.Tensor,
                 weights: torch.Tensor, top: int, scale: Optional[torch.Tensor] = None,
-                d_gate: Optional[torch.Tensor] = None) -> None:
+                d_gate: Optional[torch.Tensor] = None, then: Optional[tuple] = None) -> None:
         """x[r] += d[r] + sum_j weights[r, j] * y[place[r * top + j]] (float32; d may be None); with ``scale``
         [width] what is added is multiplied by it column by column first.  ``d_gate`` (float32 [n, 1], may be a
-        column of wider rows): d[r] is multiplied by sigmoid(d_gate[r]) first."""
+        column of wider rows): d[r] is multiplied by sigmoid(d_gate[r]) first.  ``then`` as for ``linear``: the norm
+        without statistics of the summed rows, in the same kernel."""
         n, width = x.shape
         _need(x, torch.float32, "combine x", 2)
         _need(y, torch.float32, "combine y", 2)
@@ -1003,12 +1049,21 @@ class KernelOps:
             _need(scale, torch.float32, "combine scale", 1)
             if scale.shape[0] != width:
                 raise KernelError("combine: one factor per column is needed")
+        norm = then or (None, None, None, None)
+        if then is not None:
+            for t_, count in zip(norm, (1, width, width)):
+                _need(t_, torch.float32, "combine norm")
+                if t_.numel() != count:
+                    raise KernelError("combine: the norm's numbers do not fit the columns")
+            _need(norm[3], self.act_dtype, "combine norm rows", 2)
+            if norm[3].shape != x.shape:
+                raise KernelError("combine: the norm's rows are not the stream's")
         if d_gate is not None:
             _need_rows(d_gate, torch.float32, "combine d_gate")
             if d is None or tuple(d_gate.shape) != (n, 1):
                 raise KernelError("combine: one gate number per row of d is needed")
         self._pcall("combine", _p(x), _p(d), _p(y), _p(place), _p(weights), _c_int(n), _c_int(top), _c_int(width),
-                    _p(scale), _p(d_gate), _c_int(d_gate.stride(0) if d_gate is not None else 0), self._stream())
+                    _p(scale), _p(d_gate), _c_int(d_gate.stride(0) if d_gate is not None else 0), *(_p(t_) for t_ in norm), self._stream())
 
     # -- element-wise steps of gated designs (their library is loaded at first use) ---------------------
     def _gated_lib(self):

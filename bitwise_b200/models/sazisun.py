@@ -20,7 +20,7 @@ from __future__ import annotations
 
 from ..config.registry import register_architecture
 from ..config.sazisun import SazisunConfig
-from ..parts.block import PreNormBlock
+from ..parts.block import PreNormBlock, chain_norms
 from ..parts.embedding import OutputHead, TokenEmbedding
 from ..parts.mlp import DenseFFN, SwiGLU
 from ..parts.norm import TanhNorm
@@ -77,6 +77,7 @@ def build_sazisun(config: SazisunConfig) -> DecoderModel:
             state = entries
             entries += 1
         schedule.append(LayerRun(i, entry_of[i if shared is None else shared], shared is None, state))
+    chain_norms(blocks)
     embedding = TokenEmbedding(c.vocab, c.width, tensor="embed")
     head = OutputHead(c.vocab, c.width, TanhNorm(c.width), tied_to=embedding, norm_name="final.norm")
     return DecoderModel(c, embedding, blocks, head, schedule=schedule, position_encodings=list(rotaries.values()),

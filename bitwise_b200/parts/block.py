@@ -17,7 +17,14 @@ from .base import FeedForward, Mixer, Norm, Part, SlotStateNeed, StepContext
 
 
 class PreNormBlock(Part):
-    """``feed_forward`` None: the layer is its mixer alone (and has no second norm)."""
+    """``feed_forward`` None: the layer is its mixer alone (and has no second norm).
+
+    A norm that works entry by entry (one that has ``after``) is formed by the kernel that finishes the rows it reads: the
+    second norm by the mixer's last one, and ``next_norm``, the norm that the block after this one begins with, by this
+    block's last one.  ``opened``: the block before has formed the first norm.  Both are set where the model is assembled; the
+    mixer and the feed-forward then take ``then``."""
+    next_norm: Optional[Norm] = None
+    opened = False
     graph_safe = True  # kernels only: a step through this part can be captured
 
     def __init__(self, width: int, mixer: Mixer, feed_forward: FeedForward, mixer_norm: Norm, ffn_norm: Norm,
@@ -57,12 +64,24 @@ class PreNormBlock(Part):
     def forward(self, ctx: StepContext, x: torch.Tensor, cache) -> None:
         """Run the block on the float32 stream ``x`` in place."""
         xn = ctx.workspace.rows("normed", ctx.n, self.width, ctx.act_dtype)
-        self.mixer_norm.forward(ctx, x, xn)
-        self.mixer.forward(ctx, xn, x, cache)
+        if not self.opened:
+            self.mixer_norm.forward(ctx, x, xn)
+        last = {"then": self.next_norm.after(xn)} if self.next_norm is not None else {}
         if self.feed_forward is None:
+            self.mixer.forward(ctx, xn, x, cache, **last)
             return
-        self.ffn_norm.forward(ctx, x, xn)
-        self.feed_forward.forward(ctx, xn, x)
+        if hasattr(self.ffn_norm, "after"):
+            self.mixer.forward(ctx, xn, x, cache, then=self.ffn_norm.after(xn))
+        else:
+            self.mixer.forward(ctx, xn, x, cache)
+            self.ffn_norm.forward(ctx, x, xn)
+        self.feed_forward.forward(ctx, xn, x, **last)
+
+
+def chain_norms(blocks) -> None:
+    """Blocks that run one after the other in this order, and no other way: each forms the first norm of the next."""
+    for a, b in zip(blocks, blocks[1:]):
+        a.next_norm, b.opened = b.mixer_norm, True
 
 
 class ParallelBlock(PreNormBlock):

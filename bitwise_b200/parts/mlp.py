@@ -62,8 +62,10 @@ class SwiGLU(FeedForward):
         # (only an activation other than SiLU is named to the kernels' bindings)
         return {} if self.activation == "silu" else {"activation": self.activation}
 
-    def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, accumulate: bool = True) -> None:
-        """``accumulate`` False: the output is written to ``x`` (float32) instead of added to it."""
+    def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, accumulate: bool = True,
+                then: Optional[tuple] = None) -> None:
+        """``accumulate`` False: the output is written to ``x`` (float32) instead of added to it.  ``then``: the norm that
+        follows on the finished rows (``TanhNorm.after``)."""
         ops, n = ctx.ops, ctx.n
         h = ctx.workspace.rows("ffn_h", n, self.intermediate, ctx.act_dtype)
         if self.fused:
@@ -75,7 +77,7 @@ class SwiGLU(FeedForward):
                 ops.glu_gelu(gate_up, h)
             else:
                 ops.swiglu(gate_up, h)
-        ops.linear(h, self.w_down, x, residual=x if accumulate else None)
+        ops.linear(h, self.w_down, x, residual=x if accumulate else None, **({"then": then} if then else {}))
 
 
 class DenseFFN(FeedForward):

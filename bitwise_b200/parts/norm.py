@@ -115,6 +115,10 @@ class TanhNorm(Norm):
     def param_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in (self.alpha, self.weight, self.bias))
 
+    def after(self, out):
+        """What a kernel that finishes the stream's rows needs to form this norm of them into ``out`` as well."""
+        return self.alpha, self.weight, self.bias, out
+
     def forward(self, ctx: StepContext, x, out, rows=None) -> None:
         ctx.ops.tanh_norm(x, self.alpha, self.weight, self.bias, out, rows)
 

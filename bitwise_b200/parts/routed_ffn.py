@@ -138,8 +138,9 @@ class RoutedFFN(FeedForward):
                   if t is not None)
         return own + (self.shared.param_bytes() if self.shared is not None else 0)
 
-    def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor) -> None:
-        self.forward_sum(ctx, xn, None, x)
+    def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, then: Optional[tuple] = None) -> None:
+        """``then``: the norm that follows on the finished rows (``TanhNorm.after``)."""
+        self.forward_sum(ctx, xn, None, x, then=then)
 
     def forward_scaled(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, scale: torch.Tensor) -> None:
         """``x += scale * feed_forward(xn)`` column by column (``scale`` float32 [width])."""
@@ -148,7 +149,7 @@ class RoutedFFN(FeedForward):
         self.forward_sum(ctx, xn, None, x, scale=scale)
 
     def forward_sum(self, ctx: StepContext, xn: torch.Tensor, d: Optional[torch.Tensor], x: torch.Tensor,
-                    scale: Optional[torch.Tensor] = None) -> None:
+                    scale: Optional[torch.Tensor] = None, then: Optional[tuple] = None) -> None:
         """``x += d + feed_forward(xn)``; ``d`` (float32 rows, or None) is used as scratch."""
         ops, ws, n, top = ctx.ops, ctx.workspace, ctx.n, self.top
         act = ctx.act_dtype
@@ -161,12 +162,11 @@ class RoutedFFN(FeedForward):
             logits, d_gate = z[:, :self.experts], z[:, self.experts:self.experts + 1]
         chosen = ws.rows("route_chosen", n, top, torch.int32)
         weights = ws.rows("route_weights", n, top, torch.float32)
-        ops.route(logits, self.correction, self.groups, self.keep_groups, top, self.weight_scale, chosen, weights,
-                  **self._route_options)
         lists = ws.rows("route_lists", 3, self.experts + 1, torch.int32)
         order = ws.rows("route_order", n, top, torch.int32)
         place = ws.rows("route_place", n, top, torch.int32)
-        ops.group_rows(chosen, self.experts, lists[0], lists[1:3], order, place)
+        ops.route(logits, self.correction, self.groups, self.keep_groups, top, self.weight_scale, chosen, weights,
+                  lists=(lists[0], lists[1:3], order, place), **self._route_options)
         grouped = (lists[0], lists[1:3], order)
         # the chosen experts, all in one product each for gate/up and down
         cols = self.w_gate_up.shape[1]
@@ -192,11 +192,11 @@ class RoutedFFN(FeedForward):
                 ops.add_rows(x, d)
             d = ws.rows("shared_out", n, self.width, torch.float32)
             self.shared.forward(ctx, xn, d, accumulate=False)
-            ops.combine(x, d, y, place, weights, top, scale=scale, d_gate=d_gate)
+            ops.combine(x, d, y, place, weights, top, scale=scale, d_gate=d_gate, **({"then": then} if then else {}))
             return
         if self.shared is not None:
             self.shared.forward(ctx, xn, d if d is not None else x)
-        ops.combine(x, d, y, place, weights, top, scale=scale)
+        ops.combine(x, d, y, place, weights, top, scale=scale, **({"then": then} if then else {}))
 
 
 register_feed_forward("routed", RoutedFFN)

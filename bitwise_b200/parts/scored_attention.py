@@ -210,9 +210,10 @@ class ScoredAttention(Mixer):
 
     # -- one step --------------------------------------------------------------------------
     def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, cache: PagedKVView,
-                accumulate: bool = True, projected: Optional[torch.Tensor] = None) -> None:
+                accumulate: bool = True, projected: Optional[torch.Tensor] = None, then: Optional[tuple] = None) -> None:
         """``accumulate`` False: the output is written to ``x`` instead of added to it.  ``projected``: the product
-        of ``xn`` with ``w_in`` (float32 rows) where the caller has formed it."""
+        of ``xn`` with ``w_in`` (float32 rows) where the caller has formed it.  ``then``: the norm that follows on the
+        finished rows (``TanhNorm.after``)."""
         ops, ws, n = ctx.ops, ctx.workspace, ctx.n
         gate_logits = None
         if self.gate is not None:
@@ -260,7 +261,7 @@ class ScoredAttention(Mixer):
                              dist_a=self.dist_a, dist_b=self.dist_b, sinks=self.sinks, keep_first=self.keep_first, **options)
         if self.gate is not None and self.difference is None:
             self.gate.apply(ctx, xn, mixed, gate_logits)
-        ops.linear(mixed, self.w_o, x, residual=x if accumulate else None)
+        ops.linear(mixed, self.w_o, x, residual=x if accumulate else None, **({"then": then} if then else {}))
 
 
 # A query-tile height larger than any step: the step's tile list of this height has one entry

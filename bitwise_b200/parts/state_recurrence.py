@@ -349,8 +349,9 @@ class StateSpace(_StateMixer):
         return (self.w_in, self.conv_t, self.conv_b, self.step_bias, self.rate, self.skip, self.norm, self.w_o)
 
     def forward(self, ctx: StepContext, xn: torch.Tensor, x: torch.Tensor, cache: SlotStateView,
-                accumulate: bool = True) -> None:
-        """``accumulate`` False: the output is written to ``x`` instead of added to it."""
+                accumulate: bool = True, then: Optional[tuple] = None) -> None:
+        """``accumulate`` False: the output is written to ``x`` instead of added to it.  ``then``: the norm that follows on
+        the finished rows (``TanhNorm.after``)."""
         ops, ws, n, H, ch = ctx.ops, ctx.workspace, ctx.n, self.heads, self.channels
         tiles = ctx.query_tiles(SEQUENCE_TILE)
         conv_state = cache.beside.state if self.taps > 1 else None
@@ -369,7 +370,7 @@ class StateSpace(_StateMixer):
                        step=ready[:, step:step + H], decay=ready[:, step + H:step + 2 * H], skip=self.skip)
         gated = ws.rows("scan_gated", n, self.inner, ctx.act_dtype)
         ops.gated_group_norm(o, u[:, :self.inner], self.norm, self.eps, gated, self.norm_groups)
-        ops.linear(gated, self.w_o, x, residual=x if accumulate else None)
+        ops.linear(gated, self.w_o, x, residual=x if accumulate else None, **({"then": then} if then else {}))
 
 
 register_mixer("channel_delta", ChannelDelta)

@@ -207,7 +207,11 @@ class CpuOps:
         out.copy_((g * torch.sigmoid(alpha * g) * (u + 1.0)).to(out.dtype))
 
     def route(self, logits, correction, groups, keep, top, weight_scale, chosen, weights, softmax_top=False, scoring=None,
-              group_max=False, sum_eps=None):
+              group_max=False, sum_eps=None, lists=None):
+        if lists is not None:
+            self.route(logits, correction, groups, keep, top, weight_scale, chosen, weights, softmax_top, scoring, group_max, sum_eps)
+            self.group_rows(chosen, logits.shape[1], *lists)
+            return
         if scoring == "softmax":
             if correction is not None or not group_max:
                 raise NotImplementedError("the stand-in keeps groups by their largest score")
@@ -248,12 +252,14 @@ class CpuOps:
             src = x[int(order[i]) // order_div] if gather else x[i]
             out[i] = self._activated(w[int(self._entry_expert[i])].float() @ src.float(), activation).to(out.dtype)
 
-    def combine(self, x, d, y, place, weights, top, scale=None, d_gate=None):
+    def combine(self, x, d, y, place, weights, top, scale=None, d_gate=None, then=None):
         n = x.shape[0]
         add = (weights[:, :, None] * y[place.reshape(-1).long()[:n * top]].view(n, top, -1)).sum(1)
         if d is not None:
             add = add + (d if d_gate is None else d * torch.sigmoid(d_gate))
         x += add if scale is None else scale * add
+        if then is not None:
+            self.tanh_norm(x, *then)
 
     def gla_scan(self, u, z, bias, tau, state, norm_w, eps, out, heads, dim, vdim, q_scale, ctx, tiles, scratch=None):
         t_seq, t_row0, t_rows, count = tiles
@@ -280,13 +286,15 @@ class CpuOps:
         inv = torch.rsqrt(src.pow(2).mean(-1, keepdim=True) + eps)
         out.copy_(((src * inv) * weight).to(out.dtype))
 
-    def linear(self, x, w, out, residual=None, activation=None):
+    def linear(self, x, w, out, residual=None, activation=None, then=None):
         y = x.float() @ w.float().t()
         if activation is not None:
             y = self._activated(y, activation)
         if residual is not None:
             y = residual + y
         out.copy_(y.to(out.dtype))
+        if then is not None:
+            self.tanh_norm(out, *then)
 
     # -- recurrences over a matrix of state per head, the token shift, two mixers side by side ------------
     @staticmethod

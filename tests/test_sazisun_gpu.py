@@ -350,6 +350,58 @@ def test_experts_with_the_square_of_relu_and_a_gated_shared_one(dtype, rows, exp
     assert err <= (1e-5 * float(want.abs().max()) if dtype == "float32" else 2.0 * slack + 1e-4), (err, slack)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("experts,groups,keep,top", [(8, 4, 2, 3), (5, 1, 1, 5), (64, 8, 3, 6), (256, 8, 4, 8)])
+@pytest.mark.parametrize("rows", [1, 8, 16, 17])
+def test_routing_and_its_lists_in_one_kernel(dtype, experts, groups, keep, top, rows):
+    ops = ops_of(dtype)
+    z = torch.randn(rows, experts, generator=torch.Generator().manual_seed(experts + rows)).to(DEV)
+    i32 = lambda *s: torch.full(s, -7, dtype=torch.int32, device=DEV)
+    out = []
+    for together in (False, True):
+        chosen, weights = i32(rows, top), torch.zeros(rows, top, device=DEV)
+        lists = (i32(experts + 1), i32(2, experts + 1), i32(rows, top), i32(rows, top))
+        options = dict(scoring="softmax", group_max=True, sum_eps=1e-20)
+        if together:
+            ops.route(z, None, groups, keep, top, 1.5, chosen, weights, lists=lists, **options)
+        else:
+            ops.route(z, None, groups, keep, top, 1.5, chosen, weights, **options)
+            ops.group_rows(chosen, experts, *lists)
+        out.append((chosen, weights, *lists))
+    assert all(torch.equal(a, b) for a, b in zip(*out))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rows,width,inner", [(1, 64, 128), (8, 1024, 2048), (9, 80, 192), (16, 256, 64), (17, 256, 64), (5, 50, 36), (300, 128, 64)])
+def test_a_product_and_the_norm_behind_it_in_one_kernel(dtype, rows, width, inner):
+    """The bits of the product with its residual sum and of the stand-alone norm, in steps of few rows (one kernel on the
+    serving precision) and of many; the same behind the experts' combination."""
+    ops = ops_of(dtype)
+    g = torch.Generator().manual_seed(width + rows)
+    r = lambda *s: torch.randn(*s, generator=g)
+    x, w = r(rows, inner).to(act(dtype)).to(DEV), (r(width, inner) / math.sqrt(inner)).to(act(dtype)).to(DEV)
+    res, nw, nb, alpha = r(rows, width).to(DEV), 1.0 + 0.2 * r(width).to(DEV), r(width).to(DEV), torch.tensor([0.7], device=DEV)
+    norm = lambda: torch.zeros(rows, width, dtype=act(dtype), device=DEV)
+    y, n1, y2, n2 = res.clone(), norm(), res.clone(), norm()
+    ops.linear(x, w, y, residual=y)
+    ops.tanh_norm(y, alpha, nw, nb, n1)
+    before = ops.launches
+    ops.linear(x, w, y2, residual=y2, then=(alpha, nw, nb, n2))
+    if dtype == "bfloat16" and rows <= 16 and inner % 64 == 0:
+        assert ops.launches - before == 1
+    assert torch.equal(y, y2) and torch.equal(n1, n2)
+    top = 2
+    yy, wt, d, gate = r(rows * top, width).to(DEV), r(rows, top).to(DEV), r(rows, width).to(DEV), r(rows, 5).to(DEV)[:, 3:4]
+    place = torch.randperm(rows * top, generator=g).to(torch.int32).reshape(rows, top).to(DEV)
+    a, n1, b, n2 = res.clone(), norm(), res.clone(), norm()
+    ops.combine(a, d, yy, place, wt, top, d_gate=gate)
+    ops.tanh_norm(a, alpha, nw, nb, n1)
+    ops.combine(b, d, yy, place, wt, top, d_gate=gate, then=(alpha, nw, nb, n2))
+    assert torch.equal(a, b) and torch.equal(n1, n2)
+    want = d64(res) + torch.sigmoid(d64(gate)) * d64(d) + (d64(wt)[:, :, None] * d64(yy)[place.cpu().long().reshape(-1)].view(rows, top, width)).sum(1)
+    close(a, want, "float32", "combination")
+
+
 # ---- whole models -------------------------------------------------------------------------------
 def model_of(name, dtype):
     from bitwise_b200 import Model
