@@ -1481,8 +1481,8 @@ def sazisun_kernel_table(z, pk, page=16):
         h1, gu, y = torch.empty(pr, ff, dtype=bf, device=dev), torch.empty(pr, 2 * ff, dtype=bf, device=dev), torch.empty(pr, width, device=dev)
         xs = torch.empty(pr, width, dtype=bf, device=dev)
         used = len(set(chosen.flatten().tolist()))
-        ms = time_it(lambda: ops.grouped_linear(xb, w1, h1, pr, lists=grouped, order_div=top, sorted_x=xs, activation="relu2"))
-        tms = time_it(lambda: (ops.grouped_linear(xb, w1g, gu, pr, lists=grouped, order_div=top, sorted_x=xs), ops.glu_clamped(gu, h1, 7.0, 1.7)))
+        ms = time_it(lambda: ops.grouped_linear(xb, w1, h1, pr, lists=grouped, order_div=top, sorted_x=xs, activation="relu2", max_rows=n))
+        tms = time_it(lambda: (ops.grouped_linear(xb, w1g, gu, pr, lists=grouped, order_div=top, sorted_x=xs, max_rows=n), ops.glu_clamped(gu, h1, 7.0, 1.7)))
         if prefill:
             put(f"experts_up_relu2_{label}", ms, frac_flops(2.0 * pr * ff * width, ms), tms, frac_flops(4.0 * pr * ff * width, tms), "bf16 peak",
                 "gated experts' gate/up and activation")

@@ -378,8 +378,8 @@ grouped_linear_mma_kernel(const act_t* __restrict__ x, int x_stride, int x_group
   bw::pdl_enter();
   constexpr int THREADS = WM * WN * 32;
   constexpr int TM = BM / WM, TN = BN / WN, MI = TM / 16, NI = TN / 8;
-  constexpr int XQ = BM * 4 / THREADS, WQ = BN * 4 / THREADS;  // 16-byte pieces a thread copies per slice
-  static_assert(NI % 2 == 0 && XQ >= 1 && WQ >= 1, "tile shape");
+  constexpr int XQ = (BM * 4 + THREADS - 1) / THREADS, WQ = BN * 4 / THREADS;  // 16-byte pieces a thread copies per slice
+  static_assert(NI % 2 == 0 && WQ >= 1, "tile shape");
   extern __shared__ __align__(16) unsigned char raw[];
   typedef __nv_bfloat16 (*Tile)[kMmaRow];
   __nv_bfloat16* xs_base = reinterpret_cast<__nv_bfloat16*>(raw);
@@ -423,7 +423,7 @@ grouped_linear_mma_kernel(const act_t* __restrict__ x, int x_stride, int x_group
   for (int q = 0; q < XQ; ++q) {
     const int i = i0 + lr + (THREADS / 4) * q;
     xrow[q] = nullptr;
-    if (i < i_end) {
+    if (i < i_end && lr + (THREADS / 4) * q < BM) {
       const int src = order ? order[i] / order_div : i;
       xrow[q] = x + static_cast<size_t>(src) * x_stride + (group_off ? 0 : g * x_group_cols);
     }
@@ -441,7 +441,7 @@ grouped_linear_mma_kernel(const act_t* __restrict__ x, int x_stride, int x_group
 #pragma unroll
     for (int q = 0; q < XQ; ++q) {
       const bool v = xrow[q] && kk < k;
-      bw::copy16_async(bw::smem_addr(&xs[lr + (THREADS / 4) * q][piece * 8]), v ? xrow[q] + kk : x, v);
+      if (BM * 4 >= THREADS || lr + (THREADS / 4) * q < BM) bw::copy16_async(bw::smem_addr(&xs[lr + (THREADS / 4) * q][piece * 8]), v ? xrow[q] + kk : x, v);
     }
 #pragma unroll
     for (int q = 0; q < WQ; ++q) {
@@ -689,8 +689,8 @@ BW_API int BW_FN(group_rows)(const int* chosen, int pairs, int experts, int* gro
 BW_API int BW_FN(grouped_linear)(const act_t* x, int x_stride, int x_group_cols, const int* order, int order_div,
                                  const act_t* w, void* out, int out_is_f32, int o_stride, int o_group_cols,
                                  const int* group_off, const int* tile_prefix, int rows, int groups, int n, int k,
-                                 int act, cudaStream_t stream) {
-  // act: what an output passes before it is stored (bw::out_act: 0 nothing, 1 the square of relu)
+                                 int act, int max_rows, cudaStream_t stream) {
+  // max_rows > 0: no group's list is longer (a step of few rows). act: what an output passes before it is stored (bw::out_act: 0 nothing, 1 the square of relu)
   if (act != bw::kOutNone && act != bw::kOutRelu2) {
     bw::set_error("grouped_linear: unknown activation %d", act);
     return -1;
@@ -725,6 +725,16 @@ BW_API int BW_FN(grouped_linear)(const act_t* x, int x_stride, int x_group_cols,
       return launch_grouped_mma<act_t, 128, 128, 2, 4, 4>(bgrid, stream, x, x_stride, x_group_cols, order, order_div, w,
                                                           static_cast<act_t*>(out), o_stride, o_group_cols, group_off,
                                                           prefix, rows, groups, n, k, act);
+    }
+    if (group_off && max_rows > 0 && max_rows <= 16) {
+      // a tile of 16 rows holds a whole list: the product is a stream of the experts' weights, many slices of it in flight
+      if (out_is_f32)
+        return launch_grouped_mma<float, 16, 64, 1, 4, 10>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
+                                                           static_cast<float*>(out), o_stride, o_group_cols, group_off,
+                                                           tile_prefix, rows, groups, n, k, act);
+      return launch_grouped_mma<act_t, 16, 64, 1, 4, 10>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,
+                                                         static_cast<act_t*>(out), o_stride, o_group_cols, group_off,
+                                                         tile_prefix, rows, groups, n, k, act);
     }
     if (out_is_f32)
       return launch_grouped_mma<float, 64, 64, 2, 2, 6>(grid, stream, x, x_stride, x_group_cols, order, order_div, w,

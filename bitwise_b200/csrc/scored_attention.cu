@@ -688,6 +688,7 @@ __global__ void __launch_bounds__(128) scored_difference_kernel(const Difference
 constexpr int kMmaWarps = 4;
 constexpr int kMmaRows = 16 * kMmaWarps;
 constexpr int kMmaKeys = 32;
+constexpr int kTableSlice = 264;  // page numbers of a block's keys that are staged in shared memory
 
 template <int VD16 /* value size / 16 */>
 __global__ void __launch_bounds__(kMmaWarps * 32)
@@ -696,16 +697,19 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
                             const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
                             const int* __restrict__ tile_rows, const int* __restrict__ seq_pos0,
                             const int* __restrict__ seq_row0, __nv_bfloat16* out, int o_stride, int heads, int kv_heads,
-                            int hb, int dim, int page, const ScoreArgs sa, int span_tiles, int spans, float* partial) {
+                            int hb, int dim, int page, const ScoreArgs sa, int span_tiles, int spans, float* partial, int q_rows,
+                            int bufs) {
+  // q_rows: queries that a block has room for (64, or 16 in a decode step); bufs: buffers of key tiles, 2 or 4
   bw::pdl_enter();
   extern __shared__ __align__(16) unsigned char smem_raw[];
+  __shared__ int table_slice[kTableSlice];
   constexpr int vdim = VD16 * 16;
   constexpr int VT = VD16 * 2;  // accumulator tiles of 8 value columns
   const int kst = dim + 8;      // row strides in elements: 16 bytes more than a row, so that
   const int vst_own = vdim + 8; // ldmatrix reads eight rows from eight different banks
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [64][kst]
-  __nv_bfloat16* ks_all = qs + kMmaRows * kst;                      // [2][32][kst]: the tile in use and the next
-  __nv_bfloat16* vs_all = vcache ? ks_all + 2 * kMmaKeys * kst : ks_all;  // [2][32][vst]; the keys where values are keys
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [q_rows][kst]
+  __nv_bfloat16* ks_all = qs + q_rows * kst;                        // [bufs][32][kst]: the tile in use and the next ones
+  __nv_bfloat16* vs_all = vcache ? ks_all + bufs * kMmaKeys * kst : ks_all;  // [bufs][32][vst]; the keys where values are keys
   const int vst = vcache ? vst_own : kst;
   const int t = blockIdx.x, g = blockIdx.y;
   const int rep = heads / kv_heads, v_heads = kv_heads / sa.maps, gv = g / sa.maps;
@@ -760,8 +764,16 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
       return;
     }
   }
+  // The page numbers of the block's keys, looked up once (a block walks 256 keys at most where spans are used as they are meant;
+  // longer walks look them up key by key).
+  const int slice0 = k_begin / page, slice_n = (min(k_end, last) / page) - slice0 + 1;
+  const bool staged = slice_n <= kTableSlice;
+  if (staged) {
+    for (int i = tid; i < slice_n; i += kMmaWarps * 32) table_slice[i] = bt[slice0 + i];
+    __syncthreads();
+  }
   // the queries' rows (a block with keys to walk only)
-  for (int c = tid; c < kMmaRows * dparts; c += kMmaWarps * 32) {
+  for (int c = tid; c < q_rows * dparts; c += kMmaWarps * 32) {
     const int sr = c / dparts, part = c - sr * dparts;
     const bool valid = sr < nq;
     const __nv_bfloat16* src = valid ? q + static_cast<size_t>(row0 + sr / nh) * q_stride + (h0 + sr % nh * hstep) * dim + part * 8 : q;
@@ -786,7 +798,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
       const __nv_bfloat16* src = kcache;
       if (have) {
         const int blk = page_shift >= 0 ? kp >> page_shift : kp / page, slot = kp - blk * page;
-        src = kcache + ((static_cast<size_t>(bt[blk]) * kv_heads + g) * page + slot) * dim + part_k * 8;
+        src = kcache + ((static_cast<size_t>(staged ? table_slice[blk - slice0] : bt[blk]) * kv_heads + g) * page + slot) * dim + part_k * 8;
       }
       if (part_k < dparts) bw::copy16_async(bw::smem_addr(kd + kk * kst + part_k * 8), src, have);
     }
@@ -797,24 +809,28 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
         const __nv_bfloat16* src = vcache;
         if (have) {
           const int blk = page_shift >= 0 ? kp >> page_shift : kp / page, slot = kp - blk * page;
-          src = vcache + ((static_cast<size_t>(bt[blk]) * v_heads + gv) * page + slot) * vdim + part_v * 8;
+          src = vcache + ((static_cast<size_t>(staged ? table_slice[blk - slice0] : bt[blk]) * v_heads + gv) * page + slot) * vdim + part_v * 8;
         }
         if (part_v < vparts) bw::copy16_async(bw::smem_addr(vd + kk * vst + part_v * 8), src, have);
       }
     }
-    bw::copies_commit();
   };
-  if (k_begin <= k_end) request_tile(k_begin, 0);
-  for (int k0 = k_begin, buf = 0; k0 <= k_end; k0 = skip_gap(k0 + kMmaKeys, keep_end, win_begin), buf ^= 1) {
-    // the next tile is requested while this one is used; its buffer was released by the
+  // the first tiles; every step commits one group of copies, so that waiting for all but the youngest bufs - 1 groups means
+  // that the step's tile is there
+  int k_req = k_begin, b_req = 0;
+  for (int i = 0; i < bufs - 1; ++i) {
+    if (k_req <= k_end) request_tile(k_req, b_req), k_req = skip_gap(k_req + kMmaKeys, keep_end, win_begin), ++b_req;
+    bw::copies_commit();
+  }
+  for (int k0 = k_begin, buf = 0; k0 <= k_end; k0 = skip_gap(k0 + kMmaKeys, keep_end, win_begin), buf = (buf + 1) & (bufs - 1)) {
+    // the next tiles are requested while this one is used; the buffer that the youngest takes was released by the
     // barrier at the end of the step before
-    const int k_next = skip_gap(k0 + kMmaKeys, keep_end, win_begin);
-    if (k_next <= k_end) {
-      request_tile(k_next, buf ^ 1);
-      bw::copies_wait<1>();
-    } else {
-      bw::copies_wait<0>();
+    if (k_req <= k_end) {
+      request_tile(k_req, b_req & (bufs - 1));
+      k_req = skip_gap(k_req + kMmaKeys, keep_end, win_begin), ++b_req;
     }
+    bw::copies_commit();
+    if (bufs == 4) bw::copies_wait<3>(); else bw::copies_wait<1>();
     __syncthreads();
     const __nv_bfloat16* ks = ks_all + buf * kMmaKeys * kst;
     const __nv_bfloat16* vs = vs_all + buf * kMmaKeys * vst;
@@ -982,7 +998,7 @@ int launch_scored_mma(dim3 grid, size_t smem, cudaStream_t stream, const __nv_bf
                       const __nv_bfloat16* kcache, const __nv_bfloat16* vcache, const int* block_table, int max_blocks,
                       const int* tile_seq, const int* tile_row0, const int* tile_rows, const int* seq_pos0,
                       const int* seq_row0, __nv_bfloat16* out, int o_stride, int heads, int kv_heads, int hb, int dim,
-                      int page, const ScoreArgs& sa, int span_tiles, int spans, float* partial) {
+                      int page, const ScoreArgs& sa, int span_tiles, int spans, float* partial, int q_rows, int bufs) {
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
     cudaError_t e = cudaFuncSetAttribute(scored_attention_mma_kernel<VD16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -995,7 +1011,7 @@ int launch_scored_mma(dim3 grid, size_t smem, cudaStream_t stream, const __nv_bf
   }
   bw::launch_pdl(scored_attention_mma_kernel<VD16>, grid, dim3(kMmaWarps * 32), smem, stream, q, q_stride, kcache, vcache,
                  block_table, max_blocks, tile_seq, tile_row0, tile_rows, seq_pos0, seq_row0, out, o_stride, heads, kv_heads,
-                 hb, dim, page, sa, span_tiles, spans, partial);
+                 hb, dim, page, sa, span_tiles, spans, partial, q_rows, bufs);
   return bw::launch_status();
 }
 
@@ -1154,8 +1170,11 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
   }
   const int rep = heads / kv_heads;
   const int hb = rep < kMmaRows ? rep : kMmaRows;
-  const size_t smem = (static_cast<size_t>(kMmaRows + 2 * kMmaKeys) * (dim + 8) +
-                       (vcache ? static_cast<size_t>(2 * kMmaKeys) * (vdim + 8) : 0)) * sizeof(__nv_bfloat16);
+  // A step of single rows: blocks of few queries, whose time is the way of the keys to them, ask for more tiles ahead.
+  const bool single = tiles == n && hb <= 16;
+  const int q_rows = single ? 16 : kMmaRows, bufs = single ? 4 : 2;
+  const size_t smem = (static_cast<size_t>(q_rows + bufs * kMmaKeys) * (dim + 8) +
+                       (vcache ? static_cast<size_t>(bufs * kMmaKeys) * (vdim + 8) : 0)) * sizeof(__nv_bfloat16);
   ScoreArgs sa;
   sa.scale = scale, sa.softcap = softcap, sa.sink = sink, sa.slopes = slopes, sa.window = window;
   sa.dist_a = dist_a, sa.dist_b = dist_a ? dist_b : nullptr, sa.sinks = sinks, sa.keep_first = window > 0 ? keep_first : 0;
@@ -1171,7 +1190,7 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
     rc = launch_scored_mma<V>(grid, smem, stream, static_cast<in_t>(q), q_stride, static_cast<in_t>(kcache),               \
                               static_cast<in_t>(vcache), block_table, max_blocks, tile_seq, tile_row0, tile_rows, seq_pos0, \
                               seq_row0, static_cast<__nv_bfloat16*>(out), o_stride, heads, kv_heads, hb, dim, page, sa,     \
-                              split ? kSpanTiles : 0, spans, partial);                                                      \
+                              split ? kSpanTiles : 0, spans, partial, q_rows, bufs);                                        \
     break;
   switch (vdim / 16) {
     BW_SCORED_MMA(1) BW_SCORED_MMA(2) BW_SCORED_MMA(3) BW_SCORED_MMA(4) BW_SCORED_MMA(5) BW_SCORED_MMA(6) BW_SCORED_MMA(7)

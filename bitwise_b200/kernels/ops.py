@@ -974,14 +974,15 @@ class KernelOps:
 
     def grouped_linear(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows: int, x_group_cols: int = 0,
                        o_group_cols: int = 0, lists=None, order_div: int = 1, gather: bool = True,
-                       sorted_x: Optional[torch.Tensor] = None, activation: Optional[str] = None) -> None:
+                       sorted_x: Optional[torch.Tensor] = None, activation: Optional[str] = None, max_rows: int = 0) -> None:
         """One product per group with w [groups, n, k].  Without ``lists`` every group g takes rows
         0 .. rows-1: out[r, g * o_group_cols + j] = sum_i x[r, g * x_group_cols + i] w[g, j, i].  With
         ``lists`` = (group_off, tile_prefix, order) from ``group_rows`` entry i of group g reads row
         order[i] // order_div of x (row i when ``gather`` is False) and writes row i of out; ``rows``
         is then the length of the list.  ``sorted_x``: scratch [rows, k] for the gathered rows, used
         where ``grouped_takes_tiles`` says so.  ``activation`` "relu2" (out act_dtype): the square of relu of
-        every output, in the product's epilogue."""
+        every output, in the product's epilogue.  ``max_rows`` > 0: no group's list is longer (the rows of the step, as a
+        row chooses an expert once); a step of few rows then takes tiles of 16 rows."""
         groups, n, k = w.shape
         if activation not in (None, "relu2") or (activation and out.dtype != self.act_dtype):
             raise KernelError(f"grouped_linear: activation {activation!r} on {out.dtype} outputs")
@@ -1016,7 +1017,7 @@ class KernelOps:
                 x, order, order_div = src, None, 1
         self._pcall("grouped_linear", _p(x), _c_int(x.shape[1]), _c_int(x_group_cols), _p(order), _c_int(order_div),
                     _p(w), _p(out), _c_int(int(out.dtype == torch.float32)), _c_int(out.shape[1]), _c_int(o_group_cols),
-                    _p(group_off), _p(tile_prefix), _c_int(rows), _c_int(groups), _c_int(n), _c_int(k), _c_int(act), self._stream())
+                    _p(group_off), _p(tile_prefix), _c_int(rows), _c_int(groups), _c_int(n), _c_int(k), _c_int(act), _c_int(max_rows), self._stream())
 
     def glu_clamped(self, gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float) -> None:
         """out = g' * sigmoid(alpha * g') * (u' + 1) for rows laid out [gate | up], with

@@ -176,15 +176,15 @@ class RoutedFFN(FeedForward):
         h = ws.rows("routed_h", n, top * self.inner, act).view(pairs, self.inner)
         if self.gated:
             gate_up = ws.rows("routed_gate_up", n, top * cols, act).view(pairs, cols)
-            ops.grouped_linear(xn, self.w_gate_up, gate_up, pairs, lists=grouped, order_div=top, sorted_x=sorted_x)
+            ops.grouped_linear(xn, self.w_gate_up, gate_up, pairs, lists=grouped, order_div=top, sorted_x=sorted_x, max_rows=n)
             if self.activation == "silu":
                 ops.swiglu(gate_up, h)
             else:
                 ops.glu_clamped(gate_up, h, self.limit, self.alpha)
         else:
-            ops.grouped_linear(xn, self.w_gate_up, h, pairs, lists=grouped, order_div=top, sorted_x=sorted_x, activation=self.activation)
+            ops.grouped_linear(xn, self.w_gate_up, h, pairs, lists=grouped, order_div=top, sorted_x=sorted_x, max_rows=n, activation=self.activation)
         y = ws.rows("routed_y", n, top * self.width, torch.float32).view(pairs, self.width)
-        ops.grouped_linear(h, self.w_down, y, pairs, lists=grouped, gather=False)
+        ops.grouped_linear(h, self.w_down, y, pairs, lists=grouped, gather=False, max_rows=n)
         # the shared expert adds into d (or, without d, into the stream), then everything into the stream
         if d_gate is not None:
             # a gated one waits in a buffer of its own for its factor

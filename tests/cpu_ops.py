@@ -238,7 +238,7 @@ class CpuOps:
         place.reshape(-1)[:pairs] = torch.arange(pairs, dtype=torch.int32)
 
     def grouped_linear(self, x, w, out, rows, x_group_cols=0, o_group_cols=0, lists=None, order_div=1, gather=True,
-                       sorted_x=None, activation=None):
+                       sorted_x=None, activation=None, max_rows=0):
         if lists is None:
             # one product per group over the same rows: group g reads the columns g * x_group_cols .. + k of x
             # and writes the columns g * o_group_cols .. + n of out (w: [groups, n, k])
