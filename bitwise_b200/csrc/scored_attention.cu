@@ -414,20 +414,89 @@ __device__ __forceinline__ bool key_seen(const ScoreArgs& sa, int pq, int lo, in
 }
 
 #if BW_ACT_BF16
-// The same on the serving precision's tensor-core path, where the scores come from bfloat16
-// operands: tanh through the hardware's exponential, tanh(x) = 1 - 2 / (exp(2x) + 1) (relative
-// error of a few 1e-7, against the 4e-3 of a bfloat16 operand).
-__device__ __forceinline__ float modify_score_fast(float s, const ScoreArgs& sa, const HeadBias& hb, int pq, int kp) {
+// What one of a thread's two queries (halves of its fragments) brings to a key tile, and what it carries along.
+struct QueryWalk {
+  HeadBias hb;
+  int pq, lo;   // its position, the first key it sees
+  bool ok;      // there is such a query
+  float m, l;   // running maximum; this thread's share of the sum (the shares are joined at the end)
+};
+
+// The same on the serving precision's tensor-core path, where the scores come from bfloat16 operands: tanh through the hardware's
+// exponential, tanh(x) = 1 - 2 / (exp(2x) + 1) (relative error of a few 1e-7, against the 4e-3 of a bfloat16 operand). A lane holds
+// eight scores of a key tile per query, keys kp0, kp0 + 1, kp0 + 8, .. + 25, those of query h in the entries 2h and 2h + 1.
+template <int HALVES>
+__device__ __forceinline__ void modify_scores_fast(float (&sc)[4][4], const ScoreArgs& sa, const QueryWalk (&qw)[2], int kp0) {
   if (sa.softcap > 0.0f) {
     // cap * tanh(x) = cap - 2 cap / (exp(2x) + 1), x = s * scale / cap; exp(2x) = 2^(s * cap_exp)
-    const float e = bw::exp2_approx(__fmul_rn(s, sa.cap_exp));
-    s = __fmaf_rn(__fmul_rn(-2.0f, sa.softcap), __fdividef(1.0f, __fadd_rn(e, 1.0f)), sa.softcap);
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int h = 0; h < HALVES; ++h) {
+        float& v = sc[i >> 1][2 * h + (i & 1)];
+        const float e = bw::exp2_approx(__fmul_rn(v, sa.cap_exp));
+        v = __fmaf_rn(__fmul_rn(-2.0f, sa.softcap), __fdividef(1.0f, __fadd_rn(e, 1.0f)), sa.softcap);
+      }
   } else {
-    s = __fmul_rn(s, sa.scale);
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int h = 0; h < HALVES; ++h) sc[i >> 1][2 * h + (i & 1)] = __fmul_rn(sc[i >> 1][2 * h + (i & 1)], sa.scale);
   }
-  if (sa.slopes) s = __fsub_rn(s, __fmul_rn(hb.slope, static_cast<float>(pq - kp)));
-  if (sa.dist_a) s = __fsub_rn(s, __fmul_rn(hb.a, __logf(__fmaf_rn(hb.b, static_cast<float>(pq - kp), 1.0f))));
-  return s;
+  if (sa.slopes) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int h = 0; h < HALVES; ++h) {
+        float& v = sc[i >> 1][2 * h + (i & 1)];
+        v = __fsub_rn(v, __fmul_rn(qw[h].hb.slope, static_cast<float>(qw[h].pq - (kp0 + (i >> 1) * 8 + (i & 1)))));
+      }
+  }
+  if (sa.dist_a) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int h = 0; h < HALVES; ++h) {
+        float& v = sc[i >> 1][2 * h + (i & 1)];
+        v = __fsub_rn(v, __fmul_rn(qw[h].hb.a, __logf(__fmaf_rn(qw[h].hb.b, static_cast<float>(qw[h].pq - (kp0 + (i >> 1) * 8 + (i & 1))), 1.0f))));
+      }
+  }
+}
+
+// Scores of a key tile into weights relative to the queries' running maxima, which move on with the sums; al: the factors of what
+// was accumulated before. `whole`: every query sees every key of the tile.
+template <int HALVES>
+__device__ __forceinline__ void weigh_tile(float (&sc)[4][4], const ScoreArgs& sa, QueryWalk (&qw)[2], int kp0, bool whole, float (&al)[2]) {
+  modify_scores_fast<HALVES>(sc, sa, qw, kp0);
+  float mt[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
+  if (!whole) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int h = 0; h < HALVES; ++h)
+        if (!(qw[h].ok && key_seen(sa, qw[h].pq, qw[h].lo, kp0 + (i >> 1) * 8 + (i & 1)))) sc[i >> 1][2 * h + (i & 1)] = -INFINITY;
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+#pragma unroll
+    for (int h = 0; h < HALVES; ++h) mt[h] = fmaxf(mt[h], sc[i >> 1][2 * h + (i & 1)]);
+#pragma unroll
+  for (int h = 0; h < HALVES; ++h) {
+    mt[h] = fmaxf(mt[h], __shfl_xor_sync(0xffffffffu, mt[h], 1)), mt[h] = fmaxf(mt[h], __shfl_xor_sync(0xffffffffu, mt[h], 2));
+    mt[h] = fmaxf(qw[h].m, mt[h]);
+    // (a query that has seen no key yet holds zeros, which need no factor)
+    al[h] = qw[h].m == -INFINITY ? (mt[h] == -INFINITY ? 1.0f : 0.0f) : __expf(__fsub_rn(qw[h].m, mt[h]));
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+#pragma unroll
+    for (int h = 0; h < HALVES; ++h) {
+      float& v = sc[i >> 1][2 * h + (i & 1)];
+      v = v == -INFINITY ? 0.0f : __expf(__fsub_rn(v, mt[h]));
+      sum[h] = __fadd_rn(sum[h], v);
+    }
+#pragma unroll
+  for (int h = 0; h < HALVES; ++h) qw[h].l = __fmaf_rn(qw[h].l, al[h], sum[h]), qw[h].m = mt[h];
 }
 #endif
 
@@ -688,18 +757,22 @@ __global__ void __launch_bounds__(128) scored_difference_kernel(const Difference
 constexpr int kMmaWarps = 4;
 constexpr int kMmaRows = 16 * kMmaWarps;
 constexpr int kMmaKeys = 32;
+__host__ __device__ constexpr int mma_q_rows(bool single) { return single ? 16 : kMmaRows; }  // queries that a block has room for
+__host__ __device__ constexpr int mma_bufs(bool single) { return single ? 4 : 2; }            // buffers of key tiles
 constexpr int kTableSlice = 264;  // page numbers of a block's keys that are staged in shared memory
 
-template <int VD16 /* value size / 16 */>
+// SINGLE: a step of single rows, whose blocks have at most 16 queries. All warps of a block take them then: each forms all scores and
+// weights, and every fourth part of 16 value columns is its own (the sums are the same either way); and as the block's time is the way
+// of the keys to it, more tiles are asked for ahead.
+template <int VD16 /* value size / 16 */, bool SINGLE>
 __global__ void __launch_bounds__(kMmaWarps * 32)
 scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ kcache,
                             const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_table, int max_blocks,
                             const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
                             const int* __restrict__ tile_rows, const int* __restrict__ seq_pos0,
                             const int* __restrict__ seq_row0, __nv_bfloat16* out, int o_stride, int heads, int kv_heads,
-                            int hb, int dim, int page, const ScoreArgs sa, int span_tiles, int spans, float* partial, int q_rows,
-                            int bufs) {
-  // q_rows: queries that a block has room for (64, or 16 in a decode step); bufs: buffers of key tiles, 2 or 4
+                            int hb, int dim, int page, const ScoreArgs sa, int span_tiles, int spans, float* partial) {
+  constexpr int q_rows = mma_q_rows(SINGLE), bufs = mma_bufs(SINGLE);
   bw::pdl_enter();
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int table_slice[kTableSlice];
@@ -721,16 +794,13 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   const int p0 = seq_pos0[seq] + (row0 - seq_row0[seq]);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dparts = dim >> 3, vparts = vdim >> 3;
-  // A block of at most 16 queries (a decode step's) gives them to all its warps: each forms all scores and weights, and every
-  // fourth part of 16 value columns is its own. Else a warp has 16 queries of the block. The sums are the same either way.
-  const bool narrow = nq <= 16;
-  const int wr = narrow ? 0 : warp * 16;
+  const int wr = SINGLE ? 0 : warp * 16;
   // this thread's two queries: stacked rows sa_ and sb_ of the block
   const int sr_a = wr + (lane >> 2), sr_b = sr_a + 8;
   const bool ok_a = sr_a < nq, ok_b = sr_b < nq;
   const int pq_a = p0 + (ok_a ? sr_a / nh : 0), pq_b = p0 + (ok_b ? sr_b / nh : 0);
-  const int lo_a = first_seen(sa, pq_a), lo_b = first_seen(sa, pq_b);
-  const HeadBias slope_a = head_bias(sa, h0 + sr_a % nh * hstep, ok_a), slope_b = head_bias(sa, h0 + sr_b % nh * hstep, ok_b);
+  QueryWalk qw[2] = {{head_bias(sa, h0 + sr_a % nh * hstep, ok_a), pq_a, first_seen(sa, pq_a), ok_a, -INFINITY, 0.0f},
+                     {head_bias(sa, h0 + sr_b % nh * hstep, ok_b), pq_b, first_seen(sa, pq_b), ok_b, -INFINITY, 0.0f}};
   const int keep = sa.window > 0 ? sa.keep_first : 0;
   // the positions that this warp's queries span: tiles outside are skipped by the whole warp
   const int w_first = min(wr, max(nq - 1, 0)) / nh, w_last = min(wr + 15, max(nq - 1, 0)) / nh;
@@ -739,7 +809,6 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
   const bool warp_full = wr + 15 < nq;  // all 16 stacked rows of the warp are queries
   const int w_seen_to = p0 + w_first;           // keys up to here are seen by every query of the warp ...
   const int w_seen_from = first_seen(sa, p0 + w_last);  // ... from here on
-  float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
   float acc[VT][4];
 #pragma unroll
   for (int j = 0; j < VT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
@@ -830,7 +899,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
       k_req = skip_gap(k_req + kMmaKeys, keep_end, win_begin), ++b_req;
     }
     bw::copies_commit();
-    if (bufs == 4) bw::copies_wait<3>(); else bw::copies_wait<1>();
+    bw::copies_wait<bufs - 1>();
     __syncthreads();
     const __nv_bfloat16* ks = ks_all + buf * kMmaKeys * kst;
     const __nv_bfloat16* vs = vs_all + buf * kMmaKeys * vst;
@@ -849,60 +918,23 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
         bw::mma16816(sc[2 * jp + 1], a, b[2], b[3]);
       }
     }
-    float mt_a = -INFINITY, mt_b = -INFINITY;
     // a tile that every query of the warp sees whole needs no mask
     const bool whole = warp_full && k0 + kMmaKeys - 1 <= w_seen_to && (k0 >= w_seen_from || k0 + kMmaKeys <= keep);
-    if (whole) {
+    const int kp0 = k0 + 2 * (lane & 3);
+    float al[2] = {1.0f, 1.0f};
+    if (!SINGLE || nq > 8) {
+      weigh_tile<2>(sc, sa, qw, kp0, whole, al);
+    } else {  // (a block of at most 8 queries has none in the fragments' second halves)
+      weigh_tile<1>(sc, sa, qw, kp0, whole, al);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int kp = k0 + j * 8 + 2 * (lane & 3) + e;
-          const float va = modify_score_fast(sc[j][e], sa, slope_a, pq_a, kp);
-          const float vb = modify_score_fast(sc[j][2 + e], sa, slope_b, pq_b, kp);
-          sc[j][e] = va, sc[j][2 + e] = vb;
-          mt_a = fmaxf(mt_a, va), mt_b = fmaxf(mt_b, vb);
-        }
-      }
-    } else {
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int kp = k0 + j * 8 + 2 * (lane & 3) + e;
-          float va = modify_score_fast(sc[j][e], sa, slope_a, pq_a, kp);
-          float vb = modify_score_fast(sc[j][2 + e], sa, slope_b, pq_b, kp);
-          if (!(ok_a && key_seen(sa, pq_a, lo_a, kp))) va = -INFINITY;
-          if (!(ok_b && key_seen(sa, pq_b, lo_b, kp))) vb = -INFINITY;
-          sc[j][e] = va, sc[j][2 + e] = vb;
-          mt_a = fmaxf(mt_a, va), mt_b = fmaxf(mt_b, vb);
-        }
-      }
+      for (int i = 0; i < 8; ++i) sc[i >> 1][2 + (i & 1)] = 0.0f;
     }
-    mt_a = fmaxf(mt_a, __shfl_xor_sync(0xffffffffu, mt_a, 1)), mt_a = fmaxf(mt_a, __shfl_xor_sync(0xffffffffu, mt_a, 2));
-    mt_b = fmaxf(mt_b, __shfl_xor_sync(0xffffffffu, mt_b, 1)), mt_b = fmaxf(mt_b, __shfl_xor_sync(0xffffffffu, mt_b, 2));
-    const float mn_a = fmaxf(m_a, mt_a), mn_b = fmaxf(m_b, mt_b);
-    const float al_a = m_a == -INFINITY ? 0.0f : __expf(__fsub_rn(m_a, mn_a));
-    const float al_b = m_b == -INFINITY ? 0.0f : __expf(__fsub_rn(m_b, mn_b));
-    float sum_a = 0.0f, sum_b = 0.0f;
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float pa = sc[j][e] == -INFINITY ? 0.0f : __expf(__fsub_rn(sc[j][e], mn_a));
-        const float pb = sc[j][2 + e] == -INFINITY ? 0.0f : __expf(__fsub_rn(sc[j][2 + e], mn_b));
-        sc[j][e] = pa, sc[j][2 + e] = pb;
-        sum_a = __fadd_rn(sum_a, pa), sum_b = __fadd_rn(sum_b, pb);
-      }
-    }
-    l_a = __fmaf_rn(l_a, al_a, sum_a), l_b = __fmaf_rn(l_b, al_b, sum_b);  // this thread's share; joined at the end
-    m_a = mn_a, m_b = mn_b;
     // (a maximum that stayed gives the factor exp(0) = 1 exactly: nothing to rescale then)
-    if (__any_sync(0xffffffffu, al_a != 1.0f || al_b != 1.0f)) {
+    if (__any_sync(0xffffffffu, al[0] != 1.0f || al[1] != 1.0f)) {
 #pragma unroll
       for (int j = 0; j < VT; ++j) {
-        acc[j][0] = __fmul_rn(acc[j][0], al_a), acc[j][1] = __fmul_rn(acc[j][1], al_a);
-        acc[j][2] = __fmul_rn(acc[j][2], al_b), acc[j][3] = __fmul_rn(acc[j][3], al_b);
+        acc[j][0] = __fmul_rn(acc[j][0], al[0]), acc[j][1] = __fmul_rn(acc[j][1], al[0]);
+        acc[j][2] = __fmul_rn(acc[j][2], al[1]), acc[j][3] = __fmul_rn(acc[j][3], al[1]);
       }
     }
     // weighted values: 16 keys at a time, the weights as hi + lo
@@ -918,7 +950,7 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
       }
 #pragma unroll
       for (int jp = 0; jp < VD16; ++jp) {  // 16 value columns at a time
-        if (narrow && (jp & 3) != warp) continue;
+        if (SINGLE && (jp & 3) != warp) continue;
         uint32_t b[4];
         bw::ldsm4_trans(b, bw::smem_addr(vs + (kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * vst + jp * 16 + (lane >> 4) * 8));
         bw::mma16816(acc[2 * jp], hi, b[0], b[1]);
@@ -931,6 +963,8 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     __syncthreads();  // every warp has used the tile: its buffer may be filled again
   }
   bw::copies_wait<0>();  // (a block without a key tile has not waited for its queries' copies yet)
+  const float m_a = qw[0].m, m_b = qw[1].m;
+  float l_a = qw[0].l, l_b = qw[1].l;
   l_a = __fadd_rn(l_a, __shfl_xor_sync(0xffffffffu, l_a, 1)), l_a = __fadd_rn(l_a, __shfl_xor_sync(0xffffffffu, l_a, 2));
   l_b = __fadd_rn(l_b, __shfl_xor_sync(0xffffffffu, l_b, 1)), l_b = __fadd_rn(l_b, __shfl_xor_sync(0xffffffffu, l_b, 2));
   if (span_tiles > 0) {
@@ -938,17 +972,17 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     const int colp = 2 * (lane & 3);
     if (ok_a) {
       float* rec = partial + ((static_cast<size_t>(row0 + sr_a / nh) * heads + h0 + sr_a % nh * hstep) * spans + span) * (vdim + 2);
-      if ((lane & 3) == 0 && (warp == 0 || !narrow)) rec[0] = m_a, rec[1] = l_a;
+      if ((lane & 3) == 0 && (warp == 0 || !SINGLE)) rec[0] = m_a, rec[1] = l_a;
 #pragma unroll
       for (int j = 0; j < VT; ++j)
-        if (!narrow || ((j >> 1) & 3) == warp) rec[2 + j * 8 + colp] = acc[j][0], rec[2 + j * 8 + colp + 1] = acc[j][1];
+        if (!SINGLE || ((j >> 1) & 3) == warp) rec[2 + j * 8 + colp] = acc[j][0], rec[2 + j * 8 + colp + 1] = acc[j][1];
     }
     if (ok_b) {
       float* rec = partial + ((static_cast<size_t>(row0 + sr_b / nh) * heads + h0 + sr_b % nh * hstep) * spans + span) * (vdim + 2);
-      if ((lane & 3) == 0 && (warp == 0 || !narrow)) rec[0] = m_b, rec[1] = l_b;
+      if ((lane & 3) == 0 && (warp == 0 || !SINGLE)) rec[0] = m_b, rec[1] = l_b;
 #pragma unroll
       for (int j = 0; j < VT; ++j)
-        if (!narrow || ((j >> 1) & 3) == warp) rec[2 + j * 8 + colp] = acc[j][2], rec[2 + j * 8 + colp + 1] = acc[j][3];
+        if (!SINGLE || ((j >> 1) & 3) == warp) rec[2 + j * 8 + colp] = acc[j][2], rec[2 + j * 8 + colp + 1] = acc[j][3];
     }
     return;
   }
@@ -962,14 +996,14 @@ scored_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, c
     __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_a / nh) * o_stride + (h0 + sr_a % nh * hstep) * vdim + col;
 #pragma unroll
     for (int j = 0; j < VT; ++j)
-      if (!narrow || ((j >> 1) & 3) == warp)
+      if (!SINGLE || ((j >> 1) & 3) == warp)
         *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][0], inv_a), __fmul_rn(acc[j][1], inv_a));
   }
   if (ok_b) {
     __nv_bfloat16* dst = out + static_cast<size_t>(row0 + sr_b / nh) * o_stride + (h0 + sr_b % nh * hstep) * vdim + col;
 #pragma unroll
     for (int j = 0; j < VT; ++j)
-      if (!narrow || ((j >> 1) & 3) == warp)
+      if (!SINGLE || ((j >> 1) & 3) == warp)
         *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(__fmul_rn(acc[j][2], inv_b), __fmul_rn(acc[j][3], inv_b));
   }
 }
@@ -993,15 +1027,15 @@ scored_attention_merge_kernel(const float* __restrict__ partial, __nv_bfloat16* 
   }
 }
 
-template <int VD16>
+template <int VD16, bool SINGLE>
 int launch_scored_mma(dim3 grid, size_t smem, cudaStream_t stream, const __nv_bfloat16* q, int q_stride,
                       const __nv_bfloat16* kcache, const __nv_bfloat16* vcache, const int* block_table, int max_blocks,
                       const int* tile_seq, const int* tile_row0, const int* tile_rows, const int* seq_pos0,
                       const int* seq_row0, __nv_bfloat16* out, int o_stride, int heads, int kv_heads, int hb, int dim,
-                      int page, const ScoreArgs& sa, int span_tiles, int spans, float* partial, int q_rows, int bufs) {
+                      int page, const ScoreArgs& sa, int span_tiles, int spans, float* partial) {
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
-    cudaError_t e = cudaFuncSetAttribute(scored_attention_mma_kernel<VD16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(scored_attention_mma_kernel<VD16, SINGLE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
     if (e != cudaSuccess) {
       bw::set_error("scored_attention: %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
@@ -1009,9 +1043,9 @@ int launch_scored_mma(dim3 grid, size_t smem, cudaStream_t stream, const __nv_bf
     }
     allowed = smem;
   }
-  bw::launch_pdl(scored_attention_mma_kernel<VD16>, grid, dim3(kMmaWarps * 32), smem, stream, q, q_stride, kcache, vcache,
+  bw::launch_pdl(scored_attention_mma_kernel<VD16, SINGLE>, grid, dim3(kMmaWarps * 32), smem, stream, q, q_stride, kcache, vcache,
                  block_table, max_blocks, tile_seq, tile_row0, tile_rows, seq_pos0, seq_row0, out, o_stride, heads, kv_heads,
-                 hb, dim, page, sa, span_tiles, spans, partial, q_rows, bufs);
+                 hb, dim, page, sa, span_tiles, spans, partial);
   return bw::launch_status();
 }
 
@@ -1065,10 +1099,13 @@ BW_API int BW_FN(qkv_prepare)(const float* u, int cols, const float* conv_w, con
                          reinterpret_cast<uintptr_t>(conv_wt) | reinterpret_cast<uintptr_t>(q_norm) |
                          reinterpret_cast<uintptr_t>(k_norm) | reinterpret_cast<uintptr_t>(bias) |
                          reinterpret_cast<uintptr_t>(vmix_src) | reinterpret_cast<uintptr_t>(v_keep)) & 15) == 0;
+  // (with many rows a warp takes three heads one after the other: what it looks up about the row serves them all)
+  const int per_block = kPrepWarps * (n >= 256 ? 3 : 1);
+  const dim3 grid(n, (total + per_block - 1) / per_block);
   if (by_four)
-    bw::launch_pdl(qkv_prepare_vec_kernel, dim3(n, (total + kPrepWarps - 1) / kPrepWarps), dim3(kPrepWarps * 32), 0, stream, a);
+    bw::launch_pdl(qkv_prepare_vec_kernel, grid, dim3(kPrepWarps * 32), 0, stream, a);
   else
-    bw::launch_pdl(qkv_prepare_kernel, dim3(n, (total + kPrepWarps - 1) / kPrepWarps), dim3(kPrepWarps * 32), 0, stream, a);
+    bw::launch_pdl(qkv_prepare_kernel, grid, dim3(kPrepWarps * 32), 0, stream, a);
   return bw::launch_status();
 }
 
@@ -1170,9 +1207,8 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
   }
   const int rep = heads / kv_heads;
   const int hb = rep < kMmaRows ? rep : kMmaRows;
-  // A step of single rows: blocks of few queries, whose time is the way of the keys to them, ask for more tiles ahead.
   const bool single = tiles == n && hb <= 16;
-  const int q_rows = single ? 16 : kMmaRows, bufs = single ? 4 : 2;
+  const int q_rows = mma_q_rows(single), bufs = mma_bufs(single);
   const size_t smem = (static_cast<size_t>(q_rows + bufs * kMmaKeys) * (dim + 8) +
                        (vcache ? static_cast<size_t>(bufs * kMmaKeys) * (vdim + 8) : 0)) * sizeof(__nv_bfloat16);
   ScoreArgs sa;
@@ -1185,18 +1221,21 @@ BW_API int bw_bf16_scored_attention_mma(const void* q, int q_stride, const void*
   const dim3 grid(tiles, kv_heads, (rep + hb - 1) / hb * spans);
   typedef const __nv_bfloat16* in_t;
   int rc = -1;
+#define BW_SCORED_MMA_AS(V, S)                                                                                             \
+  launch_scored_mma<V, S>(grid, smem, stream, static_cast<in_t>(q), q_stride, static_cast<in_t>(kcache),                   \
+                          static_cast<in_t>(vcache), block_table, max_blocks, tile_seq, tile_row0, tile_rows, seq_pos0,     \
+                          seq_row0, static_cast<__nv_bfloat16*>(out), o_stride, heads, kv_heads, hb, dim, page, sa,         \
+                          split ? kSpanTiles : 0, spans, partial)
 #define BW_SCORED_MMA(V)                                                                                                   \
   case V:                                                                                                                  \
-    rc = launch_scored_mma<V>(grid, smem, stream, static_cast<in_t>(q), q_stride, static_cast<in_t>(kcache),               \
-                              static_cast<in_t>(vcache), block_table, max_blocks, tile_seq, tile_row0, tile_rows, seq_pos0, \
-                              seq_row0, static_cast<__nv_bfloat16*>(out), o_stride, heads, kv_heads, hb, dim, page, sa,     \
-                              split ? kSpanTiles : 0, spans, partial, q_rows, bufs);                                        \
+    rc = single ? BW_SCORED_MMA_AS(V, true) : BW_SCORED_MMA_AS(V, false);                                                  \
     break;
   switch (vdim / 16) {
     BW_SCORED_MMA(1) BW_SCORED_MMA(2) BW_SCORED_MMA(3) BW_SCORED_MMA(4) BW_SCORED_MMA(5) BW_SCORED_MMA(6) BW_SCORED_MMA(7)
     BW_SCORED_MMA(8) BW_SCORED_MMA(16)
   }
 #undef BW_SCORED_MMA
+#undef BW_SCORED_MMA_AS
   if (rc != 0 || !split || maps > 1) return rc;
   bw::launch_pdl(scored_attention_merge_kernel, dim3((n * heads + 3) / 4), dim3(128), 0, stream,
                  static_cast<const float*>(partial), static_cast<__nv_bfloat16*>(out), o_stride, n * heads, heads, vdim, spans, sink, sinks);
