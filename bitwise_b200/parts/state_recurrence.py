@@ -340,7 +340,7 @@ class StateSpace(_StateMixer):
 
     def load_params(self, state: Dict[str, torch.Tensor], prefix: str) -> None:
         t = {k: state[f"{prefix}.{v}"] for k, v in self.names.items()}
-        self.w_in = stacked_rows([t["in"]])
+        self.w_in = stacked_rows([t["in"]], 64)  # (whole pieces of 64 columns: what the product's wide tiles take)
         self.conv_t, self.conv_b = t["conv"].t().contiguous(), t["conv_bias"]
         self.step_bias, self.skip, self.norm, self.w_o = t["step_bias"], t["skip"], t["norm"], t["out"]
         self.rate = torch.exp(t["decay_log"].double()).float()
