@@ -1325,7 +1325,7 @@ def sazisun_config(z):
         if i % 2 == 0:
             m = StateSpaceConfig(z["s_heads"], z["s_vdim"], z["state"], z["s_groups"], z["taps"], z["norm_groups"])
         else:
-            m = TwoMapAttentionConfig(z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dim"] ** -0.5, 0.6, 50.0, 5e5, z["rot_dims"],
+            m = TwoMapAttentionConfig(z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dim"] ** -0.5, 0.5, 30.0, 5e5, z["rot_dims"],
                                       WavelengthScalingConfig(8.0, 1.0, 4.0, 8192), kv_from=1 if i % 4 == 3 else None)
         f = FeedForwardConfig(z["dense_ff"]) if i == 0 else ExpertsConfig(z["ff"], z["experts"], z["top"], 2.5, z["groups"], z["keep"],
                                                                            z["shared_ff"])
@@ -1344,7 +1344,7 @@ def sazisun_twin(z):
             m = FavudraMixerConfig("gla", z["s_heads"], z["state"], z["s_vdim"], tau=16.0, decay_rank=64)
         else:
             m = FavudraMixerConfig("attention", 2 * z["heads"], z["dim"], z["vdim"], kv_heads=2 * z["kv_heads"], scale=z["dim"] ** -0.5,
-                                   conv=z["taps"], rot_base=5e5, rot_dims=z["rot_dims"], softcap=50.0, kv_from=1 if i % 4 == 3 else None)
+                                   conv=z["taps"], rot_base=5e5, rot_dims=z["rot_dims"], softcap=30.0, kv_from=1 if i % 4 == 3 else None)
         layers.append(FavudraLayerConfig(m, z["dense_ff"]))
     return FavudraConfig(vocab=z["vocab"], width=z["width"], eps=1e-5, embedding_scale=z["width"] ** 0.5, logit_scale=0.25,
                          layers=tuple(layers))
@@ -1394,9 +1394,9 @@ def sazisun_kernel_table(z, pk, page=16):
         kc, vc = rnd(nseq * blocks + 1, 2 * G, page, dim).to(bf), rnd(nseq * blocks + 1, G, page, vdim).to(bf)
         vc2 = rnd(nseq * blocks + 1, 2 * G, page, vdim).to(bf)
         q, o1, o2 = rnd(n, 2 * H * dim).to(bf), torch.empty(n, H * vdim, dtype=bf, device=dev), torch.empty(n, 2 * H * vdim, dtype=bf, device=dev)
-        lam, gate = torch.full((1,), 0.6, device=dev), rnd(n, H * vdim)
-        attend = lambda vv, oo, **k: ops.scored_attention(q, kc, vv, table, oo, 2 * H, 2 * G, dim, vdim, dim ** -0.5, 50.0, False, None, 0, b, **k)
-        ms = time_it(lambda: attend(vc, o1, difference=(lam, 0.4, 1e-5, gate, 1)))
+        lam, gate = torch.full((1,), 0.5, device=dev), rnd(n, H * vdim)
+        attend = lambda vv, oo, **k: ops.scored_attention(q, kc, vv, table, oo, 2 * H, 2 * G, dim, vdim, dim ** -0.5, 30.0, False, None, 0, b, **k)
+        ms = time_it(lambda: attend(vc, o1, difference=(lam, 0.5, 1e-5, gate, 1)))
         tms = time_it(lambda: attend(vc2, o2))
         pairs = sum(sum(p + 1 for p in range(p0, p0 + c)) for p0, c in seqs)
         if prefill:

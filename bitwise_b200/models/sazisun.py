@@ -9,8 +9,8 @@ Two kinds of mixer, in any order:
 * ``mamba2``: a state-space recurrence behind a short convolution, its output gated and normed in groups (``StateSpace``).
 
 The feed-forward is the dense gated one (SiLU), or routed: softmax scores over all experts, groups of experts of which the best
-stay eligible by their largest score, weights divided by their sum, experts with the square of relu, and a shared expert
-multiplied by the sigmoid of one number per token; or absent.  The head is the embedding table behind a last norm.
+stay eligible by their largest score, weights divided by their sum, experts with the square of relu, and a shared expert behind
+a sigmoid gate; or absent.  The head is the embedding table behind a last norm.
 
 Tensor names: ``embed``, ``final.norm``, and per layer ``l<i>.norm1``, ``l<i>.norm2`` (each with ``.b`` and ``.alpha``), ``l<i>.mix.*``
 (see the mixers), ``l<i>.mlp.{gate, up, down}`` or ``l<i>.mlp.e<k>.{up, down}``, ``l<i>.mlp.router``, ``l<i>.mlp.shared.{up, down, sg}``.
